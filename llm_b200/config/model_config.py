@@ -546,6 +546,108 @@ class PotipelConfig:
 
 
 @dataclass(frozen=True)
+class NidoraxConfig:
+    """config.json of a Nidorax folder: a decoder whose layers are listed one by one and whose norms stand behind the
+    residual sums, x <- norm(postln_alpha * x + sublayer(x)), every sublayer reading x itself.  Keys: `architecture`,
+    `width`, `vocab`, `norm.eps`, `postln_alpha`, and per layer `type`, `mixer` and `mlp` ({kind: moe, expert: {ff}, router:
+    {experts, top, groups: {count, keep}}} or null).  Mixers:
+      lightning         heads, dim, vdim, decay (a number per head)
+      latent_attention  heads, dim, rot_dim, vdim, kv_rank, scale, rot {dims, base, scaling {factor, original, fast, slow} or
+                        absent}, and kv_from (the layer whose latents it reads) where it keeps none of its own
+    The design has no length limit of its own: max_position (optional) bounds what the engine sizes its tables for."""
+
+    architecture: str
+    width: int
+    vocab: int
+    norm_eps: float
+    postln_alpha: float
+    layers: tuple                      # of dicts, validated
+    max_position: int = 131072
+    eos_token_id: Optional[int] = None
+
+    MIXERS = ("lightning", "latent_attention")
+
+    @classmethod
+    def _mixer(cls, kind: str, m: dict, where: str) -> dict:
+        if kind == "lightning":
+            mixer = {k: _take(m, k, int) for k in ("heads", "dim", "vdim")}
+            if min(mixer.values()) <= 0:
+                raise ConfigError(f"config.json: {where}: sizes must be positive")
+            decay = _take(m, "decay", list)
+            if len(decay) != mixer["heads"] or any(isinstance(d, bool) or not isinstance(d, (int, float)) or not 0 <= d <= 1
+                                                   for d in decay):
+                raise ConfigError(f"config.json: {where}.decay must list one number of 0 to 1 per head")
+            mixer["decay"] = tuple(float(d) for d in decay)
+            return mixer
+        if kind == "latent_attention":
+            mixer = {k: _take(m, k, int) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank")}
+            mixer["scale"], mixer["kv_from"] = _take(m, "scale", float), _take(m, "kv_from", int, None)
+            if min(mixer[k] for k in ("heads", "dim", "vdim", "kv_rank")) <= 0 or mixer["rot_dim"] < 0 or mixer["rot_dim"] % 2:
+                raise ConfigError(f"config.json: {where}: sizes must be positive and rot_dim even")
+            mixer["rot_dims"], mixer["rot_base"], mixer["rot_scaling"] = 0, 1.0, None
+            if mixer["rot_dim"]:
+                mixer["rot_dims"], mixer["rot_base"] = _rot_of(m, where, mixer["rot_dim"])
+                sc = m["rot"].get("scaling")
+                if sc is not None:
+                    if not isinstance(sc, dict):
+                        raise ConfigError(f"config.json: {where}.rot.scaling must be an object or null")
+                    sc = {k: _take(sc, k, float) for k in ("factor", "original", "fast", "slow")}
+                    if min(sc.values()) <= 0 or mixer["rot_base"] <= 1:
+                        raise ConfigError(f"config.json: {where}.rot.scaling: its numbers must be positive and rot.base above 1")
+                mixer["rot_scaling"] = sc
+            return mixer
+        raise ConfigError(f"config.json: {where[:-6]}.type '{kind}' is not a mixer of this design {cls.MIXERS}")
+
+    @staticmethod
+    def _mlp(ff, where: str):
+        if ff is None:
+            return None
+        mlp = _moe_of(ff, where)
+        groups = _take(ff["router"], "groups", dict, {"count": 1, "keep": 1})
+        mlp["groups"], mlp["keep"] = _take(groups, "count", int), _take(groups, "keep", int)
+        if mlp["experts"] > 256:
+            raise ConfigError(f"config.json: {where}.mlp.router: {mlp['experts']} experts (at most 256)")
+        if mlp["groups"] <= 0 or mlp["experts"] % mlp["groups"] or not (0 < mlp["keep"] <= mlp["groups"]) \
+                or mlp["top"] > mlp["keep"] * (mlp["experts"] // mlp["groups"]):
+            raise ConfigError(f"config.json: {where}.mlp.router: {mlp['experts']} experts must divide into groups.count groups, "
+                              f"1 <= keep <= count, and top fit into the kept groups")
+        return mlp
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "NidoraxConfig":
+        norm = _take(d, "norm", dict)
+        layers = _take(d, "layers", list)
+        if not layers:
+            raise ConfigError("config.json: 'layers' must list at least one layer")
+        out = []
+        for i, layer in enumerate(layers):
+            where = f"layers[{i}]"
+            if not isinstance(layer, dict):
+                raise ConfigError(f"config.json: {where} must be an object")
+            kind = _take(layer, "type", str)
+            mixer = cls._mixer(kind, _take(layer, "mixer", dict), where + ".mixer")
+            src = mixer.get("kv_from")
+            if src is not None:
+                if not (0 <= src < i) or out[src]["type"] != "latent_attention" or out[src]["mixer"]["kv_from"] is not None:
+                    raise ConfigError(f"config.json: {where}.mixer.kv_from={src} must name an earlier layer that keeps its own latents")
+                for k in ("kv_rank", "rot_dim", "rot_dims", "rot_base", "rot_scaling"):
+                    if out[src]["mixer"][k] != mixer[k]:
+                        raise ConfigError(f"config.json: {where}.mixer.{k} differs from that of layer {src}, whose latents it reads")
+            out.append({"type": kind, "mixer": mixer, "mlp": cls._mlp(layer.get("mlp"), where)})
+        eos = d.get("eos_token_id")
+        cfg = cls(architecture=_take(d, "architecture", str), width=_take(d, "width", int), vocab=_take(d, "vocab", int),
+                  norm_eps=_take(norm, "eps", float), postln_alpha=_take(d, "postln_alpha", float), layers=tuple(out),
+                  max_position=_take(d, "max_position", int, 131072), eos_token_id=eos if isinstance(eos, int) else None)
+        if cfg.width <= 0 or cfg.vocab <= 0 or cfg.max_position <= 0:
+            raise ConfigError("config.json: width, vocab and max_position must be positive")
+        return cfg
+
+    @property
+    def max_position_embeddings(self) -> int:
+        return self.max_position
+
+
+@dataclass(frozen=True)
 class Architecture:
     """One registry entry: how to read the config and how to lay the model out."""
 

@@ -1,0 +1,408 @@
+// Linear attention with one fixed decay per head:
+//
+//   S_t = d_h S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t          S [dim, vdim] per head, float32, in the request's state slot
+//
+// scan.cu walks it token by token for any sizes (its "const" form).  This file holds the two forms that real sizes run on.
+//
+// Single tokens (a decode step): the state is read and written once and everything else is small.  A CTA owns 64 columns of
+// one head's state; its 128 threads are 16 float4 columns x 8 row lanes; up to 16 rows of a thread are in flight at once.
+// q, k and v are read as they left the projection, a tensor or its unsummed split-K partial results, and pass silu here.
+//
+// Prompt portions (bfloat16): chunks of 64 tokens.  With n tokens in the chunk and S_0 the state that enters it,
+//     o_i = d^(i+1) S_0^T q_i + sum_{j <= i} d^(i-j) (q_i . k_j) v_j,       S_n = d^n S_0 + sum_j d^(n-1-j) k_j v_j^T
+// so the chunks' own contributions to the state are made side by side (chunk_state), chained from the request's state by one
+// multiply-add per chunk and element (chunk_chain, float32), and the outputs are made side by side again (chunk_out).  q, k and
+// v are bfloat16 (silu already taken, in the epilogue of the product that made them), so q . k and k v^T have exact factors;
+// every float32 operand of a product (the state, the decayed scores, the decayed values) enters it as the sum of three bfloat16
+// numbers, which hold its 24 bits, and every sum is float32.  The products are warp-level MMAs (mma.sync): their operands are
+// made in registers by the warp that uses them, and a tile is 64 rows.
+#include "common.cuh"
+
+namespace {
+
+__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+
+// ---- single tokens -----------------------------------------------------------------------------------------
+constexpr int DEC_COLS = 64, DEC_TX = DEC_COLS / 4, DEC_ROWS = 8, DEC_THREADS = DEC_TX * DEC_ROWS, DEC_BATCH = 16, DEC_MAX_DIM = 512;
+
+// proj row e: [q: heads * dim | k: heads * dim | v: heads * vdim | ...], pre-activation.  out [e, heads * vdim] float32.
+template <typename T>
+__global__ void __launch_bounds__(DEC_THREADS)
+lightning_decode_kernel(float* __restrict__ out, long long out_stride, MaybePartial<T> proj, long long proj_stride,
+                        const float* __restrict__ decay, float* __restrict__ state, long long slot_stride,
+                        const int* __restrict__ state_slots, int heads, int dim, int vdim) {
+  __shared__ float q_s[DEC_MAX_DIM], k_s[DEC_MAX_DIM];
+  __shared__ float4 part[DEC_ROWS][DEC_TX];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, tx = tid % DEC_TX, ty = tid / DEC_TX;
+  const int entry = blockIdx.z, head = blockIdx.y, col = blockIdx.x * DEC_COLS + tx * 4;
+  const size_t row = (size_t)entry * proj_stride;
+  const bool live = col < vdim;                           // vdim is a multiple of 4
+  float4* S = reinterpret_cast<float4*>(state + (size_t)state_slots[entry] * slot_stride + (size_t)head * dim * vdim + col);
+  const int pitch = vdim / 4;
+  float4 s[DEC_BATCH];
+  auto load = [&](int r0) {
+#pragma unroll
+    for (int i = 0; i < DEC_BATCH; ++i) {
+      const int r = r0 + ty + i * DEC_ROWS;
+      if (live && r < dim) s[i] = S[(size_t)r * pitch];
+    }
+  };
+  load(0);                                                // under the sums and the activations below
+  for (int d = tid; d < dim; d += DEC_THREADS) {
+    q_s[d] = silu_f(proj.at(row + (size_t)head * dim + d));
+    k_s[d] = silu_f(proj.at(row + (size_t)(heads + head) * dim + d));
+  }
+  float v[4] = {0.f, 0.f, 0.f, 0.f};
+  if (live)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) v[c] = silu_f(proj.at(row + (size_t)2 * heads * dim + (size_t)head * vdim + col + c));
+  const float d = decay[head];
+  float o[4] = {0.f, 0.f, 0.f, 0.f};
+  __syncthreads();
+  for (int r0 = 0; r0 < dim; r0 += DEC_BATCH * DEC_ROWS) {
+    if (r0) load(r0);
+#pragma unroll
+    for (int i = 0; i < DEC_BATCH; ++i) {
+      const int r = r0 + ty + i * DEC_ROWS;
+      if (!live || r >= dim) continue;
+      const float kr = k_s[r], qr = q_s[r];
+      s[i].x = fmaf(d, s[i].x, kr * v[0]); s[i].y = fmaf(d, s[i].y, kr * v[1]);
+      s[i].z = fmaf(d, s[i].z, kr * v[2]); s[i].w = fmaf(d, s[i].w, kr * v[3]);
+      o[0] = fmaf(s[i].x, qr, o[0]); o[1] = fmaf(s[i].y, qr, o[1]);
+      o[2] = fmaf(s[i].z, qr, o[2]); o[3] = fmaf(s[i].w, qr, o[3]);
+      S[(size_t)r * pitch] = s[i];
+    }
+  }
+  part[ty][tx] = make_float4(o[0], o[1], o[2], o[3]);
+  __syncthreads();
+  if (ty == 0 && live) {
+    float4 a = part[0][tx];
+#pragma unroll
+    for (int g = 1; g < DEC_ROWS; ++g) {
+      const float4 b = part[g][tx];
+      a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
+    }
+    float* dst = out + (size_t)entry * out_stride + (size_t)head * vdim + col;
+    dst[0] = a.x; dst[1] = a.y; dst[2] = a.z; dst[3] = a.w;
+  }
+}
+
+// ---- prompt portions -----------------------------------------------------------------------------------------
+constexpr int CC = 64, VT = 64, WARPS = 4, THREADS = WARPS * 32, PAD = 8, VP = VT + PAD;
+using bf16 = __nv_bfloat16;
+
+// The chunk with the running number idx: its entry, first token, length and place among its entry's chunks; false when the
+// step has fewer chunks.
+__device__ __forceinline__ bool chunk_of(const int* cu_tokens, int n_entries, int idx, int& c0, int& n) {
+  for (int e = 0; e < n_entries; ++e) {
+    const int t0 = cu_tokens[e], len = cu_tokens[e + 1] - t0, chunks = (len + CC - 1) / CC;
+    if (idx < chunks) { c0 = t0 + idx * CC; n = min(CC, len - idx * CC); return true; }
+    idx -= chunks;
+  }
+  return false;
+}
+
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void cp_async16(void* smem_dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(smem_dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory"); }
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const bf16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const bf16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
+}
+__device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// Two float32 numbers as three pairs of bfloat16 numbers whose sums they are (to the last of their 24 bits or so).
+__device__ __forceinline__ void split3(float x, float y, uint32_t (&p)[3]) {
+#pragma unroll
+  for (int i = 0; i < 3; ++i) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    p[i] = *reinterpret_cast<const uint32_t*>(&h);
+    x -= __low2float(h); y -= __high2float(h);
+  }
+}
+
+// rows [0, n) of a [.., cols] tensor into shared memory with pitch `pitch`, zeros in rows n .. CC and columns up to `cols_pad`
+// (cols a multiple of 8, cols_pad of 8)
+__device__ __forceinline__ void bring_rows(bf16* dst, int pitch, const bf16* src, long long stride, int n, int cols, int cols_pad) {
+  const int per = cols_pad / 8;
+  for (int i = threadIdx.x; i < CC * per; i += THREADS) {
+    const int r = i / per, c = (i % per) * 8;
+    bf16* at = dst + r * pitch + c;
+    if (r < n && c < cols) cp_async16(at, src + (size_t)r * stride + c);
+    else *reinterpret_cast<uint4*>(at) = make_uint4(0, 0, 0, 0);
+  }
+}
+
+// seg[chunk, head] [dim, vdim] = sum_j d^(n-1-j) k_j v_j^T.  Grid (chunks, heads, value tiles).
+__global__ void __launch_bounds__(THREADS)
+lightning_chunk_state_kernel(const bf16* __restrict__ k, const bf16* __restrict__ v, long long stride, const float* __restrict__ decay,
+                             const int* __restrict__ cu_tokens, int n_entries, int heads, int dim, int vdim, float* __restrict__ seg) {
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  pdl_launch_dependents();
+  pdl_wait();
+  int c0, n;
+  if (!chunk_of(cu_tokens, n_entries, blockIdx.x, c0, n)) return;
+  const int head = blockIdx.y, col0 = blockIdx.z * VT, kp = dim + PAD;
+  bf16* k_s = reinterpret_cast<bf16*>(smem_raw);          // [CC][dim + PAD]
+  bf16* v_s = k_s + CC * kp;                              // [3][CC][VP]: the decayed values in three pieces
+  const float d = decay[head];
+  bring_rows(k_s, kp, k + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
+  {
+    const bf16* src = v + (size_t)c0 * stride + (size_t)head * vdim + col0;
+    for (int i = threadIdx.x; i < CC * (VT / 8); i += THREADS) {
+      const int r = i / (VT / 8), c = (i % (VT / 8)) * 8;
+      float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (r < n && col0 + c < vdim) {
+        Vec8<bf16>::load(src + (size_t)r * stride + c, x);
+        const float w = powf(d, (float)(n - 1 - r));
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] *= w;
+      }
+      uint32_t p[4][3];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) split3(x[2 * j], x[2 * j + 1], p[j]);
+#pragma unroll
+      for (int s = 0; s < 3; ++s)
+        *reinterpret_cast<uint4*>(v_s + (s * CC + r) * VP + c) = make_uint4(p[0][s], p[1][s], p[2][s], p[3][s]);
+    }
+  }
+  cp_async_wait_all();
+  __syncthreads();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float* dst = seg + ((size_t)blockIdx.x * heads + head) * dim * vdim;
+  for (int m0 = warp * 16; m0 < dim; m0 += WARPS * 16) {  // 16 rows of the state at a time
+    float acc[VT / 8][4];
+#pragma unroll
+    for (int i = 0; i < VT / 8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+#pragma unroll
+    for (int t0 = 0; t0 < CC; t0 += 16) {
+      uint32_t a[4];
+      ldsm4_t(a, k_s + (t0 + (lane & 7) + ((lane >> 4) << 3)) * kp + m0 + (((lane >> 3) & 1) << 3));
+#pragma unroll
+      for (int s = 0; s < 3; ++s)
+#pragma unroll
+        for (int x = 0; x < VT / 16; ++x) {
+          uint32_t b[4];
+          ldsm4_t(b, v_s + (s * CC + t0 + (lane & 15)) * VP + x * 16 + ((lane >> 4) << 3));
+          mma(acc[2 * x], a, b[0], b[1]);
+          mma(acc[2 * x + 1], a, b[2], b[3]);
+        }
+    }
+    const int r = m0 + (lane >> 2);
+#pragma unroll
+    for (int x = 0; x < VT / 8; ++x) {
+      const int c = col0 + x * 8 + 2 * (lane & 3);
+      if (c >= vdim) continue;
+      *reinterpret_cast<float2*>(dst + (size_t)r * vdim + c) = make_float2(acc[x][0], acc[x][1]);
+      *reinterpret_cast<float2*>(dst + (size_t)(r + 8) * vdim + c) = make_float2(acc[x][2], acc[x][3]);
+    }
+  }
+}
+
+// seg[chunk] holds the chunk's own contribution on entry and the state that enters the chunk on exit; the request's state
+// moves to the end of the entry.  A thread per four elements of the state; eight chunks' loads are issued together.
+__global__ void __launch_bounds__(256)
+lightning_chunk_chain_kernel(float* __restrict__ seg, const float* __restrict__ decay, float* __restrict__ state, long long slot_stride,
+                             const int* __restrict__ state_slots, const int* __restrict__ cu_tokens, int heads, int dim, int vdim) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t per = (size_t)heads * dim * vdim / 4;
+  const size_t el = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (el >= per) return;
+  const int entry = blockIdx.y;
+  size_t first = 0;
+  for (int e = 0; e < entry; ++e) first += (cu_tokens[e + 1] - cu_tokens[e] + CC - 1) / CC;
+  const int len = cu_tokens[entry + 1] - cu_tokens[entry], chunks = (len + CC - 1) / CC;
+  const float d = decay[el / ((size_t)dim * vdim / 4)];
+  const float whole = powf(d, (float)CC), last = powf(d, (float)(len - (chunks - 1) * CC));
+  float4* S_g = reinterpret_cast<float4*>(state + (size_t)state_slots[entry] * slot_stride) + el;
+  float4* at = reinterpret_cast<float4*>(seg) + first * per + el;
+  float4 S = *S_g;
+  for (int c0 = 0; c0 < chunks; c0 += 8) {
+    float4 own[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (c0 + i < chunks) own[i] = at[(size_t)(c0 + i) * per];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (c0 + i >= chunks) break;
+      at[(size_t)(c0 + i) * per] = S;
+      const float w = c0 + i + 1 < chunks ? whole : last;
+      S.x = fmaf(w, S.x, own[i].x); S.y = fmaf(w, S.y, own[i].y); S.z = fmaf(w, S.z, own[i].z); S.w = fmaf(w, S.w, own[i].w);
+    }
+  }
+  *S_g = S;
+}
+
+// The outputs of a chunk: a warp per 16 tokens.  Grid (chunks, heads, value tiles).
+__global__ void __launch_bounds__(THREADS)
+lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const bf16* __restrict__ q, const bf16* __restrict__ k,
+                           const bf16* __restrict__ v, long long stride, const float* __restrict__ decay,
+                           const int* __restrict__ cu_tokens, int n_entries, int heads, int dim, int vdim,
+                           const float* __restrict__ seg) {
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  __shared__ float pw[CC + 1];
+  pdl_launch_dependents();
+  pdl_wait();
+  int c0, n;
+  if (!chunk_of(cu_tokens, n_entries, blockIdx.x, c0, n)) return;
+  const int head = blockIdx.y, col0 = blockIdx.z * VT, kp = dim + PAD;
+  bf16* q_s = reinterpret_cast<bf16*>(smem_raw);          // [CC][dim + PAD]
+  bf16* k_s = q_s + CC * kp;                              // [CC][dim + PAD]
+  bf16* v_s = k_s + CC * kp;                              // [CC][VP]
+  bf16* S_s = v_s + CC * VP;                              // [3][dim][VP]: the state that enters the chunk in three pieces
+  bring_rows(q_s, kp, q + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
+  bring_rows(k_s, kp, k + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
+  bring_rows(v_s, VP, v + (size_t)c0 * stride + (size_t)head * vdim + col0, stride, n, min(VT, vdim - col0), VT);
+  const float d = decay[head];
+  if (threadIdx.x <= CC) pw[threadIdx.x] = powf(d, (float)threadIdx.x);
+  {
+    const float* src = seg + ((size_t)blockIdx.x * heads + head) * dim * vdim + col0;
+    for (int i = threadIdx.x; i < dim * (VT / 8); i += THREADS) {
+      const int r = i / (VT / 8), c = (i % (VT / 8)) * 8;
+      float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (col0 + c < vdim) Vec8<float>::load(src + (size_t)r * vdim + c, x);
+      uint32_t p[4][3];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) split3(x[2 * j], x[2 * j + 1], p[j]);
+#pragma unroll
+      for (int s = 0; s < 3; ++s)
+        *reinterpret_cast<uint4*>(S_s + (s * dim + r) * VP + c) = make_uint4(p[0][s], p[1][s], p[2][s], p[3][s]);
+    }
+  }
+  cp_async_wait_all();
+  __syncthreads();
+  const int lane = threadIdx.x & 31, i0 = (threadIdx.x >> 5) * 16;
+  if (i0 >= n) return;
+  const bf16* q_at = q_s + (i0 + (lane & 15)) * kp + ((lane >> 4) << 3);
+  float o[VT / 8][4];
+#pragma unroll
+  for (int i = 0; i < VT / 8; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
+  // what the state that enters the chunk contributes: d^(i+1) S_0^T q_i
+#pragma unroll 2
+  for (int k0 = 0; k0 < dim; k0 += 16) {
+    uint32_t a[4];
+    ldsm4(a, q_at + k0);
+#pragma unroll
+    for (int s = 0; s < 3; ++s)
+#pragma unroll
+      for (int x = 0; x < VT / 16; ++x) {
+        uint32_t b[4];
+        ldsm4_t(b, S_s + (s * dim + k0 + (lane & 15)) * VP + x * 16 + ((lane >> 4) << 3));
+        mma(o[2 * x], a, b[0], b[1]);
+        mma(o[2 * x + 1], a, b[2], b[3]);
+      }
+  }
+  const int ra = i0 + (lane >> 2), rb = ra + 8;           // the lane's two rows
+#pragma unroll
+  for (int x = 0; x < VT / 8; ++x) {
+    o[x][0] *= pw[ra + 1]; o[x][1] *= pw[ra + 1];
+    o[x][2] *= pw[rb + 1]; o[x][3] *= pw[rb + 1];
+  }
+  // the chunk's own tokens, 16 keys at a time up to the warp's last row
+  for (int j0 = 0; j0 <= i0; j0 += 16) {
+    float p[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll 4
+    for (int k0 = 0; k0 < dim; k0 += 16) {
+      uint32_t a[4], b[4];
+      ldsm4(a, q_at + k0);
+      ldsm4(b, k_s + (j0 + (lane & 7) + ((lane >> 4) << 3)) * kp + k0 + (((lane >> 3) & 1) << 3));
+      mma(p[0], a, b[0], b[1]);
+      mma(p[1], a, b[2], b[3]);
+    }
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int dist = (c < 2 ? ra : rb) - (j0 + 8 * x + 2 * (lane & 3) + (c & 1));
+        p[x][c] = dist >= 0 ? p[x][c] * pw[dist] : 0.f;
+      }
+    uint32_t w[4][3];
+    split3(p[0][0], p[0][1], w[0]);
+    split3(p[0][2], p[0][3], w[1]);
+    split3(p[1][0], p[1][1], w[2]);
+    split3(p[1][2], p[1][3], w[3]);
+#pragma unroll
+    for (int x = 0; x < VT / 16; ++x) {
+      uint32_t b[4];
+      ldsm4_t(b, v_s + (j0 + (lane & 15)) * VP + x * 16 + ((lane >> 4) << 3));
+#pragma unroll
+      for (int s = 0; s < 3; ++s) {
+        const uint32_t a[4] = {w[0][s], w[1][s], w[2][s], w[3][s]};
+        mma(o[2 * x], a, b[0], b[1]);
+        mma(o[2 * x + 1], a, b[2], b[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int x = 0; x < VT / 8; ++x) {
+    const int c = col0 + x * 8 + 2 * (lane & 3);
+    if (c >= vdim) continue;
+    float* dst = out + (size_t)head * vdim + c;
+    if (ra < n) *reinterpret_cast<float2*>(dst + (size_t)(c0 + ra) * out_stride) = make_float2(o[x][0], o[x][1]);
+    if (rb < n) *reinterpret_cast<float2*>(dst + (size_t)(c0 + rb) * out_stride) = make_float2(o[x][2], o[x][3]);
+  }
+}
+
+}  // namespace
+
+// One token per entry.  proj: rows [q | k | v | ...] of the element kind, or float32 partial results [splits][rows][stride]; silu
+// is taken here.  state: slot s at state + s * slot_stride, [heads, dim, vdim] float32; vdim a multiple of 4, dim up to 512.
+LLMK_API int llmk_lightning_decode(float* out, long long out_stride, const void* proj, const float* partials, int splits,
+                                   long long split_stride, long long proj_stride, const float* decay, float* state,
+                                   long long slot_stride, const int* state_slots, int n_entries, int heads, int dim, int vdim,
+                                   int dtype, cudaStream_t stream) {
+  if (n_entries == 0) return 0;
+  LLMK_REQUIRE((proj != nullptr) != (partials != nullptr), "lightning_decode: give proj or partials");
+  LLMK_REQUIRE(dim > 0 && dim <= DEC_MAX_DIM && vdim > 0 && vdim % 4 == 0, "lightning_decode: key size %d (1 to %d) or value size %d (a multiple of 4)",
+               dim, DEC_MAX_DIM, vdim);
+  LLMK_REQUIRE(slot_stride % 4 == 0 && (uintptr_t)state % 16 == 0, "lightning_decode: the state must lie on the 16-byte grid");
+  LLMK_REQUIRE(n_entries <= 65535 && heads <= 65535, "lightning_decode: too many entries or heads for one launch");
+  return dispatch_dtype(dtype, [&](auto* tag) {
+    using T = LLMK_ELEM(tag);
+    MaybePartial<T> p{(const T*)proj, partials, splits, split_stride};
+    launch_kernel(lightning_decode_kernel<T>, dim3((vdim + DEC_COLS - 1) / DEC_COLS, heads, n_entries), dim3(DEC_THREADS), 0, stream, out,
+                  out_stride, p, proj_stride, decay, state, slot_stride, state_slots, heads, dim, vdim);
+    LLMK_LAUNCH_CHECK("lightning_decode");
+  });
+}
+
+// Entries of any length, bfloat16 q, k, v with silu already taken (one row stride; head h at column h * dim, of v h * vdim).
+// dim a multiple of 16 up to 256, vdim of 8.  seg: float32 scratch [n_tokens / 64 + n_entries, heads, dim, vdim].
+LLMK_API int llmk_lightning_chunks(float* out, long long out_stride, const void* q, const void* k, const void* v, long long stride,
+                                   const float* decay, float* state, long long slot_stride, const int* state_slots,
+                                   const int* cu_tokens, int n_entries, int n_tokens, int heads, int dim, int vdim, float* seg,
+                                   cudaStream_t stream) {
+  if (n_entries == 0 || n_tokens == 0) return 0;
+  LLMK_REQUIRE(dim > 0 && dim % 16 == 0 && dim <= 256 && vdim > 0 && vdim % 8 == 0,
+               "lightning_chunks: key size %d (a multiple of 16 up to 256) or value size %d (a multiple of 8)", dim, vdim);
+  LLMK_REQUIRE(stride % 8 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0 && (uintptr_t)v % 16 == 0 && out_stride % 2 == 0 &&
+                   (uintptr_t)out % 8 == 0 && slot_stride % 4 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)seg % 16 == 0,
+               "lightning_chunks: operands off the 16-byte grid");
+  LLMK_REQUIRE(n_entries <= 65535 && heads <= 65535, "lightning_chunks: too many entries or heads for one launch");
+  const int chunks = n_tokens / CC + n_entries, tiles = (vdim + VT - 1) / VT;
+  const size_t smem1 = ((size_t)CC * (dim + PAD) + 3 * CC * VP) * sizeof(bf16);
+  const size_t smem3 = ((size_t)2 * CC * (dim + PAD) + CC * VP + (size_t)3 * dim * VP) * sizeof(bf16);
+  cudaFuncSetAttribute(lightning_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+  cudaFuncSetAttribute(lightning_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
+  launch_kernel(lightning_chunk_state_kernel, dim3(chunks, heads, tiles), dim3(THREADS), smem1, stream, (const bf16*)k, (const bf16*)v, stride,
+                decay, cu_tokens, n_entries, heads, dim, vdim, seg);
+  const size_t per = (size_t)heads * dim * vdim / 4;
+  launch_kernel(lightning_chunk_chain_kernel, dim3((unsigned)((per + 255) / 256), n_entries), dim3(256), 0, stream, seg, decay, state,
+                slot_stride, state_slots, cu_tokens, heads, dim, vdim);
+  launch_kernel(lightning_chunk_out_kernel, dim3(chunks, heads, tiles), dim3(THREADS), smem3, stream, out, out_stride, (const bf16*)q,
+                (const bf16*)k, (const bf16*)v, stride, decay, cu_tokens, n_entries, heads, dim, vdim, (const float*)seg);
+  LLMK_LAUNCH_CHECK("lightning_chunks");
+}

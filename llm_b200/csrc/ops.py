@@ -35,6 +35,15 @@ class PartialSum:
         return self.rows * self.cols
 
 
+class WeightedRows:
+    """The result of a routed feed-forward before its last sum: row t is sum_j weights[t, j] * y[pair_slot[t, j]] for y
+    float32 [slots, cols] (a slot of -1 counts nothing).  The norm behind the residual sum takes it as it is (sum_rmsnorm);
+    the buffers are valid until the next routed feed-forward runs."""
+
+    def __init__(self, y: torch.Tensor, pair_slot: torch.Tensor, weights: torch.Tensor, top: int, rows: int):
+        self.y, self.pair_slot, self.weights, self.top, self.rows = y, pair_slot, weights, top, rows
+
+
 def _split_args(x):
     """(direct pointer, partials pointer, splits, split stride) of a tensor, a PartialSum or None."""
     if isinstance(x, PartialSum):
@@ -146,6 +155,46 @@ def add_rmsnorm(resid: torch.Tensor, delta, gamma: torch.Tensor, out, rows: int,
                                    c_int(hidden), c_float(eps), c_int(_kind(ref.dtype)), _stream()))
 
 
+def sum_rmsnorm(resid: torch.Tensor, alpha: float, y, gain: torch.Tensor, out, rows: int, eps: float, dtype: torch.dtype) -> None:
+    """The norm behind a residual sum, in float32: resid[:rows] = rms(alpha * resid + y) * gain; out[:rows] (if given) the
+    same rows in the compute dtype.  y: a tensor of that dtype, a PartialSum or WeightedRows."""
+    hidden = resid.shape[-1]
+    assert resid.dtype == gain.dtype == torch.float32 and resid.is_contiguous() and gain.is_contiguous() and gain.numel() == hidden
+    assert out is None or (out.is_contiguous() and out.shape[-1] == hidden and out.dtype == dtype)
+    wy = slots = weights = None
+    top = 0
+    if isinstance(y, WeightedRows):
+        wy, slots, weights, top = y.y, y.pair_slot, y.weights, y.top
+        assert wy.dtype == weights.dtype == torch.float32 and slots.dtype == torch.int32 and wy.is_contiguous() and wy.shape[1] == hidden
+        assert slots.is_contiguous() and weights.is_contiguous() and slots.numel() >= rows * top and weights.numel() >= rows * top
+        y = None
+    elif isinstance(y, PartialSum):
+        assert y.cols == hidden and y.rows == rows
+    else:
+        assert y.is_contiguous() and y.shape[-1] == hidden and y.dtype == dtype
+    d, parts, splits, stride = _split_args(y)
+    _check(load().llmk_sum_rmsnorm(_ptr(resid), c_float(alpha), d, parts, splits, stride, _ptr(wy), _ptr(slots), _ptr(weights), c_int(top),
+                                   _ptr(gain), _ptr(out), c_int(rows), c_int(hidden), c_float(eps), c_int(_kind(dtype)), _stream()))
+
+
+def row_rmsnorm_sigmoid(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, gate, gate_col: int, rows: int, eps: float) -> None:
+    """out[:rows] = x / sqrt(mean(x^2) + eps) * w * sigmoid(gate[:, gate_col:gate_col + n]) over whole rows of x float32
+    [rows, n]; gate: a tensor of out's dtype (unit column stride) or a PartialSum."""
+    n = x.shape[-1]
+    assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and out.shape[-1] == n
+    assert w.dtype == torch.float32 and w.is_contiguous() and w.numel() == n and gate.dtype == out.dtype
+    if isinstance(gate, PartialSum):
+        assert gate.cols >= gate_col + n and gate.rows == rows
+        gate_stride = gate.cols
+    else:
+        _rows_contig(gate, "gate")
+        assert gate.shape[1] >= gate_col + n
+        gate_stride = gate.stride(0)
+    d, parts, splits, stride = _split_args(gate)
+    _check(load().llmk_row_rmsnorm_sigmoid(_ptr(out), _ptr(x), _ptr(w), d, parts, splits, stride, c_longlong(gate_stride),
+                                           c_longlong(gate_col), c_int(rows), c_int(n), c_float(eps), c_int(_kind(out.dtype)), _stream()))
+
+
 def add_dyt(resid: torch.Tensor, delta, w: torch.Tensor, b: torch.Tensor, alpha: float, out, rows: int) -> None:
     """resid[:rows] += delta (a tensor or a PartialSum, if given); out[:rows] = tanh(alpha * resid) * w + b
     (if out given): Dynamic Tanh, a norm without statistics."""
@@ -220,10 +269,11 @@ def head_rmsnorm_gate(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, gate,
 
 
 def rope_pairs_kv_write(qkv, freqs, positions: torch.Tensor, slot_map, k_pages, v_pages, n_tokens: int, n_heads: int,
-                        n_kv: int, dim: int, vdim: int, q_out=None) -> torch.Tensor:
+                        n_kv: int, dim: int, vdim: int, q_out=None, amp: float = 1.0) -> torch.Tensor:
     """Rotate the neighbouring pairs (2i, 2i+1), i < len(freqs), of every q and k head by position * freqs[i] and store
     k and v at slot_map in the pages (n_kv 0: queries only).  qkv is a tensor [T, >= n_heads*dim + n_kv*(dim+vdim)]
-    (q is then rotated in place unless q_out is given) or a PartialSum (q_out required).  Returns the rotated q."""
+    (q is then rotated in place unless q_out is given) or a PartialSum (q_out required); amp multiplies cos and sin.  Returns the
+    rotated q."""
     assert positions.dtype == torch.int32
     width = n_heads * dim + n_kv * (dim + vdim)
     if isinstance(qkv, PartialSum):
@@ -248,7 +298,7 @@ def rope_pairs_kv_write(qkv, freqs, positions: torch.Tensor, slot_map, k_pages, 
     _check(load().llmk_rope_pairs_kv_write(d, parts, splits, stride, c_longlong(src_stride), _ptr(q_out), c_longlong(q_out.stride(0)),
                                            _ptr(freqs), c_int(pairs), _ptr(positions), _ptr(slot_map), _ptr(k_pages), _ptr(v_pages),
                                            c_int(n_tokens), c_int(n_heads), c_int(n_kv), c_int(dim), c_int(vdim), c_int(page),
-                                           c_int(_kind(qkv.dtype)), _stream()))
+                                           c_int(_kind(qkv.dtype)), _stream(), c_float(amp)))
     return q_out
 
 
@@ -570,6 +620,83 @@ def gate_scan(out: torch.Tensor, q: torch.Tensor, v: torch.Tensor, z: torch.Tens
         count_launches(2)
 
 
+def const_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, ctx,
+               heads: int, dim: int, vdim: int, seg_len: int = 0, seg_state=None, seg_decay=None) -> None:
+    """S_t = decay_h S_(t-1) + silu(k_t) silu(v_t)^T, o_t = S_t^T silu(q_t) per head (scan.cu), for any sizes.  q, k
+    [T, heads*dim] and v [T, heads*vdim]: column ranges of one projection in the compute dtype, pre-activation; decay float32
+    [heads]; state float32 [slots, >= heads*dim*vdim]; out float32 [T, heads*vdim].  Segments as in wkv_scan."""
+    for t in (out, q, k, v, state):
+        _rows_contig(t, "const_scan operand")
+    assert q.stride(0) == k.stride(0) == v.stride(0) and q.dtype == k.dtype == v.dtype
+    assert q.shape[1] == k.shape[1] == heads * dim and v.shape[1] == out.shape[1] == heads * vdim
+    assert out.dtype == state.dtype == decay.dtype == torch.float32 and decay.numel() == heads and state.shape[1] >= heads * dim * vdim
+    _check(load().llmk_const_scan(_ptr(out), c_longlong(out.stride(0)), _ptr(q), _ptr(k), _ptr(v), c_longlong(q.stride(0)), _ptr(decay),
+                                  _ptr(state), c_longlong(state.stride(0)), _ptr(ctx.state_slots), _ptr(ctx.cu_tokens), c_int(ctx.n_entries),
+                                  c_int(heads), c_int(dim), c_int(vdim), c_int(_kind(q.dtype)), _stream(), c_int(ctx.n_tokens),
+                                  c_int(seg_len), *_segment_scratch(ctx, seg_len, seg_state, seg_decay, heads * dim * vdim, heads * dim)))
+    if seg_len:
+        count_launches(2)
+
+
+# ---- linear attention with a fixed decay per head (lightning.cu) ---------------------------
+
+LIGHTNING_CHUNK = 64       # tokens per chunk of a prompt portion
+
+
+def lightning_decode_available(dim: int, vdim: int, state: torch.Tensor) -> bool:
+    """Whether the single-token kernel takes these sizes."""
+    return dim <= 512 and vdim % 4 == 0 and state.stride(0) % 4 == 0 and state.data_ptr() % 16 == 0
+
+
+def lightning_decode(out: torch.Tensor, proj, decay: torch.Tensor, state: torch.Tensor, ctx, heads: int, dim: int, vdim: int) -> None:
+    """One token per entry: row e of proj (a tensor or a PartialSum) is [q | k | v | ...], pre-activation; as const_scan."""
+    cols = heads * (2 * dim + vdim)
+    n = ctx.n_entries
+    if isinstance(proj, PartialSum):
+        assert proj.cols >= cols and proj.rows == n
+        stride = proj.cols
+    else:
+        _rows_contig(proj, "proj")
+        assert proj.shape[1] >= cols
+        stride = proj.stride(0)
+    _rows_contig(out, "out"); _rows_contig(state, "state")
+    assert out.dtype == state.dtype == decay.dtype == torch.float32 and decay.numel() == heads
+    assert out.shape[1] == heads * vdim and state.shape[1] >= heads * dim * vdim and ctx.n_tokens == n
+    d, parts, splits, split_stride = _split_args(proj)
+    _check(load().llmk_lightning_decode(_ptr(out), c_longlong(out.stride(0)), d, parts, splits, split_stride, c_longlong(stride), _ptr(decay),
+                                        _ptr(state), c_longlong(state.stride(0)), _ptr(ctx.state_slots), c_int(n), c_int(heads), c_int(dim),
+                                        c_int(vdim), c_int(_kind(proj.dtype)), _stream()))
+
+
+def lightning_chunks_available(dtype, dim: int, vdim: int, stride: int, heads: int) -> bool:
+    """Whether the chunk-wise kernels take these sizes (bfloat16 operands on the 16-byte grid)."""
+    return (dtype == torch.bfloat16 and dim % 16 == 0 and dim <= 256 and vdim % 8 == 0 and stride % 8 == 0
+            and (heads * dim) % 8 == 0)
+
+
+def lightning_chunk_scratch(n_chunks: int, heads: int, dim: int, vdim: int) -> int:
+    """Float32 elements of the chunk-wise form's scratch for n_chunks chunks."""
+    return n_chunks * heads * dim * vdim
+
+
+def lightning_chunks(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor,
+                     ctx, heads: int, dim: int, vdim: int, scratch: torch.Tensor) -> None:
+    """const_scan for entries of any length on the tensor cores, chunk by chunk (lightning.cu): q, k, v bfloat16 with silu
+    already taken.  scratch: flat float32 of at least lightning_chunk_scratch(n_tokens // 64 + n_entries, ...) elements."""
+    for t in (out, q, k, v, state):
+        _rows_contig(t, "lightning_chunks operand")
+    assert q.stride(0) == k.stride(0) == v.stride(0) and q.dtype == k.dtype == v.dtype == torch.bfloat16
+    assert q.shape[1] == k.shape[1] == heads * dim and v.shape[1] == out.shape[1] == heads * vdim
+    assert out.dtype == state.dtype == decay.dtype == scratch.dtype == torch.float32 and decay.numel() == heads
+    assert state.shape[1] >= heads * dim * vdim and scratch.is_contiguous()
+    assert scratch.numel() >= lightning_chunk_scratch(ctx.n_tokens // LIGHTNING_CHUNK + ctx.n_entries, heads, dim, vdim)
+    _check(load().llmk_lightning_chunks(_ptr(out), c_longlong(out.stride(0)), _ptr(q), _ptr(k), _ptr(v), c_longlong(q.stride(0)), _ptr(decay),
+                                        _ptr(state), c_longlong(state.stride(0)), _ptr(ctx.state_slots), _ptr(ctx.cu_tokens),
+                                        c_int(ctx.n_entries), c_int(ctx.n_tokens), c_int(heads), c_int(dim), c_int(vdim), _ptr(scratch),
+                                        _stream()))
+    count_launches(2)
+
+
 def delta_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b: torch.Tensor, a: torch.Tensor,
                a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, ctx, heads: int, qk_heads: int, dim: int,
                vdim: int, q_scale: float, norm_eps: float = 1e-6) -> None:
@@ -667,8 +794,40 @@ def clamped_glu(out: torch.Tensor, gate_up, bias, rows: int, limit: float, alpha
                                    c_float(alpha), c_int(_kind(out.dtype)), _stream()))
 
 
+def latent_q_rope_store(x, q_out: torch.Tensor, heads: int, dim: int, gain, rank: int, rot: int, freqs, amp: float, positions,
+                        eps: float, slot_map, pages, n_tokens: int) -> None:
+    """Queries and latents of one product: x [T, heads * (rot + dim) + rank + rot] (a float32 tensor or a PartialSum) holds per
+    head [rot channels that turn | dim plain], then the latent and the shared rotated key part.  q_out [T, heads * (rot + dim)]
+    gets the queries with pairs (2i, 2i+1), i < len(freqs), of every head turned by position * freqs[i] (cos and sin times
+    amp); the token's cache row pages[slot_map[t]] = [turned key part | rms(latent) * gain | zeros].  pages None: queries only
+    (x may then end after them)."""
+    per = heads * (rot + dim)
+    width = per + (rank + rot if pages is not None else 0)
+    if isinstance(x, PartialSum):
+        assert x.cols >= width and x.rows == n_tokens
+        x_stride = x.cols
+    else:
+        _rows_contig(x, "x")
+        assert x.dtype == torch.float32 and x.shape[1] >= width
+        x_stride = x.stride(0)
+    _rows_contig(q_out, "q_out")
+    assert q_out.shape[1] == per and positions.dtype == torch.int32
+    pairs = 0 if freqs is None else freqs.numel()
+    assert freqs is None or (freqs.dtype == torch.float32 and freqs.is_contiguous())
+    row_width = 0
+    if pages is not None:
+        assert pages.is_contiguous() and pages.shape[1] == 1 and pages.dtype == q_out.dtype and slot_map.dtype == torch.int32
+        assert gain.dtype == torch.float32 and gain.is_contiguous() and gain.numel() == rank
+        row_width = pages.shape[3]
+    d, parts, splits, stride = _split_args(x)
+    _check(load().llmk_latent_q_rope_store(d, parts, splits, stride, c_longlong(x_stride), _ptr(q_out), c_longlong(q_out.stride(0)), c_int(heads),
+                                           c_int(dim), _ptr(gain if pages is not None else None), c_int(rank), c_int(rot), _ptr(freqs),
+                                           c_int(pairs), c_float(amp), _ptr(positions), c_float(eps), _ptr(slot_map), _ptr(pages),
+                                           c_int(n_tokens), c_int(row_width), c_int(_kind(q_out.dtype)), _stream()))
+
+
 def latent_rope_norm_store(x: torch.Tensor, q_gain, q_rank: int, cq_out, gain: torch.Tensor, rot: int, freqs, positions,
-                           eps: float, slot_map, pages, n_tokens: int) -> None:
+                           eps: float, slot_map, pages, n_tokens: int, amp: float = 1.0) -> None:
     """x float32 [T, q_rank + rank + rot]: cq_out[t] = rms(x[:q_rank]) * q_gain (if q_rank), and the token's cache row
     pages[slot_map[t]] = [the rot last numbers with pairs (2i, 2i+1), i < len(freqs), turned by position * freqs[i] |
     rms(the rank numbers between) * gain | zeros]; pages None: no row is written."""
@@ -690,11 +849,11 @@ def latent_rope_norm_store(x: torch.Tensor, q_gain, q_rank: int, cq_out, gain: t
     _check(load().llmk_latent_rope_norm_store(_ptr(x), c_longlong(x.stride(0)), _ptr(q_gain), c_int(q_rank), _ptr(cq_out),
                                               c_longlong(cq_out.stride(0) if cq_out is not None else 0), _ptr(gain), c_int(rank),
                                               c_int(rot), _ptr(freqs), c_int(pairs), _ptr(positions), c_float(eps), _ptr(slot_map),
-                                              _ptr(pages), c_int(n_tokens), c_int(width), c_int(_kind(kind)), _stream()))
+                                              _ptr(pages), c_int(n_tokens), c_int(width), c_int(_kind(kind)), _stream(), c_float(amp)))
 
 
 def norm_rope_kv_write(qkv, q_gain, k_gain, eps: float, freqs, halves: bool, positions: torch.Tensor, slot_map, k_pages, v_pages,
-                       n_tokens: int, n_heads: int, n_kv: int, dim: int, vdim: int, q_out=None) -> torch.Tensor:
+                       n_tokens: int, n_heads: int, n_kv: int, dim: int, vdim: int, q_out=None, amp: float = 1.0) -> torch.Tensor:
     """As rope_pairs_kv_write, with the RMS norm of the token's whole q projection (weights q_gain, float32
     [n_heads * dim]) and whole k projection (k_gain [n_kv * dim]) first, either None for none, and the choice of pairs:
     halves turns channel i against channel i + len(freqs), else 2i against 2i + 1.  Returns the tensor that holds q."""
@@ -724,7 +883,7 @@ def norm_rope_kv_write(qkv, q_gain, k_gain, eps: float, freqs, halves: bool, pos
                                           _ptr(q_gain), _ptr(k_gain), c_float(eps), _ptr(freqs), c_int(pairs), c_int(int(halves)),
                                           _ptr(positions), _ptr(slot_map), _ptr(k_pages), _ptr(v_pages), c_int(n_tokens),
                                           c_int(n_heads), c_int(n_kv), c_int(dim), c_int(vdim), c_int(page), c_int(_kind(qkv.dtype)),
-                                          _stream()))
+                                          _stream(), c_float(amp)))
     return q_out
 
 
@@ -744,7 +903,8 @@ def moe_max_tiles(n_pairs: int, experts: int, tile: int = 0) -> int:
 
 
 def moe_route(h: torch.Tensor, w: torch.Tensor, bias, logits: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-              n_tokens: int, top: int, over_all: bool = False, sigmoid_groups=None) -> None:
+              n_tokens: int, top: int, over_all: bool = False, groups=None, softmax: bool = False, group_max: bool = False,
+              renorm_eps: float = -1.0) -> None:
     """Router (over_all: the weights are the chosen experts' shares of the softmax over all experts, not
     renormalised): logits = h @ w.T with float32 accumulation (the tensor-core product in bfloat16 where it takes the
     shape, the CUDA-core product otherwise) into `logits` (float32 [>= n_tokens, experts]); plus bias, the `top`
@@ -761,11 +921,14 @@ def moe_route(h: torch.Tensor, w: torch.Tensor, bias, logits: torch.Tensor, ids:
         gemm_simt(h, w, logits, n_tokens)
         z = logits
     d, parts, splits, stride = _split_args(z)
-    if sigmoid_groups is not None:
-        # (groups, keep): sigmoid scores, `bias` is the correction that enters the choice only; see routed.cu
-        groups, keep = sigmoid_groups
-        _check(load().llmk_moe_topk_sigmoid(d, parts, splits, stride, _ptr(bias), _ptr(ids), _ptr(weights), c_int(n_tokens),
-                                            c_int(experts), c_int(top), c_int(groups), c_int(keep), _stream()))
+    if groups is not None:
+        # (groups, keep): sigmoid scores, or a softmax over all experts; `bias` is the correction that enters the choice only; a
+        # group counts by its two largest choice scores, or (group_max) by its largest; renorm_eps >= 0: the chosen scores are
+        # divided by their sum + renorm_eps.  See routed.cu
+        count, keep = groups
+        _check(load().llmk_moe_topk_grouped(d, parts, splits, stride, _ptr(bias), _ptr(ids), _ptr(weights), c_int(n_tokens),
+                                            c_int(experts), c_int(top), c_int(count), c_int(keep), c_int(int(softmax)),
+                                            c_int(int(group_max)), c_float(renorm_eps), _stream()))
         return
     _check(load().llmk_moe_topk(d, parts, splits, stride, _ptr(bias), _ptr(ids), _ptr(weights), c_int(n_tokens),
                                 c_int(experts), c_int(top), c_int(int(over_all)), _stream()))

@@ -123,7 +123,7 @@ LLMK_API int llmk_rope_kv_write(const void* qkv, const float* partials, int spli
 // The other common layout of RoPE: channels 2i and 2i+1 of a head form a pair (not i and i + HS/2),
 // only the first 2 * rot_pairs channels of a head turn, and the angle is position * freqs[i], one
 // float32 product, with freqs given by the caller (so any scaling of the frequencies is the caller's
-// business and no table bounds the position).  Keys and values may differ in size: a row of the
+// business and no table bounds the position); amp multiplies cos and sin.  Keys and values may differ in size: a row of the
 // source holds n_heads * dim query channels, n_kv * dim key channels, n_kv * vdim value channels.
 namespace {
 
@@ -132,7 +132,7 @@ __global__ void __launch_bounds__(128)
 rope_pairs_kv_write_kernel(MaybePartial<T> src, long long src_stride, T* __restrict__ q_out, long long q_out_stride,
                            const float* __restrict__ freqs, int rot_pairs, const int* __restrict__ positions,
                            const int* __restrict__ slot_map, T* __restrict__ k_pages, T* __restrict__ v_pages,
-                           int n_heads, int n_kv, int dim, int vdim, int page_size) {
+                           int n_heads, int n_kv, int dim, int vdim, int page_size, float amp) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -155,6 +155,7 @@ rope_pairs_kv_write_kernel(MaybePartial<T> src, long long src_stride, T* __restr
     if (i < rot_pairs && d1 < dim) {
       float s, c;
       sincosf(pos * freqs[i], &s, &c);
+      s *= amp; c *= amp;
       const float ra = a * c - b * s, rb = b * c + a * s;
       a = ra;
       b = rb;
@@ -184,7 +185,7 @@ norm_rope_kv_write_kernel(MaybePartial<T> src, long long src_stride, T* __restri
                           const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
                           const float* __restrict__ freqs, int rot_pairs, int halves, const int* __restrict__ positions,
                           const int* __restrict__ slot_map, T* __restrict__ k_pages, T* __restrict__ v_pages,
-                          int n_heads, int n_kv, int dim, int vdim, int page_size) {
+                          int n_heads, int n_kv, int dim, int vdim, int page_size, float amp) {
   extern __shared__ float row_s[];            // [(n_heads + n_kv) * dim]
   __shared__ float red[32];
   pdl_launch_dependents();
@@ -227,6 +228,7 @@ norm_rope_kv_write_kernel(MaybePartial<T> src, long long src_stride, T* __restri
       const float b = row_s[c_base + d1] * r * (gain ? gain[g_base + d1] : 1.f);
       float sn, cs;
       sincosf(pos * freqs[i], &sn, &cs);
+      sn *= amp; cs *= amp;
       dst[d0] = from_f32<T>(a * cs - b * sn);
       dst[d1] = from_f32<T>(b * cs + a * sn);
     } else {
@@ -289,7 +291,7 @@ LLMK_API int llmk_rope_pairs_kv_write(const void* qkv, const float* partials, in
                                       long long src_stride, void* q_out, long long q_out_stride, const float* freqs,
                                       int rot_pairs, const int* positions, const int* slot_map, void* k_pages,
                                       void* v_pages, int n_tokens, int n_heads, int n_kv, int dim, int vdim,
-                                      int page_size, int dtype, cudaStream_t stream) {
+                                      int page_size, int dtype, cudaStream_t stream, float amp) {
   if (n_tokens == 0) return 0;
   LLMK_REQUIRE((qkv != nullptr) != (partials != nullptr), "rope_pairs_kv_write: give qkv or partials");
   LLMK_REQUIRE(rot_pairs >= 0 && 2 * rot_pairs <= dim, "rope_pairs_kv_write: %d pairs do not fit a head of %d", rot_pairs, dim);
@@ -299,7 +301,7 @@ LLMK_API int llmk_rope_pairs_kv_write(const void* qkv, const float* partials, in
     MaybePartial<T> src{(const T*)qkv, partials, splits, split_stride};
     launch_kernel(rope_pairs_kv_write_kernel<T>, dim3(n_tokens), dim3(128), 0, stream, src, src_stride, (T*)q_out,
                   q_out_stride, freqs, rot_pairs, positions, slot_map, (T*)k_pages, (T*)v_pages, n_heads, n_kv, dim,
-                  vdim, page_size);
+                  vdim, page_size, amp);
     LLMK_LAUNCH_CHECK("rope_pairs_kv_write");
   });
 }
@@ -310,7 +312,7 @@ LLMK_API int llmk_norm_rope_kv_write(const void* qkv, const float* partials, int
                                      long long src_stride, void* q_out, long long q_out_stride, const float* q_gain,
                                      const float* k_gain, float eps, const float* freqs, int rot_pairs, int halves,
                                      const int* positions, const int* slot_map, void* k_pages, void* v_pages, int n_tokens,
-                                     int n_heads, int n_kv, int dim, int vdim, int page_size, int dtype, cudaStream_t stream) {
+                                     int n_heads, int n_kv, int dim, int vdim, int page_size, int dtype, cudaStream_t stream, float amp) {
   if (n_tokens == 0) return 0;
   LLMK_REQUIRE((qkv != nullptr) != (partials != nullptr), "norm_rope_kv_write: give qkv or partials");
   LLMK_REQUIRE(rot_pairs >= 0 && 2 * rot_pairs <= dim, "norm_rope_kv_write: %d pairs do not fit a head of %d", rot_pairs, dim);
@@ -324,7 +326,7 @@ LLMK_API int llmk_norm_rope_kv_write(const void* qkv, const float* partials, int
       cudaFuncSetAttribute(norm_rope_kv_write_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_kernel(norm_rope_kv_write_kernel<T>, dim3(n_tokens), dim3(256), smem, stream, src, src_stride, (T*)q_out,
                   q_out_stride, q_gain, k_gain, eps, freqs, rot_pairs, halves, positions, slot_map, (T*)k_pages, (T*)v_pages,
-                  n_heads, n_kv, dim, vdim, page_size);
+                  n_heads, n_kv, dim, vdim, page_size, amp);
     LLMK_LAUNCH_CHECK("norm_rope_kv_write");
   });
 }

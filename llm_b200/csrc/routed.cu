@@ -82,24 +82,47 @@ topk_kernel(MaybePartial<float> z, const float* __restrict__ bias, int* __restri
   }
 }
 
-// Sigmoid router with groups: scores s = sigmoid(z); the choice is made on s + correction, the weights are the chosen
-// experts' s themselves (not renormalised).  The experts form `groups` equal runs of neighbours; a group's score is the sum
-// of its two largest choice scores (of its one, in groups of one), and only experts of the `keep` best groups can be chosen:
-// the others are struck out (minus infinity, since choice scores may be negative).  Ties go to the lower index, for groups
-// and for experts.  One warp per token.
+// Router with groups: scores s = sigmoid(z), or (softmax) the softmax of z over all experts; the choice is made on
+// s + correction, the weights are the chosen experts' s, as they are or (renorm_eps >= 0) divided by their sum + renorm_eps.
+// The experts form `groups` equal runs of neighbours; a group's score is the sum of its two largest choice scores (of its one,
+// in groups of one), or (group_max) its largest; only experts of the `keep` best groups can be chosen: the others are struck
+// out (minus infinity, since choice scores may be negative).  Ties go to the lower index, for groups and for experts.  One
+// warp per token.
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-topk_sigmoid_kernel(MaybePartial<float> z, const float* __restrict__ correction, int* __restrict__ ids,
-                    float* __restrict__ weights, int n_tokens, int experts, int top, int groups, int keep) {
+topk_grouped_kernel(MaybePartial<float> z, const float* __restrict__ correction, int* __restrict__ ids,
+                    float* __restrict__ weights, int n_tokens, int experts, int top, int groups, int keep, int softmax,
+                    int group_max, float renorm_eps) {
   __shared__ float c_s[ROUTE_WARPS][MAX_EXPERTS], s_s[ROUTE_WARPS][MAX_EXPERTS], g_s[ROUTE_WARPS][MAX_EXPERTS];
   pdl_launch_dependents();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * ROUTE_WARPS + warp;
   if (t >= n_tokens) return;
-  for (int e = lane; e < experts; e += 32) {
-    const float sc = 1.f / (1.f + expf(-z.at((size_t)t * experts + e)));
-    s_s[warp][e] = sc;
-    c_s[warp][e] = sc + (correction ? correction[e] : 0.f);
+  if (softmax) {
+    float mx = -INFINITY, sum = 0.f;
+    for (int e = lane; e < experts; e += 32) {
+      const float v = z.at((size_t)t * experts + e);
+      s_s[warp][e] = v;
+      mx = fmaxf(mx, v);
+    }
+    mx = warp_max(mx);
+    for (int e = lane; e < experts; e += 32) {          // a lane reads back what it wrote itself
+      const float p = expf(s_s[warp][e] - mx);
+      s_s[warp][e] = p;
+      sum += p;
+    }
+    const float inv = 1.f / warp_sum(sum);
+    for (int e = lane; e < experts; e += 32) {
+      const float sc = s_s[warp][e] * inv;
+      s_s[warp][e] = sc;
+      c_s[warp][e] = sc + (correction ? correction[e] : 0.f);
+    }
+  } else {
+    for (int e = lane; e < experts; e += 32) {
+      const float sc = 1.f / (1.f + expf(-z.at((size_t)t * experts + e)));
+      s_s[warp][e] = sc;
+      c_s[warp][e] = sc + (correction ? correction[e] : 0.f);
+    }
   }
   __syncwarp();
   if (keep < groups) {
@@ -110,7 +133,7 @@ topk_sigmoid_kernel(MaybePartial<float> z, const float* __restrict__ correction,
         const float v = c_s[warp][g * per + i];
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
-      g_s[warp][g] = per > 1 ? a + b : a;
+      g_s[warp][g] = per > 1 && !group_max ? a + b : a;
     }
     __syncwarp();
     // strike out every group but the `keep` best: keep rounds of arg-max mark a group with +infinity
@@ -134,6 +157,7 @@ topk_sigmoid_kernel(MaybePartial<float> z, const float* __restrict__ correction,
       if (g_s[warp][e / per] != INFINITY) c_s[warp][e] = -INFINITY;
     __syncwarp();
   }
+  float sum = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY;
     int arg = 0x7fffffff;
@@ -151,9 +175,16 @@ topk_sigmoid_kernel(MaybePartial<float> z, const float* __restrict__ correction,
       const bool found = arg < experts;
       ids[(size_t)t * top + j] = found ? arg : -1;              // nothing left to choose: the pair is dropped
       weights[(size_t)t * top + j] = found ? s_s[warp][arg] : 0.f;
-      if (found) c_s[warp][arg] = -INFINITY;
+      if (found) {
+        sum += s_s[warp][arg];
+        c_s[warp][arg] = -INFINITY;
+      }
     }
     __syncwarp();
+  }
+  if (renorm_eps >= 0.f && lane == 0) {
+    const float inv = 1.f / (sum + renorm_eps);
+    for (int j = 0; j < top; ++j) weights[(size_t)t * top + j] *= inv;
   }
 }
 
@@ -359,21 +390,22 @@ LLMK_API int llmk_moe_topk(const float* logits, const float* partials, int split
   LLMK_LAUNCH_CHECK("moe_topk");
 }
 
-// The sigmoid router with groups (see topk_sigmoid_kernel): correction float32 [experts] or null; groups divides experts;
-// 1 <= keep <= groups.
-LLMK_API int llmk_moe_topk_sigmoid(const float* logits, const float* partials, int splits, long long split_stride,
+// The router with groups (see topk_grouped_kernel): correction float32 [experts] or null; groups divides experts;
+// 1 <= keep <= groups; softmax 0: sigmoid scores; group_max 0: a group's score is the sum of its two largest; renorm_eps < 0:
+// the weights are the chosen scores as they are.
+LLMK_API int llmk_moe_topk_grouped(const float* logits, const float* partials, int splits, long long split_stride,
                                    const float* correction, int* ids, float* weights, int n_tokens, int experts, int top,
-                                   int groups, int keep, cudaStream_t stream) {
+                                   int groups, int keep, int softmax, int group_max, float renorm_eps, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
-  LLMK_REQUIRE((logits != nullptr) != (partials != nullptr), "moe_topk_sigmoid: give logits or partials");
-  LLMK_REQUIRE(experts > 0 && experts <= MAX_EXPERTS, "moe_topk_sigmoid: %d experts (1 to %d)", experts, MAX_EXPERTS);
-  LLMK_REQUIRE(top > 0 && top <= experts, "moe_topk_sigmoid: top %d of %d experts", top, experts);
+  LLMK_REQUIRE((logits != nullptr) != (partials != nullptr), "moe_topk_grouped: give logits or partials");
+  LLMK_REQUIRE(experts > 0 && experts <= MAX_EXPERTS, "moe_topk_grouped: %d experts (1 to %d)", experts, MAX_EXPERTS);
+  LLMK_REQUIRE(top > 0 && top <= experts, "moe_topk_grouped: top %d of %d experts", top, experts);
   LLMK_REQUIRE(groups > 0 && experts % groups == 0 && keep > 0 && keep <= groups,
-               "moe_topk_sigmoid: %d experts in %d groups of which %d are kept", experts, groups, keep);
+               "moe_topk_grouped: %d experts in %d groups of which %d are kept", experts, groups, keep);
   MaybePartial<float> z{logits, partials, splits, split_stride};
-  launch_kernel(topk_sigmoid_kernel, dim3((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), 0, stream, z,
-                correction, ids, weights, n_tokens, experts, top, groups, keep);
-  LLMK_LAUNCH_CHECK("moe_topk_sigmoid");
+  launch_kernel(topk_grouped_kernel, dim3((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), 0, stream, z,
+                correction, ids, weights, n_tokens, experts, top, groups, keep, softmax, group_max, renorm_eps);
+  LLMK_LAUNCH_CHECK("moe_topk_grouped");
 }
 
 // ids [n_pairs] -> meta[0] (tiles in use), tile_expert [max_tiles], slot_src [max_tiles * 64] (the pair of

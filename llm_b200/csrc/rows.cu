@@ -128,6 +128,174 @@ LLMK_API int llmk_add_rmsnorm(float* resid, const void* delta, const float* part
   });
 }
 
+// ---- the norm behind a residual sum -------------------------------------------
+// resid = rms(alpha * resid + delta) * gamma, and out (if given) the same rows in the element kind: a block that norms the sum
+// itself keeps the normed rows as its residual stream, and its sublayers read them as they are.  delta is a tensor, the
+// partial results of a split-K product, or the weighted rows of a routed feed-forward, sum_j weights[t, j] y[slot(t, j)]
+// (float32, in the order of j), which then need no kernel and no buffer of their own.
+struct WeightedRows { const float* y; const int* pair_slot; const float* weights; int top; };
+
+// NV > 0: rows of up to NV * 2048 elements on the 8-grid stay in registers; 0: any rows, in shared memory.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+sum_rmsnorm_kernel(float* __restrict__ resid, float alpha, MaybePartial<T> delta, WeightedRows rows, const float* __restrict__ gamma,
+                   T* __restrict__ out, int hidden, float eps) {
+  extern __shared__ float row_s[];
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t base = (size_t)blockIdx.x * hidden;
+  const int* slots = rows.pair_slot + (size_t)blockIdx.x * rows.top;
+  const float* wts = rows.weights + (size_t)blockIdx.x * rows.top;
+  float ss = 0.f;
+  if constexpr (NV > 0) {
+    float v[NV][8];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 256 + threadIdx.x) * 8;
+      if (c >= hidden) continue;
+      Vec8<float>::load(resid + base + c, v[i]);
+      float d[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (delta.present()) delta.at8(base + c, d);
+      if (rows.y) {
+#pragma unroll 4
+        for (int j = 0; j < rows.top; ++j) {
+          const int slot = slots[j];
+          if (slot < 0) continue;
+          float y[8];
+          Vec8<float>::load(rows.y + (size_t)slot * hidden + c, y);
+          const float w = wts[j];
+#pragma unroll
+          for (int k = 0; k < 8; ++k) d[k] = fmaf(w, y[k], d[k]);
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < 8; ++k) { v[i][k] = fmaf(alpha, v[i][k], d[k]); ss = fmaf(v[i][k], v[i][k], ss); }
+    }
+    const float rstd = 1.f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 256 + threadIdx.x) * 8;
+      if (c >= hidden) continue;
+      float g[8];
+      Vec8<float>::load(gamma + c, g);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v[i][k] *= rstd * g[k];
+      Vec8<float>::store(resid + base + c, v[i]);
+      if (out) Vec8<T>::store(out + base + c, v[i]);
+    }
+    return;
+  } else {
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+      float d = delta.present() ? delta.at(base + c) : 0.f;
+      if (rows.y)
+        for (int j = 0; j < rows.top; ++j)
+          if (slots[j] >= 0) d = fmaf(wts[j], rows.y[(size_t)slots[j] * hidden + c], d);
+      const float v = fmaf(alpha, resid[base + c], d);
+      row_s[c] = v;
+      ss = fmaf(v, v, ss);
+    }
+    const float rstd = 1.f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+      const float v = row_s[c] * rstd * gamma[c];
+      resid[base + c] = v;
+      if (out) out[base + c] = from_f32<T>(v);
+    }
+  }
+}
+
+// delta / partials as in llmk_add_rmsnorm; y float32 [slots, hidden] with pair_slot int32 and weights float32 [rows, top], or
+// null; gamma float32 [hidden]; out [rows, hidden] of the element kind or null.
+LLMK_API int llmk_sum_rmsnorm(float* resid, float alpha, const void* delta, const float* partials, int splits, long long split_stride,
+                              const float* y, const int* pair_slot, const float* weights, int top, const float* gamma, void* out,
+                              int n_rows, int hidden, float eps, int dtype, cudaStream_t stream) {
+  if (n_rows == 0) return 0;
+  LLMK_REQUIRE(!(delta && partials), "sum_rmsnorm: give delta or partials, not both");
+  LLMK_REQUIRE(y == nullptr || (pair_slot && weights && top > 0), "sum_rmsnorm: weighted rows lack their slots or weights");
+  const size_t smem = (size_t)hidden * sizeof(float);
+  LLMK_REQUIRE(smem <= 200 * 1024, "sum_rmsnorm: rows of %d elements exceed the shared memory", hidden);
+  return dispatch_dtype(dtype, [&](auto* tag) {
+    using T = LLMK_ELEM(tag);
+    MaybePartial<T> d{(const T*)delta, partials, splits, split_stride};
+    const WeightedRows w{y, pair_slot, weights, top};
+    const bool vec = hidden % 8 == 0 && hidden <= 8192 && d.vector_ok() && (uintptr_t)resid % 16 == 0 && (uintptr_t)gamma % 16 == 0 &&
+                     (uintptr_t)out % 16 == 0 && (uintptr_t)y % 16 == 0;
+    auto go = [&](auto kern, size_t bytes) {
+      if (bytes > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+      launch_kernel(kern, dim3(n_rows), dim3(256), bytes, stream, resid, alpha, d, w, gamma, (T*)out, hidden, eps);
+    };
+    if (vec && hidden <= 2048) go(sum_rmsnorm_kernel<T, 1>, 0);
+    else if (vec && hidden <= 4096) go(sum_rmsnorm_kernel<T, 2>, 0);
+    else if (vec) go(sum_rmsnorm_kernel<T, 4>, 0);
+    else go(sum_rmsnorm_kernel<T, 0>, smem);
+    LLMK_LAUNCH_CHECK("sum_rmsnorm");
+  });
+}
+
+// ---- RMS norm over a whole row, gated ------------------------------------------
+// out[t, :] = x[t, :] / sqrt(mean(x[t, :]^2) + eps) * w * sigmoid(gate[t, :]): all heads of a linear-attention mixer normed
+// together.  x float32; gate columns of a projection, a tensor or split-K partial results.  One CTA per row.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+row_rmsnorm_sigmoid_kernel(T* __restrict__ out, const float* __restrict__ x, const float* __restrict__ w, MaybePartial<T> gate,
+                           long long gate_stride, long long gate_col, int n, float eps) {
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t base = (size_t)blockIdx.x * n, g0 = (size_t)blockIdx.x * gate_stride + gate_col;
+  float ss = 0.f;
+  if constexpr (NV > 0) {
+    float v[NV][8];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 256 + threadIdx.x) * 8;
+      if (c >= n) continue;
+      Vec8<float>::load(x + base + c, v[i]);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) ss = fmaf(v[i][k], v[i][k], ss);
+    }
+    const float rstd = 1.f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 256 + threadIdx.x) * 8;
+      if (c >= n) continue;
+      float g[8], z[8];
+      Vec8<float>::load(w + c, g);
+      gate.at8(g0 + c, z);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v[i][k] *= rstd * g[k] / (1.f + expf(-z[k]));
+      Vec8<T>::store(out + base + c, v[i]);
+    }
+  } else {
+    for (int c = threadIdx.x; c < n; c += blockDim.x) ss = fmaf(x[base + c], x[base + c], ss);
+    const float rstd = 1.f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+    for (int c = threadIdx.x; c < n; c += blockDim.x)
+      out[base + c] = from_f32<T>(x[base + c] * rstd * w[c] / (1.f + expf(-gate.at(g0 + c))));
+  }
+}
+
+// gate row t starts at element t * gate_stride + gate_col of the tensor, or of every split of the partial results.
+LLMK_API int llmk_row_rmsnorm_sigmoid(void* out, const float* x, const float* w, const void* gate, const float* partials, int splits,
+                                      long long split_stride, long long gate_stride, long long gate_col, int n_rows, int n, float eps,
+                                      int dtype, cudaStream_t stream) {
+  if (n_rows == 0) return 0;
+  LLMK_REQUIRE((gate != nullptr) != (partials != nullptr), "row_rmsnorm_sigmoid: give gate or partials");
+  return dispatch_dtype(dtype, [&](auto* tag) {
+    using T = LLMK_ELEM(tag);
+    MaybePartial<T> g{(const T*)gate, partials, splits, split_stride};
+    const bool vec = n % 8 == 0 && n <= 8192 && g.vector_ok() && gate_stride % 8 == 0 && gate_col % 8 == 0 && (uintptr_t)x % 16 == 0 &&
+                     (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0;
+    auto go = [&](auto kern) {
+      launch_kernel(kern, dim3(n_rows), dim3(256), 0, stream, (T*)out, x, w, g, gate_stride, gate_col, n, eps);
+    };
+    if (vec && n <= 2048) go(row_rmsnorm_sigmoid_kernel<T, 1>);
+    else if (vec && n <= 4096) go(row_rmsnorm_sigmoid_kernel<T, 2>);
+    else if (vec) go(row_rmsnorm_sigmoid_kernel<T, 4>);
+    else go(row_rmsnorm_sigmoid_kernel<T, 0>);
+    LLMK_LAUNCH_CHECK("row_rmsnorm_sigmoid");
+  });
+}
+
 // ---- gather of the rows whose logits are wanted -----------------------------
 // out[r, :] = resid[rows[r], :] (+ delta[rows[r], :]).  The reference runs its LM head
 // on every row (model/modules/Linear.h:25); gathering first leaves only wanted rows.

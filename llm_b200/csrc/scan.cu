@@ -8,6 +8,9 @@
 //   gate form (HGRN2):                     S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T,   o_t = S_t^T silu(q_t)
 //                                          f_t = l + (1 - l) sigmoid(z_t + b)   per head and key channel, l a lower bound:
 //                                          what the forget gate lets go is what is written, so there is no key
+//   const form (lightning attention):      S_t = d S_{t-1} + silu(k_t) silu(v_t)^T,     o_t = S_t^T silu(q_t)
+//                                          d one fixed number per head (lightning.cu has the forms for single tokens and for
+//                                          bfloat16 prompts; this one takes any sizes)
 //
 // S [dim, vdim] is float32 and lives in the request's state slot (zero at admission); it is read at the start of an
 // entry's tokens and written back at their end, so prompts, portions and single tokens run the same arithmetic.  Decays,
@@ -30,7 +33,9 @@
 namespace {
 
 constexpr int ROWS = 8, COLS = 4, CHUNK = 8, MAX_GROUPS = 32;
-enum : int { FORM_BONUS = 0, FORM_SCALAR = 1, FORM_GATE = 2 };
+enum : int { FORM_BONUS = 0, FORM_SCALAR = 1, FORM_GATE = 2, FORM_CONST = 3 };
+
+__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
@@ -42,6 +47,7 @@ struct ScanArgs {
   const float* bonus;                            // bonus form: u [heads, dim]; gate form: the lower bound l [heads, dim]
   const void* dt; long long dt_stride;           // scalar form: dt' [T, heads]
   const float *dt_bias, *a_log, *skip;           // scalar form: [heads] each
+  const float* decay;                            // const form: [heads]
   float* state; long long slot_stride;           // slot s at state + s * slot_stride: [heads, dim, vdim]
   const int *state_slots, *cu_tokens;
   int heads, qk_heads, dim, vdim;
@@ -111,6 +117,7 @@ diag_scan_kernel(ScanArgs a) {
   for (int r = 0; r < ROWS; ++r) A[r] = 1.f;
   const float neg_a = FORM == FORM_SCALAR ? -expf(a.a_log[head]) : 0.f;
   const float skip = FORM == FORM_SCALAR ? a.skip[head] : 0.f;
+  const float fixed = FORM == FORM_CONST ? a.decay[head] : 0.f;
   const float dt_b = FORM == FORM_SCALAR ? a.dt_bias[head] : 0.f;
 
   // What a thread brings of a chunk: channel d = tid of every token's q, k (and z), and up to VREGS of its values.  The
@@ -119,7 +126,8 @@ diag_scan_kernel(ScanArgs a) {
   const bool v_regs = CHUNK * VT <= VREGS * nthreads;       // else (fewer than 32 channels) the values are read when staged
   T q_r[CHUNK], k_r[CHUNK], v_r[VREGS], dt_r;
   float z_r[CHUNK];
-  const float zb = (FORM != FORM_SCALAR && tid < dim && a.z_bias) ? a.z_bias[head * dim + tid] : 0.f;
+  constexpr bool HAS_Z = FORM == FORM_BONUS || FORM == FORM_GATE;      // a decay per key channel, from a pre-activation
+  const float zb = (HAS_Z && tid < dim && a.z_bias) ? a.z_bias[head * dim + tid] : 0.f;
   const float low = (FORM == FORM_GATE && tid < dim) ? a.bonus[head * dim + tid] : 0.f;
   auto fetch = [&](int c0) {
     const int n = min(CHUNK, t1 - c0);
@@ -129,7 +137,7 @@ diag_scan_kernel(ScanArgs a) {
         const size_t at = (size_t)(c0 + c) * a.qk_stride + (size_t)qk_head * dim + tid;
         if (!STATE_ONLY) q_r[c] = q[at];
         if (FORM != FORM_GATE) k_r[c] = k[at];
-        if (FORM != FORM_SCALAR) z_r[c] = a.z[(size_t)(c0 + c) * a.z_stride + (size_t)head * dim + tid];
+        if (HAS_Z) z_r[c] = a.z[(size_t)(c0 + c) * a.z_stride + (size_t)head * dim + tid];
       }
     }
     if (v_regs) {
@@ -160,6 +168,9 @@ diag_scan_kernel(ScanArgs a) {
           if (!STATE_ONLY) qv = qv / (1.f + expf(-qv));
           av = low + (1.f - low) / (1.f + expf(-(z_r[c] + zb)));
           kv = 1.f - av;
+        } else if (FORM == FORM_CONST) {
+          if (!STATE_ONLY) qv = silu_f(qv);
+          kv = silu_f(to_f32(k_r[c]));
         } else {
           kv = to_f32(k_r[c]);
           if (FORM == FORM_BONUS)
@@ -170,18 +181,22 @@ diag_scan_kernel(ScanArgs a) {
       }
       if (!STATE_ONLY) q_s[c * dpad + tid] = qv;
       k_s[c * dpad + tid] = kv;
-      if (FORM != FORM_SCALAR) a_s[c * dpad + tid] = av;
+      if (HAS_Z) a_s[c * dpad + tid] = av;
     }
     if (v_regs) {
 #pragma unroll
       for (int i = 0; i < VREGS; ++i) {
         const int idx = tid + i * nthreads;
-        if (idx < n * VT) v_s[idx] = blockIdx.x * VT + idx % VT < vdim ? to_f32(v_r[i]) : 0.f;
+        if (idx < n * VT) {
+          const float x = blockIdx.x * VT + idx % VT < vdim ? to_f32(v_r[i]) : 0.f;
+          v_s[idx] = FORM == FORM_CONST ? silu_f(x) : x;
+        }
       }
     } else {
       for (int idx = tid; idx < n * VT; idx += nthreads) {
         const int c = idx / VT, jj = idx % VT, cc = blockIdx.x * VT + jj;
-        v_s[idx] = cc < vdim ? to_f32(v[(size_t)(c0 + c) * a.v_stride + (size_t)head * vdim + cc]) : 0.f;
+        const float x = cc < vdim ? to_f32(v[(size_t)(c0 + c) * a.v_stride + (size_t)head * vdim + cc]) : 0.f;
+        v_s[idx] = FORM == FORM_CONST ? silu_f(x) : x;
       }
     }
     __syncthreads();
@@ -190,7 +205,7 @@ diag_scan_kernel(ScanArgs a) {
       const float4 v4 = *reinterpret_cast<const float4*>(v_s + c * VT + j * COLS);
       const float vv[COLS] = {v4.x, v4.y, v4.z, v4.w};
       float kc[ROWS], ac[ROWS], qc[ROWS];
-      const float a_tok = FORM == FORM_SCALAR ? expf(neg_a * a_s[c]) : 0.f;
+      const float a_tok = FORM == FORM_SCALAR ? expf(neg_a * a_s[c]) : fixed;
 #pragma unroll
       for (int r = 0; r < ROWS; r += 4) {
         const float4 k4 = *reinterpret_cast<const float4*>(k_s + c * dpad + g * ROWS + r);
@@ -199,7 +214,7 @@ diag_scan_kernel(ScanArgs a) {
           const float4 q4 = *reinterpret_cast<const float4*>(q_s + c * dpad + g * ROWS + r);
           qc[r] = q4.x; qc[r + 1] = q4.y; qc[r + 2] = q4.z; qc[r + 3] = q4.w;
         }
-        if (FORM != FORM_SCALAR) {
+        if (HAS_Z) {
           const float4 a4 = *reinterpret_cast<const float4*>(a_s + c * dpad + g * ROWS + r);
           ac[r] = a4.x; ac[r + 1] = a4.y; ac[r + 2] = a4.z; ac[r + 3] = a4.w;
         } else {
@@ -479,6 +494,23 @@ LLMK_API int llmk_gate_scan(float* out, long long out_stride, const void* q, lon
   a.state_slots = state_slots; a.cu_tokens = cu_tokens; a.heads = a.qk_heads = heads; a.dim = dim; a.vdim = vdim;
   return dispatch_dtype(dtype, [&](auto* tag) {
     return launch_scan<LLMK_ELEM(tag), FORM_GATE>(a, n_entries, n_tokens, seg_len, seg_state, seg_decay, stream);
+  });
+}
+
+// The const form.  q, k [T, heads * dim] and v [T, heads * vdim]: column ranges of one projection result (row stride `stride`),
+// pre-activation (silu is taken here); decay float32 [heads].
+LLMK_API int llmk_const_scan(float* out, long long out_stride, const void* q, const void* k, const void* v, long long stride,
+                             const float* decay, float* state, long long slot_stride, const int* state_slots, const int* cu_tokens,
+                             int n_entries, int heads, int dim, int vdim, int dtype, cudaStream_t stream, int n_tokens, int seg_len,
+                             float* seg_state, float* seg_decay) {
+  if (n_entries == 0) return 0;
+  LLMK_REQUIRE(dim > 0 && dim <= ROWS * MAX_GROUPS && vdim > 0, "const_scan: key size %d (1 to %d)", dim, ROWS * MAX_GROUPS);
+  ScanArgs a = {};
+  a.out = out; a.out_stride = out_stride; a.q = q; a.k = k; a.v = v; a.qk_stride = a.v_stride = stride; a.decay = decay;
+  a.state = state; a.slot_stride = slot_stride; a.state_slots = state_slots; a.cu_tokens = cu_tokens;
+  a.heads = a.qk_heads = heads; a.dim = dim; a.vdim = vdim;
+  return dispatch_dtype(dtype, [&](auto* tag) {
+    return launch_scan<LLMK_ELEM(tag), FORM_CONST>(a, n_entries, n_tokens, seg_len, seg_state, seg_decay, stream);
   });
 }
 

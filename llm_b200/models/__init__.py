@@ -1,4 +1,4 @@
-from . import fopivik, llama, norusun, potipel, tevudra  # noqa: F401  (register Fopivik, LlamaForCausalLM, Norusun, Potipel, Tevudra)
+from . import fopivik, llama, nidorax, norusun, potipel, tevudra  # noqa: F401  (each registers its architecture)
 from .spec import LayerSpec, ModelSpec, PartSpec
 
 __all__ = ["LayerSpec", "ModelSpec", "PartSpec"]

@@ -248,14 +248,15 @@ class PagedAttention(Part):
             qkv = conv
         freqs = self.position.frequencies() if self.position is not None else None
         halves = getattr(self.position, "layout", "pairs") == "halves"
+        amp = getattr(self.position, "amplitude", 1.0)
         q_out = ws.get("q_rot", T, self.q_size, self.dtype) if isinstance(qkv, ops.PartialSum) else None
         if self.qk_norm or halves:
             q = ops.norm_rope_kv_write(qkv, self.q_gain, self.k_gain, self.norm_eps, freqs, halves, ctx.positions,
                                        view.group.slot_map, k_pages, v_pages, T, H, 0 if self.shares_cache else n_kv, D, V,
-                                       q_out=q_out)
+                                       q_out=q_out, amp=amp)
         else:
             q = ops.rope_pairs_kv_write(qkv, freqs, ctx.positions, view.group.slot_map, k_pages, v_pages, T, H,
-                                        0 if self.shares_cache else n_kv, D, V, q_out=q_out)
+                                        0 if self.shares_cache else n_kv, D, V, q_out=q_out, amp=amp)
         attn = ws.get("attn_out", T, H * V, self.dtype)
         ops.paged_attention(attn, q, k_pages, v_pages, view.group, ctx, H, n_kv, D, self.window or 0, self.scale,
                             value_dim=V, softcap=self.softcap, sink=self.sink, keep_first=self.keep_first,

@@ -155,6 +155,18 @@ class ResidualStream:
         # a pending term that is still to be normed and scaled before it joins the residual:
         # (the norm part that does it, multiplier); None: the term is added as it is
         self.pending_post = None
+        # the stream's rows in the compute dtype, while they are those of resid (kept by norms that stand behind the sum)
+        self.rows_cast: Optional[torch.Tensor] = None
+
+    def as_rows(self, ctx, dtype: torch.dtype) -> torch.Tensor:
+        """The stream itself as a sublayer reads it, [rows, H] in the compute dtype (nothing may be pending)."""
+        if dtype == torch.float32:
+            return self.resid[:self.rows]
+        if self.rows_cast is None:
+            from ..csrc import ops
+            self.rows_cast = ctx.workspace.get("stream_rows", self.rows, self.resid.shape[1], dtype)
+            ops.cast_rows(self.rows_cast, self.resid, self.rows)
+        return self.rows_cast
 
     def fold(self, ctx) -> None:
         """Add what is pending, so that resid is the whole stream."""

@@ -93,6 +93,44 @@ class SandwichBlock:
 register_part("block", "sandwich", SandwichBlock)
 
 
+class PostNormBlock:
+    """x <- norm1(alpha x + mixer(x)); x <- norm2(alpha x + ffn(x)): the norms stand behind the sums and every sublayer reads
+    the stream itself.  The norm's part does sum and norm in one pass (norm.close).  A layer without a feed-forward leaves out
+    norm2 and ffn."""
+
+    role = "block"
+    roles = {"mixer": "mixer", "norm1": "norm", "ffn": "ffn", "norm2": "norm"}
+
+    def __init__(self, part_specs, dtype, device, alpha: float = 1.0):
+        self.alpha, self.dtype = float(alpha), dtype
+        optional = ("norm2", "ffn") if part_specs.get("ffn") is None else ()
+        missing = [r for r in self.roles if part_specs.get(r) is None and r not in optional]
+        if missing:
+            raise ValueError(f"postnorm block lacks parts {missing}")
+        self.parts = {r: build_part(self.roles[r], part_specs[r], dtype, device) if part_specs.get(r) is not None else None
+                      for r in self.roles}
+        for r in ("norm1", "norm2"):
+            if self.parts[r] is not None and not hasattr(self.parts[r], "close"):
+                raise ValueError(f"postnorm block: the norm '{part_specs[r].kind}' cannot stand behind a sum (no close)")
+        self.mixer, self.ffn = self.parts["mixer"], self.parts["ffn"]
+        if self.ffn is not None and hasattr(self.ffn, "state_need"):
+            raise ValueError("postnorm block: the feed-forward keeps no state of its own")
+        # a feed-forward that can leave its last weighted sum to the norm does so
+        self.unsummed = {"allow_unsummed": True} if getattr(self.ffn, "leaves_unsummed", False) else {}
+
+    def forward(self, stream: ResidualStream, ctx, view) -> None:
+        p = self.parts
+        if stream.pending is not None:
+            stream.fold(ctx)
+            stream.rows_cast = None
+        p["norm1"].close(stream, self.mixer.forward(stream.as_rows(ctx, self.dtype), ctx, view), self.alpha, ctx)
+        if self.ffn is not None:
+            p["norm2"].close(stream, self.ffn.forward(stream.as_rows(ctx, self.dtype), ctx, **self.unsummed), self.alpha, ctx)
+
+
+register_part("block", "postnorm", PostNormBlock)
+
+
 class StreamBlock:
     """A place in the layer order that holds no layer but one transform of the whole stream (role "stream")."""
 

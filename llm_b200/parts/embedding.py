@@ -39,7 +39,7 @@ class TokenEmbedding(Part):
             ops.hc_embedding(stream.resid, self.table, ctx.token_ids, ctx.n_tokens, self.copies, ctx.status)
         else:
             ops.embedding(stream.resid, self.table, ctx.token_ids, ctx.n_tokens, ctx.status, self.scale)
-        stream.pending = stream.pending_post = None
+        stream.pending = stream.pending_post = stream.rows_cast = None
 
 
 class LMHead(Part):

@@ -20,9 +20,10 @@ tensor names are parameters.
 Options, each a parameter and off by default:
   q_rank    the queries pass a latent of their own: c_q = rms(Wdq h) * gain_q, q = Wuq c_q;
   rot_dim   every query head carries rot_dim more channels and the down-projection rot_dim more rows: one key part
-            shared by all heads (not normed), both turned by the position part (pairs of neighbours); the score is
-            q_plain . k_plain + q_turned . k_turned.  The cached row is then [turned key part | c], the query that meets
+            shared by all heads (not normed), both turned by the position part (pairs of neighbours, or rotate-half; with its
+            factor on cos and sin, if it has one); the score is q_plain . k_plain + q_turned . k_turned.  The cached row is then [turned key part | c], the query that meets
             it [turned query part | Wuk_h^T q_plain], and the value map skips the row's first rot_dim numbers;
+            A layer may read the turned rows that another layer of the same sizes stored, with queries and maps of its own;
   window    a query sees itself and the window - 1 tokens before it (pages behind the window go back to the pool);
   sink      the softmax's denominator holds one more term exp(sink_h), a learned number per head without key or value.
 """
@@ -59,8 +60,9 @@ class LatentAttention(Part):
         self.position = build_part("position", position, dtype, device) if position is not None else None
         # with any of these the mixer runs the path of _forward_rotary (its own layout of the projections)
         self.rotary = bool(self.q_rank or self.rot_dim or self.window or self.sink)
-        if self.rotary and (self.gated or self.shares_cache):
-            raise ValueError("latent attention: a query latent, a turned key part, a window or a sink go without gate and with latents of the layer's own")
+        if self.rotary and (self.gated or (self.shares_cache and (self.q_rank or self.window))):
+            raise ValueError("latent attention: a query latent, a turned key part, a window or a sink go without gate; a query latent "
+                             "and a window with latents of the layer's own")
         if self.rot_dim % 2 or (self.position is not None and not hasattr(self.position, "frequencies")):
             raise ValueError("latent attention: the turned part is even and its position part gives frequencies")
         if self.position is not None and self.position.dims > self.rot_dim:
@@ -88,9 +90,11 @@ class LatentAttention(Part):
         n = lambda k: self.name(self.names[k])
         if self.rotary:
             W, H, C = self.hidden_size, self.num_heads, self.rank
-            p = {n("down"): ParamInfo((C + self.rot_dim, W)), n("down_norm"): ParamInfo((C,), kind="gain", init="ones_normal"),
-                 n("up_k"): ParamInfo((H * self.head_dim, C)), n("up_v"): ParamInfo((H * self.value_dim, C)),
+            p = {n("up_k"): ParamInfo((H * self.head_dim, C)), n("up_v"): ParamInfo((H * self.value_dim, C)),
                  n("out"): ParamInfo((W, H * self.value_dim))}
+            if not self.shares_cache:
+                p[n("down")] = ParamInfo((C + self.rot_dim, W))
+                p[n("down_norm")] = ParamInfo((C,), kind="gain", init="ones_normal")
             if self.q_rank:
                 p[n("q_down")] = ParamInfo((self.q_rank, W))
                 p[n("q_down_norm")] = ParamInfo((self.q_rank,), kind="gain", init="ones_normal")
@@ -133,16 +137,25 @@ class LatentAttention(Part):
 
     def _bind_rotary(self, n):
         H, D, V, C, R, RW = self.num_heads, self.head_dim, self.value_dim, self.rank, self.rot_dim, self.row_width
-        self.gain = n("down_norm").contiguous()
+        # the turned channels in the order the kernels turn them, neighbours paired: a rotate-half layout, which pairs channel i
+        # with i + dims / 2, becomes that by reordering the rows of the projections (of queries and keys alike)
+        turn = torch.arange(R)
+        if self.position is not None and self.position.layout == "halves":
+            half = self.position.dims // 2
+            turn[:2 * half] = torch.stack([torch.arange(half), torch.arange(half) + half], dim=1).flatten()
         # the head's query rows reordered so that the turned part comes first: [turned R | plain D]
-        order = torch.cat([torch.cat([torch.arange(D, D + R), torch.arange(D)]) + h * (D + R) for h in range(H)]).to(self.device)
+        order = torch.cat([torch.cat([D + turn, torch.arange(D)]) + h * (D + R) for h in range(H)]).to(self.device)
+        down = None
+        if not self.shares_cache:
+            self.gain = n("down_norm").contiguous()
+            down = n("down")[torch.cat([torch.arange(C), C + turn]).to(self.device)]
         if self.q_rank:
-            self.w_in = torch.cat([n("q_down"), n("down")], dim=0).contiguous()          # [q_rank + C + R, W]
+            self.w_in = torch.cat([n("q_down"), down], dim=0).contiguous()               # [q_rank + C + R, W]
             self.q_gain = n("q_down_norm").contiguous()
             self.w_uq = n("q_up")[order].contiguous()
-        else:
-            self.w_in = n("down").contiguous()
-            self.w_uq = n("q")[order].contiguous()
+        else:                                                                            # [queries; latent; turned key part]
+            q = n("q")[order]
+            self.w_in = (torch.cat([q, down], dim=0) if down is not None else q).contiguous()
         # a query [turned R | plain D] -> what meets a cached row [turned R | latent C | zeros]: the turned part passes
         # through an identity, the plain part through the key map
         w_map = torch.zeros((H, RW, R + D), dtype=self.dtype, device=self.device)
@@ -167,22 +180,29 @@ class LatentAttention(Part):
         return None
 
     def _forward_rotary(self, x: torch.Tensor, ctx, view) -> torch.Tensor:
-        """One product for the two down-projections (float32 out: both are normed next); one kernel for the two norms, the
-        turning of the key part and the cache row; the query's up-projection; the turning of the queries' leading
-        channels; the per-head map to the cached row's layout; the paged attention with one key/value head (window, sink);
-        the per-head value map; the output projection."""
+        """The projections (float32 out, or split-K partial results: what is normed or turned next is not rounded before); norms,
+        turning and the cache row; the per-head map of the queries to the cached row's layout; the paged attention with one
+        key/value head (window, sink); the per-head value map; the output projection.  Without a query latent one product and
+        one kernel make queries and cache row; with one, the queries follow from it by a product of their own."""
         T, ws = ctx.n_tokens, ctx.workspace
         H, C, R, RW, Q = self.num_heads, self.rank, self.rot_dim, self.row_width, self.q_rank
         pages = view.k_pages
+        own = None if self.shares_cache else pages
         freqs = self.position.frequencies() if self.position is not None else None
-        proj = linear(x, self.w_in, ws.get("latent_down", T, self.w_in.shape[0], torch.float32), T)
-        cq = ws.get("latent_cq", T, Q, self.dtype) if Q else None
-        ops.latent_rope_norm_store(proj, self.q_gain, Q, cq, self.gain, R, freqs, ctx.positions, self.eps,
-                                   view.group.slot_map, pages, T)
-        q = linear(cq if Q else x, self.w_uq, ws.get("latent_in", T, self.q_size, self.dtype), T, allow_partial=FUSE_PARTIALS)
-        if R or isinstance(q, ops.PartialSum):
-            q = ops.rope_pairs_kv_write(q, freqs, ctx.positions, None, None, None, T, H, 0, self.head_dim + R, 0,
-                                        q_out=ws.get("latent_in", T, self.q_size, self.dtype) if isinstance(q, ops.PartialSum) else None)
+        amp = self.position.amplitude if self.position is not None else 1.0
+        q = ws.get("latent_in", T, self.q_size, self.dtype)
+        if Q:
+            proj = linear(x, self.w_in, ws.get("latent_down", T, self.w_in.shape[0], torch.float32), T)
+            cq = ws.get("latent_cq", T, Q, self.dtype)
+            ops.latent_rope_norm_store(proj, self.q_gain, Q, cq, self.gain, R, freqs, ctx.positions, self.eps,
+                                       view.group.slot_map, own, T, amp=amp)
+            qp = linear(cq, self.w_uq, q, T, allow_partial=FUSE_PARTIALS)
+            if R or isinstance(qp, ops.PartialSum):
+                q = ops.rope_pairs_kv_write(qp, freqs, ctx.positions, None, None, None, T, H, 0, self.head_dim + R, 0, q_out=q, amp=amp)
+        else:
+            proj = linear(x, self.w_in, ws.get("latent_proj", T, self.w_in.shape[0], torch.float32), T, allow_partial=FUSE_PARTIALS)
+            ops.latent_q_rope_store(proj, q, H, self.head_dim, self.gain, C, R, freqs, amp, ctx.positions, self.eps,
+                                    view.group.slot_map, own, T)
         q_lat = ws.get("latent_q", T, H * RW, self.dtype)
         ops.gemm_heads(q, self.w_uk_t, q_lat, T, H)
         o_lat = ws.get("latent_o", T, H * RW, self.dtype)

@@ -16,18 +16,32 @@ from .base import ParamInfo, Part, ResidualStream, register_part
 class RMSNorm(Part):
     role = "norm"
 
-    def __init__(self, size: int, eps: float, weight_name: str = "weight", prefix: str = "", dtype=None, device=None):
+    def __init__(self, size: int, eps: float, weight_name: str = "weight", centred: bool = False, prefix: str = "", dtype=None,
+                 device=None):
         super().__init__(prefix, dtype, device)
         self.size = size
         self.eps = float(eps)
         self.weight_name = weight_name        # "": the gain is the tensor named like the part
+        self.centred = bool(centred)          # the stored weight is the gain's distance from one
         self.gain = None
 
     def parameters(self):
-        return {self.name(self.weight_name): ParamInfo((self.size,), kind="gain", init="ones_normal")}
+        return {self.name(self.weight_name): ParamInfo((self.size,), kind="gain", init="normal" if self.centred else "ones_normal")}
 
     def bind(self, tensors):
-        self.gain = tensors[self.name(self.weight_name)]
+        w = tensors[self.name(self.weight_name)]
+        self.gain = (w + 1.0).contiguous() if self.centred else w
+
+    def close(self, stream: ResidualStream, y, alpha: float, ctx) -> None:
+        """The norm behind a residual sum: x <- rms(alpha * x + y) * gain, in float32 on the stream, with a copy of the new
+        rows in the compute dtype for the sublayers that read them (stream.rows_cast).  y: a tensor, a PartialSum or the
+        unsummed rows of a routed feed-forward (ops.WeightedRows)."""
+        out = None
+        if self.dtype != torch.float32:
+            out = ctx.workspace.get("stream_rows", stream.rows, self.size, self.dtype)
+        ops.sum_rmsnorm(stream.resid, alpha, y, self.gain, out, stream.rows, self.eps, self.dtype)
+        stream.pending = stream.pending_post = None
+        stream.rows_cast = out
 
     def forward(self, stream: ResidualStream, ctx, tag: str = "normed") -> torch.Tensor:
         out = ctx.workspace.get(tag, stream.rows, self.size, self.dtype)

@@ -8,6 +8,8 @@ values of the 32-bit angle.
 """
 from __future__ import annotations
 
+import math
+
 import numpy as np
 import torch
 
@@ -56,11 +58,18 @@ class PairRotary(Part):
     and in between blended, (1 - s) f / factor + s f with s = (original / l - low) / (high - low).  The part
     gives the frequencies (float32, evaluated in float64 and rounded once); the angle is one float32 product in
     the kernel that rotates and stores, so no table bounds the position.  layout "halves" pairs channel i with channel
-    i + dims/2 (rotate-half on the first dims channels) with the same frequencies."""
+    i + dims/2 (rotate-half on the first dims channels) with the same frequencies.
+
+    scaling_kind "yarn" (scaling {factor, original, fast, slow}) blends by index instead of wavelength: with
+    at(t) = dims ln(original / (2 pi t)) / (2 ln base), the (fractional) pair that makes t turns within the original length,
+    f_i keeps its value below lo = max(floor(at(fast)), 0), is divided by factor above hi = min(ceil(at(slow)), dims - 1),
+    and runs linearly in i between; cos and sin are multiplied by `amplitude` = 0.1 ln(factor) + 1 (1 otherwise)."""
 
     role = "position"
+    SCALING_KEYS = {"wavelength": ("factor", "low", "high", "original"), "yarn": ("factor", "original", "fast", "slow")}
 
-    def __init__(self, dims: int, base: float, scaling=None, layout: str = "pairs", prefix: str = "", dtype=None, device=None):
+    def __init__(self, dims: int, base: float, scaling=None, layout: str = "pairs", scaling_kind: str = "wavelength", prefix: str = "",
+                 dtype=None, device=None):
         super().__init__(prefix, dtype, device)
         if layout not in ("pairs", "halves"):
             raise ValueError(f"pair rotation: layout '{layout}' is neither 'pairs' nor 'halves'")
@@ -69,19 +78,28 @@ class PairRotary(Part):
             raise ValueError(f"pair rotation: dims {dims} must be even and not negative")
         self.dims, self.base = int(dims), float(base)
         self.scaling = dict(scaling) if scaling else None
+        if scaling_kind not in self.SCALING_KEYS:
+            raise ValueError(f"pair rotation: unknown kind of scaling '{scaling_kind}'; known: {sorted(self.SCALING_KEYS)}")
+        self.yarn = self.scaling is not None and scaling_kind == "yarn"
         if self.scaling:
-            for k in ("factor", "low", "high", "original"):
+            for k in self.SCALING_KEYS[scaling_kind]:
                 if k not in self.scaling:
                     raise ValueError(f"pair rotation: scaling lacks '{k}'")
-            if self.scaling["high"] == self.scaling["low"]:
+            if not self.yarn and self.scaling["high"] == self.scaling["low"]:
                 raise ValueError("pair rotation: scaling.high equals scaling.low")
+        self.amplitude = 0.1 * math.log(float(self.scaling["factor"])) + 1.0 if self.yarn else 1.0
         self._freqs = None
 
     def host_frequencies(self) -> np.ndarray:
         i = np.arange(self.dims // 2, dtype=np.float64)
         f = np.power(np.float64(self.base), -2.0 * i / max(self.dims, 1))
         sc = self.scaling
-        if sc:
+        if self.yarn:
+            at = lambda turns: self.dims * math.log(sc["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
+            lo, hi = max(math.floor(at(sc["fast"])), 0), min(math.ceil(at(sc["slow"])), self.dims - 1)
+            ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+            f = f / sc["factor"] * ramp + f * (1.0 - ramp)
+        elif sc:
             factor, low, high, orig = (float(sc[k]) for k in ("factor", "low", "high", "original"))
             wave = 2.0 * np.pi / f
             s = (orig / wave - low) / (high - low)

@@ -9,7 +9,8 @@ Further forms, all parameters: router "softmax_all", where w_e is expert e's sha
 the chosen weights do not sum to one); router "sigmoid_groups", where the scores are s = sigmoid(z), the choice is made on
 s + correction (a learned vector, `<prefix>.correction`), the experts form `groups` equal runs of neighbours of which only the
 `keep_groups` best (by the sum of their two largest choice scores) can be chosen from, and the weights are the chosen s,
-not renormalised; gated experts, down_e(act(gate_e(h)) * up_e(h)), with act silu or the clamped unit
+not renormalised; "softmax_groups", the same with s = softmax(z) over all experts, a group counted by its largest choice score
+alone, and the chosen s divided by their sum + weight_eps; gated experts, down_e(act(gate_e(h)) * up_e(h)), with act silu or the clamped unit
 g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit) (activation "clamped").
 
 On the device: the router kernel writes each token's choices and weights; the (token, choice)
@@ -44,27 +45,29 @@ class RoutedFFN(Part):
     def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, activation: str = "gelu",
                  router_bias: bool = True, shared_size: int = 0, shared_activation: str = None, gated: bool = False,
                  router: str = "softmax_chosen", groups: int = 1, keep_groups: int = 1, limit: float = 0.0, alpha: float = 1.702,
-                 prefix: str = "", dtype=None, device=None):
+                 weight_eps: float = 1e-20, prefix: str = "", dtype=None, device=None):
         super().__init__(prefix, dtype, device)
         if not (0 < top <= experts <= 256):
             raise ValueError(f"routed feed-forward: top {top} of {experts} experts (1 <= top <= experts <= 256)")
         if activation not in ops.ACTIVATIONS and activation != "clamped":
             raise ValueError(f"routed feed-forward: unknown activation '{activation}'")
         self.hidden_size, self.experts, self.top, self.expert_size = hidden_size, experts, top, expert_size
-        if router not in ("softmax_chosen", "softmax_all", "sigmoid_groups"):
+        if router not in ("softmax_chosen", "softmax_all", "sigmoid_groups", "softmax_groups"):
             raise ValueError(f"routed feed-forward: unknown router '{router}'")
         if gated and activation not in ("silu", "clamped") or (activation == "clamped" and not gated):
             raise ValueError("routed feed-forward: gated experts take the silu activation or the clamped unit, and only they the latter")
         self.clamped, self.limit, self.alpha = activation == "clamped", float(limit), float(alpha)
         if self.clamped and not self.limit > 0:
             raise ValueError("routed feed-forward: the clamped unit needs a positive limit")
-        self.sigmoid_groups = None
-        if router == "sigmoid_groups":
+        self.groups, self.route_options = None, {}
+        if router in ("sigmoid_groups", "softmax_groups"):
             if groups <= 0 or experts % groups or not (0 < keep_groups <= groups):
                 raise ValueError(f"routed feed-forward: {experts} experts in {groups} groups of which {keep_groups} are kept")
             if top > keep_groups * (experts // groups):
                 raise ValueError(f"routed feed-forward: top {top} exceeds the {keep_groups * (experts // groups)} experts of the kept groups")
-            self.sigmoid_groups = (int(groups), int(keep_groups))
+            self.groups = (int(groups), int(keep_groups))
+            if router == "softmax_groups":
+                self.route_options = {"softmax": True, "group_max": True, "renorm_eps": float(weight_eps)}
             router_bias = False
         self.activation, self.router_bias = activation, bool(router_bias)
         self.gated, self.over_all = bool(gated), router == "softmax_all"
@@ -79,7 +82,7 @@ class RoutedFFN(Part):
         p = {self.name("router"): ParamInfo((self.experts, self.hidden_size))}
         if self.router_bias:
             p[self.name("router.b")] = ParamInfo((self.experts,), kind="gain", init="normal")
-        if self.sigmoid_groups:
+        if self.groups:
             p[self.name("correction")] = ParamInfo((self.experts,), kind="gain", init="normal")
         for e in range(self.experts):
             if self.gated:
@@ -91,7 +94,7 @@ class RoutedFFN(Part):
     def bind(self, tensors):
         self.w_router = tensors[self.name("router")].contiguous()
         self.b_router = tensors[self.name("router.b")].contiguous() if self.router_bias else None
-        if self.sigmoid_groups:
+        if self.groups:
             self.b_router = tensors[self.name("correction")].contiguous()      # enters the choice, not the weights
         if self.gated:      # per expert [gate; up] stacked: one grouped product, then silu(gate) * up over the slots
             self.w_up = torch.stack([torch.cat([tensors[self.name(f"e{e}.gate")], tensors[self.name(f"e{e}.up")]], dim=0)
@@ -107,7 +110,13 @@ class RoutedFFN(Part):
         else:
             ops.silu_mul(act, gate_up, rows)
 
-    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+    @property
+    def leaves_unsummed(self) -> bool:
+        """Whether the weighted sum of a token's experts can be left to the kernel that reads it (no shared expert beside it)."""
+        return self.shared is None
+
+    def forward(self, x: torch.Tensor, ctx, allow_unsummed: bool = False):
+        """With allow_unsummed (and no shared expert) the result is an ops.WeightedRows, else a tensor."""
         T, ws, top, E = ctx.n_tokens, ctx.workspace, self.top, self.experts
         # bfloat16 runs the experts on the tensor cores (tiles of 128 slots, rows gathered into slot order
         # first); float32, and shapes the tensor-core kernel refuses, on the CUDA cores (tiles of 64)
@@ -125,7 +134,7 @@ class RoutedFFN(Part):
 
         logits = ws.get("moe_logits", T, E, f32)
         ops.moe_route(x, self.w_router, self.b_router, logits, ids, wts, T, top, over_all=self.over_all,
-                      sigmoid_groups=self.sigmoid_groups)
+                      groups=self.groups, **self.route_options)
         ops.moe_group(ids, pairs, E, meta, tile_expert, slot_src, pair_slot, max_tiles, tile)
         if tensor:
             # gated experts: a tile multiplies by its expert's gate rows and up rows and the epilogue makes silu(gate) * up
@@ -148,6 +157,8 @@ class RoutedFFN(Part):
             ops.moe_gemm_tc(act, tile_expert, meta, self.w_down, y, max_tiles)
         else:
             ops.moe_gemm(act, 0, slot_src, tile_expert, meta, self.w_down, y, max_tiles)
+        if allow_unsummed and self.leaves_unsummed:
+            return ops.WeightedRows(y, pair_slot, wts, top, T)
         shared = self.shared.forward(x, ctx, tag="ffn_shared") if self.shared is not None else None
         out = ws.get("ffn_out", T, self.hidden_size, self.dtype)
         ops.moe_combine(out, y, pair_slot, wts, shared, T, top)

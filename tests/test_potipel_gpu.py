@@ -123,7 +123,7 @@ def test_router_chooses_among_the_best_groups(E, top, count, keep):
     logits = torch.empty(T, E, device="cuda")
     ids = torch.empty(T * top, dtype=torch.int32, device="cuda")
     wts = torch.empty(T * top, device="cuda")
-    ops.moe_route(dev(h), dev(p["router"]), dev(p["correction"]), logits, ids, wts, T, top, sigmoid_groups=(count, keep))
+    ops.moe_route(dev(h), dev(p["router"]), dev(p["correction"]), logits, ids, wts, T, top, groups=(count, keep))
     ids, wts = ids.view(T, top).cpu().long(), wts.view(T, top).cpu()
     clear = margin > 1e-4
     assert int(clear.sum()) > T // 2
