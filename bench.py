@@ -481,9 +481,48 @@ POTIPEL_SIZES = {
 }
 
 
+def nidorax_config(width, pattern, repeats, heads, dim, kv_rank, rot_dim, lin_heads, lin_dim, lin_vdim, experts, top, expert_ff,
+                   vocab=32000):
+    """Layers follow `pattern` (n: lightning attention, l: latent attention with latents of its own, b: one that reads the latents
+    of the layer that kept some last) `repeats` times, each with squared-relu experts behind a grouped softmax router."""
+    mlp = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}}}
+    lin = {"heads": lin_heads, "dim": lin_dim, "vdim": lin_vdim, "decay": [1.0 - 2.0 ** -(1 + 8 * h / lin_heads) for h in range(lin_heads)]}
+    lat = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": dim, "kv_rank": kv_rank, "scale": (dim + rot_dim) ** -0.5,
+           "rot": {"dims": rot_dim, "base": 5e5, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    ls, last = [], 0
+    for i, c in enumerate(pattern * repeats):
+        if c == "l":
+            last = i
+        mixer = lin if c == "n" else lat if c == "l" else dict(lat, kv_from=last)
+        ls.append({"type": "lightning" if c == "n" else "latent_attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Nidorax", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "postln_alpha": 2.0, "layers": ls,
+            "max_position": 4096}
+
+
+def tevudra_routed_config(*sizes, **kw):
+    """Tevudra with a routed feed-forward (no shared expert) in every layer."""
+    cfg = tevudra_config(*sizes, **kw)
+    moe = {k: v for k, v in cfg["layers"][1]["mlp"].items() if k != "shared"}
+    for lay in cfg["layers"]:
+        lay["mlp"] = moe
+    return cfg
+
+
+# name -> (Nidorax config, Tevudra config of the same width, depth, heads, cached row and experts: the design here that also keeps
+# and shares latents and runs ungated experts; its like of the recurrence is Fopivik's gated linear attention, --mode fopivik)
+NIDORAX_SIZES = {
+    "2048": (nidorax_config(2048, "nlnb", 2, 16, 128, 96, 32, 16, 128, 128, 16, 4, 1408),
+             tevudra_routed_config(2048, 8, 16, 128, 128, 128, 0, 16, 4, 1408, 0)),
+    "4096": (nidorax_config(4096, "nlnb", 1, 32, 128, 96, 32, 32, 128, 128, 32, 4, 2752),
+             tevudra_routed_config(4096, 4, 32, 128, 128, 128, 0, 32, 4, 2752, 0)),
+    "1024-row64": (nidorax_config(1024, "nlnb", 2, 16, 64, 48, 16, 16, 64, 64, 8, 2, 1408),
+                   tevudra_routed_config(1024, 8, 16, 64, 64, 64, 0, 8, 2, 1408, 0)),
+}
+
+
 def design_comparison(args, peaks, design: str = "tevudra") -> int:
-    """Prefill and decode throughput of a design (Tevudra, Fopivik or Norusun) beside Llama at equal layer sizes, or of Potipel
-    beside Fopivik (random weights, bfloat16), with the device time of every kernel of one prompt step and one decode step.
+    """Prefill and decode throughput of a design (Tevudra, Fopivik or Norusun) beside Llama at equal layer sizes, of Potipel
+    beside Fopivik, or of Nidorax beside Tevudra (random weights, bfloat16), with the device time of every kernel of one prompt step and one decode step.
     One JSON line per size."""
     import collections
 
@@ -572,8 +611,8 @@ def design_comparison(args, peaks, design: str = "tevudra") -> int:
         torch.cuda.empty_cache()
         return out
 
-    table = {"fopivik": FOPIVIK_SIZES, "norusun": NORUSUN_SIZES, "potipel": POTIPEL_SIZES}.get(design, DESIGN_SIZES)
-    beside = "fopivik" if design == "potipel" else "llama"
+    table = {"fopivik": FOPIVIK_SIZES, "norusun": NORUSUN_SIZES, "potipel": POTIPEL_SIZES, "nidorax": NIDORAX_SIZES}.get(design, DESIGN_SIZES)
+    beside = {"potipel": "fopivik", "nidorax": "tevudra"}.get(design, "llama")
     sizes = [s for s in table if not args.sizes or s in args.sizes.split(",")]
     for name in sizes:
         tev, lla = table[name]
@@ -599,15 +638,15 @@ def main() -> int:
                     help="skip the runs at the Llama-2-7B and Llama-3-8B shapes, the many-request load and the 32-bit check")
     ap.add_argument("--mode", default="all",
                     choices=["all", "decode", "prefill", "timeline", "timeline_prefill", "decode_attention", "tevudra", "fopivik", "norusun",
-                             "potipel"],
+                             "potipel", "nidorax"],
                     help="decode / prefill: only that measurement, for small profiling runs (not the benchmark line); "
                          "timeline: the kernels of one decode layer with their start and end inside the step's CUDA graph; "
                          "decode_attention: the decode attention kernel alone over batches and context lengths "
                          "(--batch with --ctx: that one case); "
                          "tevudra, fopivik, norusun: that design beside Llama at equal layer sizes, prompt and decode, with every kernel's time; "
-                         "potipel: the same beside Fopivik")
+                         "potipel: the same beside Fopivik; nidorax: beside Tevudra")
     ap.add_argument("--latent", action="store_true", help="decode_attention: the key pages are the value pages too")
-    ap.add_argument("--sizes", default="", help="tevudra, fopivik, norusun: which of the sizes to run (comma-separated; default all)")
+    ap.add_argument("--sizes", default="", help="tevudra, fopivik, norusun, potipel, nidorax: which of the sizes to run (comma-separated; default all)")
     ap.add_argument("--ctx", type=int, default=0, help="decode_attention: the context length of the one case to run")
     ap.add_argument("--prompt-tokens", type=int, default=PREFILL_TOKENS, help="timeline_prefill: tokens of the prompt step")
     ap.add_argument("--heads", default="32,4,64", help="decode_attention: query heads, kv heads, head size")
@@ -630,7 +669,7 @@ def main() -> int:
     peaks = load_peaks()
     if args.mode == "decode_attention":
         return decode_attention_sweep(args, peaks, torch, ops)
-    if args.mode in ("tevudra", "fopivik", "norusun", "potipel"):
+    if args.mode in ("tevudra", "fopivik", "norusun", "potipel", "nidorax"):
         return design_comparison(args, peaks, args.mode)
     cfg = dict(MODEL, num_hidden_layers=args.layers)
     if args.mode != "all":

@@ -60,10 +60,12 @@ def yarn(dims, base, scaling=None):
     return out, 0.1 * math.log(scaling["factor"]) + 1.0
 
 
-def rotate_halves(x, positions, freqs, amp):
-    """x [..., T, dims]: channel i turns against channel i + dims / 2 by position * f_i; cos and sin carry `amp`."""
+def rotate_halves(x, positions, freqs, amp, ang=None):
+    """x [..., T, dims]: channel i turns against channel i + dims / 2 by position * f_i (or by given angles [T, dims / 2]);
+    cos and sin carry `amp`."""
     half = len(freqs)
-    ang = positions.to(x.dtype).unsqueeze(-1) * torch.tensor(freqs, dtype=x.dtype)
+    if ang is None:
+        ang = positions.to(x.dtype).unsqueeze(-1) * torch.tensor(freqs, dtype=x.dtype)
     c, s = torch.cos(ang) * amp, torch.sin(ang) * amp
     u, v = x[..., :half], x[..., half:2 * half]
     return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], dim=-1)
