@@ -96,7 +96,7 @@ latent_rope_norm_store_kernel(const float* __restrict__ x, long long x_stride, c
 // its row holds the queries alone.  Grid (tokens, parts): part 0 writes the cache row, all parts share the query channels.
 constexpr int QL_THREADS = 256;
 
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(QL_THREADS)
 latent_q_rope_store_kernel(MaybePartial<float> x, long long x_stride, T* __restrict__ q_out, long long q_stride, int heads, int dim,
                            const float* __restrict__ gain, int rank, int rot, const float* __restrict__ freqs, int pairs, float amp,
@@ -115,9 +115,25 @@ latent_q_rope_store_kernel(MaybePartial<float> x, long long x_stride, T* __restr
     sn_s[i] = sn * amp; cs_s[i] = cs * amp;
   }
   __syncthreads();
+  if (VEC) {                                  // eight channels a thread, 16-byte accesses (rot and dim multiples of 8)
+    const int per8 = (rot + dim) / 8;
+    for (int idx = blockIdx.y * QL_THREADS + tid; idx < heads * per8; idx += gridDim.y * QL_THREADS) {
+      const int i = idx % per8 * 4;           // the piece's first pair within its head
+      float u[8];
+      x.at8(row + (size_t)idx * 8, u);
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        if (i + k < pairs) {
+          const float a = u[2 * k], b = u[2 * k + 1];
+          u[2 * k] = a * cs_s[i + k] - b * sn_s[i + k];
+          u[2 * k + 1] = b * cs_s[i + k] + a * sn_s[i + k];
+        }
+      Vec8<T>::store(q_out + (size_t)t * q_stride + (size_t)idx * 8, u);
+    }
+  }
   // two neighbouring channels a thread: every head is an even number of channels before its plain part, which may end odd
   const int per = rot + dim, half = (per + 1) / 2;
-  for (int idx = blockIdx.y * QL_THREADS + tid; idx < heads * half; idx += gridDim.y * QL_THREADS) {
+  for (int idx = blockIdx.y * QL_THREADS + tid; !VEC && idx < heads * half; idx += gridDim.y * QL_THREADS) {
     const int h = idx / half, i = idx - h * half, c = 2 * i;
     const size_t at = row + (size_t)h * per + c;
     float u = x.at(at), v = c + 1 < per ? x.at(at + 1) : 0.f;
@@ -165,15 +181,16 @@ LLMK_API int llmk_latent_q_rope_store(const float* x, const float* partials, int
   LLMK_REQUIRE(heads > 0 && dim > 0 && rot >= 0 && rot % 2 == 0 && pairs >= 0 && 2 * pairs <= rot && pairs <= 512,
                "latent_q_rope_store: bad sizes: %d heads of %d + %d channels, %d pairs", heads, rot, dim, pairs);
   LLMK_REQUIRE(pages == nullptr || (rank > 0 && rank <= 8192 && row_width >= rot + rank), "latent_q_rope_store: bad rank %d or row width %d", rank, row_width);
-  const int items = heads * ((rot + dim + 1) / 2);
   // few tokens: a token's channels are spread over several CTAs
-  const int parts = n_tokens >= 256 ? 1 : max(1, min(16, items / QL_THREADS));
+  const int items = heads * ((rot + dim + 7) / 8);
+  const int parts = n_tokens >= 256 ? 1 : max(1, min(16, (items + QL_THREADS - 1) / QL_THREADS));
   return dispatch_dtype(dtype, [&](auto* tag) {
     using T = LLMK_ELEM(tag);
     MaybePartial<float> src{x, partials, splits, split_stride};
-    launch_kernel(latent_q_rope_store_kernel<T>, dim3(n_tokens, parts), dim3(QL_THREADS), pages ? (size_t)rank * sizeof(float) : 0, stream, src,
-                  x_stride, (T*)q_out, q_stride, heads, dim, gain, rank, rot, freqs, pairs, amp, positions, eps, slot_map, (T*)pages,
-                  row_width);
+    const bool vec = rot % 8 == 0 && dim % 8 == 0 && src.vector_ok() && x_stride % 8 == 0 && q_stride % 8 == 0 && (uintptr_t)q_out % 16 == 0;
+    launch_kernel(vec ? latent_q_rope_store_kernel<T, true> : latent_q_rope_store_kernel<T, false>, dim3(n_tokens, parts), dim3(QL_THREADS),
+                  pages ? (size_t)rank * sizeof(float) : 0, stream, src, x_stride, (T*)q_out, q_stride, heads, dim, gain, rank, rot, freqs,
+                  pairs, amp, positions, eps, slot_map, (T*)pages, row_width);
     LLMK_LAUNCH_CHECK("latent_q_rope_store");
   });
 }

@@ -90,7 +90,8 @@ lightning_decode_kernel(float* __restrict__ out, long long out_stride, MaybePart
 }
 
 // ---- prompt portions -----------------------------------------------------------------------------------------
-constexpr int CC = 64, VT = 64, WARPS = 4, THREADS = WARPS * 32, PAD = 8, VP = VT + PAD;
+constexpr int CC = 64, VT = 64, WARPS = 8, THREADS = WARPS * 32, PAD = 8, VP = VT + PAD;
+constexpr int HALF = VT / 2;          // a warp of chunk_out makes 16 tokens x HALF columns, one of chunk_state 16 rows x HALF columns
 using bf16 = __nv_bfloat16;
 
 // The chunk with the running number idx: its entry, first token, length and place among its entry's chunks; false when the
@@ -146,6 +147,7 @@ __global__ void __launch_bounds__(THREADS)
 lightning_chunk_state_kernel(const bf16* __restrict__ k, const bf16* __restrict__ v, long long stride, const float* __restrict__ decay,
                              const int* __restrict__ cu_tokens, int n_entries, int heads, int dim, int vdim, float* __restrict__ seg) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
+  __shared__ float pw[CC];
   pdl_launch_dependents();
   pdl_wait();
   int c0, n;
@@ -153,35 +155,39 @@ lightning_chunk_state_kernel(const bf16* __restrict__ k, const bf16* __restrict_
   const int head = blockIdx.y, col0 = blockIdx.z * VT, kp = dim + PAD;
   bf16* k_s = reinterpret_cast<bf16*>(smem_raw);          // [CC][dim + PAD]
   bf16* v_s = k_s + CC * kp;                              // [3][CC][VP]: the decayed values in three pieces
-  const float d = decay[head];
   bring_rows(k_s, kp, k + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
-  {
-    const bf16* src = v + (size_t)c0 * stride + (size_t)head * vdim + col0;
-    for (int i = threadIdx.x; i < CC * (VT / 8); i += THREADS) {
-      const int r = i / (VT / 8), c = (i % (VT / 8)) * 8;
-      float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-      if (r < n && col0 + c < vdim) {
-        Vec8<bf16>::load(src + (size_t)r * stride + c, x);
-        const float w = powf(d, (float)(n - 1 - r));
+  // a thread's eight-column pieces of the values: requested first, scaled and split when the powers of the decay are there
+  constexpr int PIECES = CC * (VT / 8) / THREADS;
+  const bf16* src = v + (size_t)c0 * stride + (size_t)head * vdim + col0;
+  float x[PIECES][8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) x[j] *= w;
-      }
-      uint32_t p[4][3];
+  for (int p = 0; p < PIECES; ++p) {
+    const int i = threadIdx.x + p * THREADS, r = i / (VT / 8), c = (i % (VT / 8)) * 8;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) split3(x[2 * j], x[2 * j + 1], p[j]);
+    for (int j = 0; j < 8; ++j) x[p][j] = 0.f;
+    if (r < n && col0 + c < vdim) Vec8<bf16>::load(src + (size_t)r * stride + c, x[p]);
+  }
+  if (threadIdx.x < CC) pw[threadIdx.x] = powf(decay[head], (float)threadIdx.x);
+  __syncthreads();
 #pragma unroll
-      for (int s = 0; s < 3; ++s)
-        *reinterpret_cast<uint4*>(v_s + (s * CC + r) * VP + c) = make_uint4(p[0][s], p[1][s], p[2][s], p[3][s]);
-    }
+  for (int p = 0; p < PIECES; ++p) {
+    const int i = threadIdx.x + p * THREADS, r = i / (VT / 8), c = (i % (VT / 8)) * 8;
+    const float w = r < n ? pw[n - 1 - r] : 0.f;
+    uint32_t q[4][3];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) split3(x[p][2 * j] * w, x[p][2 * j + 1] * w, q[j]);
+#pragma unroll
+    for (int s = 0; s < 3; ++s)
+      *reinterpret_cast<uint4*>(v_s + (s * CC + r) * VP + c) = make_uint4(q[0][s], q[1][s], q[2][s], q[3][s]);
   }
   cp_async_wait_all();
   __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, half = (warp & 1) * HALF;
   float* dst = seg + ((size_t)blockIdx.x * heads + head) * dim * vdim;
-  for (int m0 = warp * 16; m0 < dim; m0 += WARPS * 16) {  // 16 rows of the state at a time
-    float acc[VT / 8][4];
+  for (int m0 = (warp >> 1) * 16; m0 < dim; m0 += WARPS / 2 * 16) {      // 16 rows of the state x HALF columns at a time
+    float acc[HALF / 8][4];
 #pragma unroll
-    for (int i = 0; i < VT / 8; ++i)
+    for (int i = 0; i < HALF / 8; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
 #pragma unroll
@@ -191,20 +197,20 @@ lightning_chunk_state_kernel(const bf16* __restrict__ k, const bf16* __restrict_
 #pragma unroll
       for (int s = 0; s < 3; ++s)
 #pragma unroll
-        for (int x = 0; x < VT / 16; ++x) {
+        for (int i = 0; i < HALF / 16; ++i) {
           uint32_t b[4];
-          ldsm4_t(b, v_s + (s * CC + t0 + (lane & 15)) * VP + x * 16 + ((lane >> 4) << 3));
-          mma(acc[2 * x], a, b[0], b[1]);
-          mma(acc[2 * x + 1], a, b[2], b[3]);
+          ldsm4_t(b, v_s + (s * CC + t0 + (lane & 15)) * VP + half + i * 16 + ((lane >> 4) << 3));
+          mma(acc[2 * i], a, b[0], b[1]);
+          mma(acc[2 * i + 1], a, b[2], b[3]);
         }
     }
     const int r = m0 + (lane >> 2);
 #pragma unroll
-    for (int x = 0; x < VT / 8; ++x) {
-      const int c = col0 + x * 8 + 2 * (lane & 3);
+    for (int i = 0; i < HALF / 8; ++i) {
+      const int c = col0 + half + i * 8 + 2 * (lane & 3);
       if (c >= vdim) continue;
-      *reinterpret_cast<float2*>(dst + (size_t)r * vdim + c) = make_float2(acc[x][0], acc[x][1]);
-      *reinterpret_cast<float2*>(dst + (size_t)(r + 8) * vdim + c) = make_float2(acc[x][2], acc[x][3]);
+      *reinterpret_cast<float2*>(dst + (size_t)r * vdim + c) = make_float2(acc[i][0], acc[i][1]);
+      *reinterpret_cast<float2*>(dst + (size_t)(r + 8) * vdim + c) = make_float2(acc[i][2], acc[i][3]);
     }
   }
 }
@@ -244,7 +250,7 @@ lightning_chunk_chain_kernel(float* __restrict__ seg, const float* __restrict__ 
   *S_g = S;
 }
 
-// The outputs of a chunk: a warp per 16 tokens.  Grid (chunks, heads, value tiles).
+// The outputs of a chunk: two warps per 16 tokens, each half of the columns.  Grid (chunks, heads, value tiles).
 __global__ void __launch_bounds__(THREADS)
 lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const bf16* __restrict__ q, const bf16* __restrict__ k,
                            const bf16* __restrict__ v, long long stride, const float* __restrict__ decay,
@@ -261,33 +267,47 @@ lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const 
   bf16* k_s = q_s + CC * kp;                              // [CC][dim + PAD]
   bf16* v_s = k_s + CC * kp;                              // [CC][VP]
   bf16* S_s = v_s + CC * VP;                              // [3][dim][VP]: the state that enters the chunk in three pieces
+  // the state first (its pieces are made in registers), four eight-column pieces a thread in flight
+  constexpr int BATCH = 4;
+  const float* src = seg + ((size_t)blockIdx.x * heads + head) * dim * vdim + col0;
+  float x[BATCH][8];
+  auto fetch = [&](int i0) {
+#pragma unroll
+    for (int p = 0; p < BATCH; ++p) {
+      const int i = i0 + threadIdx.x + p * THREADS, r = i / (VT / 8), c = (i % (VT / 8)) * 8;
+      if (r < dim && col0 + c < vdim) Vec8<float>::load(src + (size_t)r * vdim + c, x[p]);
+      else
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[p][j] = 0.f;
+    }
+  };
+  fetch(0);
   bring_rows(q_s, kp, q + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
   bring_rows(k_s, kp, k + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
   bring_rows(v_s, VP, v + (size_t)c0 * stride + (size_t)head * vdim + col0, stride, n, min(VT, vdim - col0), VT);
-  const float d = decay[head];
-  if (threadIdx.x <= CC) pw[threadIdx.x] = powf(d, (float)threadIdx.x);
-  {
-    const float* src = seg + ((size_t)blockIdx.x * heads + head) * dim * vdim + col0;
-    for (int i = threadIdx.x; i < dim * (VT / 8); i += THREADS) {
-      const int r = i / (VT / 8), c = (i % (VT / 8)) * 8;
-      float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-      if (col0 + c < vdim) Vec8<float>::load(src + (size_t)r * vdim + c, x);
-      uint32_t p[4][3];
+  if (threadIdx.x <= CC) pw[threadIdx.x] = powf(decay[head], (float)threadIdx.x);
+  for (int i0 = 0; i0 < dim * (VT / 8); i0 += BATCH * THREADS) {
+    if (i0) fetch(i0);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) split3(x[2 * j], x[2 * j + 1], p[j]);
+    for (int p = 0; p < BATCH; ++p) {
+      const int i = i0 + threadIdx.x + p * THREADS, r = i / (VT / 8), c = (i % (VT / 8)) * 8;
+      if (r >= dim) continue;
+      uint32_t w[4][3];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) split3(x[p][2 * j], x[p][2 * j + 1], w[j]);
 #pragma unroll
       for (int s = 0; s < 3; ++s)
-        *reinterpret_cast<uint4*>(S_s + (s * dim + r) * VP + c) = make_uint4(p[0][s], p[1][s], p[2][s], p[3][s]);
+        *reinterpret_cast<uint4*>(S_s + (s * dim + r) * VP + c) = make_uint4(w[0][s], w[1][s], w[2][s], w[3][s]);
     }
   }
   cp_async_wait_all();
   __syncthreads();
-  const int lane = threadIdx.x & 31, i0 = (threadIdx.x >> 5) * 16;
+  const int lane = threadIdx.x & 31, i0 = (threadIdx.x >> 6) * 16, half = ((threadIdx.x >> 5) & 1) * HALF;
   if (i0 >= n) return;
   const bf16* q_at = q_s + (i0 + (lane & 15)) * kp + ((lane >> 4) << 3);
-  float o[VT / 8][4];
+  float o[HALF / 8][4];
 #pragma unroll
-  for (int i = 0; i < VT / 8; ++i)
+  for (int i = 0; i < HALF / 8; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
   // what the state that enters the chunk contributes: d^(i+1) S_0^T q_i
@@ -298,18 +318,18 @@ lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const 
 #pragma unroll
     for (int s = 0; s < 3; ++s)
 #pragma unroll
-      for (int x = 0; x < VT / 16; ++x) {
+      for (int i = 0; i < HALF / 16; ++i) {
         uint32_t b[4];
-        ldsm4_t(b, S_s + (s * dim + k0 + (lane & 15)) * VP + x * 16 + ((lane >> 4) << 3));
-        mma(o[2 * x], a, b[0], b[1]);
-        mma(o[2 * x + 1], a, b[2], b[3]);
+        ldsm4_t(b, S_s + (s * dim + k0 + (lane & 15)) * VP + half + i * 16 + ((lane >> 4) << 3));
+        mma(o[2 * i], a, b[0], b[1]);
+        mma(o[2 * i + 1], a, b[2], b[3]);
       }
   }
   const int ra = i0 + (lane >> 2), rb = ra + 8;           // the lane's two rows
 #pragma unroll
-  for (int x = 0; x < VT / 8; ++x) {
-    o[x][0] *= pw[ra + 1]; o[x][1] *= pw[ra + 1];
-    o[x][2] *= pw[rb + 1]; o[x][3] *= pw[rb + 1];
+  for (int i = 0; i < HALF / 8; ++i) {
+    o[i][0] *= pw[ra + 1]; o[i][1] *= pw[ra + 1];
+    o[i][2] *= pw[rb + 1]; o[i][3] *= pw[rb + 1];
   }
   // the chunk's own tokens, 16 keys at a time up to the warp's last row
   for (int j0 = 0; j0 <= i0; j0 += 16) {
@@ -323,11 +343,11 @@ lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const 
       mma(p[1], a, b[2], b[3]);
     }
 #pragma unroll
-    for (int x = 0; x < 2; ++x)
+    for (int i = 0; i < 2; ++i)
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        const int dist = (c < 2 ? ra : rb) - (j0 + 8 * x + 2 * (lane & 3) + (c & 1));
-        p[x][c] = dist >= 0 ? p[x][c] * pw[dist] : 0.f;
+        const int dist = (c < 2 ? ra : rb) - (j0 + 8 * i + 2 * (lane & 3) + (c & 1));
+        p[i][c] = dist >= 0 ? p[i][c] * pw[dist] : 0.f;
       }
     uint32_t w[4][3];
     split3(p[0][0], p[0][1], w[0]);
@@ -335,24 +355,24 @@ lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const 
     split3(p[1][0], p[1][1], w[2]);
     split3(p[1][2], p[1][3], w[3]);
 #pragma unroll
-    for (int x = 0; x < VT / 16; ++x) {
+    for (int i = 0; i < HALF / 16; ++i) {
       uint32_t b[4];
-      ldsm4_t(b, v_s + (j0 + (lane & 15)) * VP + x * 16 + ((lane >> 4) << 3));
+      ldsm4_t(b, v_s + (j0 + (lane & 15)) * VP + half + i * 16 + ((lane >> 4) << 3));
 #pragma unroll
       for (int s = 0; s < 3; ++s) {
         const uint32_t a[4] = {w[0][s], w[1][s], w[2][s], w[3][s]};
-        mma(o[2 * x], a, b[0], b[1]);
-        mma(o[2 * x + 1], a, b[2], b[3]);
+        mma(o[2 * i], a, b[0], b[1]);
+        mma(o[2 * i + 1], a, b[2], b[3]);
       }
     }
   }
 #pragma unroll
-  for (int x = 0; x < VT / 8; ++x) {
-    const int c = col0 + x * 8 + 2 * (lane & 3);
+  for (int i = 0; i < HALF / 8; ++i) {
+    const int c = col0 + half + i * 8 + 2 * (lane & 3);
     if (c >= vdim) continue;
     float* dst = out + (size_t)head * vdim + c;
-    if (ra < n) *reinterpret_cast<float2*>(dst + (size_t)(c0 + ra) * out_stride) = make_float2(o[x][0], o[x][1]);
-    if (rb < n) *reinterpret_cast<float2*>(dst + (size_t)(c0 + rb) * out_stride) = make_float2(o[x][2], o[x][3]);
+    if (ra < n) *reinterpret_cast<float2*>(dst + (size_t)(c0 + ra) * out_stride) = make_float2(o[i][0], o[i][1]);
+    if (rb < n) *reinterpret_cast<float2*>(dst + (size_t)(c0 + rb) * out_stride) = make_float2(o[i][2], o[i][3]);
   }
 }
 

@@ -245,25 +245,25 @@ row_rmsnorm_sigmoid_kernel(T* __restrict__ out, const float* __restrict__ x, con
   const size_t base = (size_t)blockIdx.x * n, g0 = (size_t)blockIdx.x * gate_stride + gate_col;
   float ss = 0.f;
   if constexpr (NV > 0) {
-    float v[NV][8];
+    float v[NV][8], m[NV][8];                 // m: weight times gate, on the way under the sum of squares
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * 256 + threadIdx.x) * 8;
       if (c >= n) continue;
+      float z[8];
       Vec8<float>::load(x + base + c, v[i]);
+      gate.at8(g0 + c, z);
+      Vec8<float>::load(w + c, m[i]);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) ss = fmaf(v[i][k], v[i][k], ss);
+      for (int k = 0; k < 8; ++k) { ss = fmaf(v[i][k], v[i][k], ss); m[i][k] /= 1.f + expf(-z[k]); }
     }
     const float rstd = 1.f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * 256 + threadIdx.x) * 8;
       if (c >= n) continue;
-      float g[8], z[8];
-      Vec8<float>::load(w + c, g);
-      gate.at8(g0 + c, z);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) v[i][k] *= rstd * g[k] / (1.f + expf(-z[k]));
+      for (int k = 0; k < 8; ++k) v[i][k] *= rstd * m[i][k];
       Vec8<T>::store(out + base + c, v[i]);
     }
   } else {
