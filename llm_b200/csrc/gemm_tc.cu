@@ -108,6 +108,8 @@ enum : int { ERR_PRODUCER = 1, ERR_MMA = 2, ERR_EPILOGUE = 3 };
 //   by_tile  row tile blockIdx.x belongs to group tile_group[blockIdx.x] and multiplies by rows
 //            g * w_row_step .. of W; tiles from *n_tiles on do nothing: the experts of a routed
 //            feed-forward over rows that were sorted by expert, each expert's run padded to whole tiles.
+//            In the swapped mode (few rows per group) a tile is tile_q rows, numbered by blockIdx.y, and the
+//            group's weights take the 128-row side: no bytes are brought for rows that are not there.
 // act: an activation on the float32 accumulator before the store (-1 none; 0 relu^2, 1 gelu erf,
 // 2 gelu tanh, 3 silu).  gate (by_z): row p of product g is multiplied by sigmoid(gate[p, g]).
 struct Grouping {
@@ -165,8 +167,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
   if (grp.mode == 2) {
     // which tiles are in use is what the kernel before this one wrote: wait for it first
     pdl_wait();
-    if ((int)blockIdx.x >= *grp.n_tiles) return;
-    group = grp.tile_group[blockIdx.x];
+    const int row_tile = SWAP ? blockIdx.y : blockIdx.x;
+    if (row_tile >= *grp.n_tiles) return;
+    group = grp.tile_group[row_tile];
   } else if (grp.mode == 1) {
     group = blockIdx.z;
   }
@@ -318,7 +321,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
       }
       if (p >= p_limit) continue;
       const int q = q0 + c;
-      if (!SWAP && grp.act >= 0) {
+      if (!CLUSTER && grp.act >= 0) {
 #pragma unroll
         for (int j = 0; j < CHUNK; ++j) v[j] = epilogue_act(v[j], grp.act);
       }
@@ -1220,6 +1223,30 @@ LLMK_API int llmk_gemm_tc_grouped(const void* A, const void* W, void* C, int M, 
   if (out_dtype == LLMK_BF16) return tile <= 128 ? LLMK_GROUPED(128, __nv_bfloat16) : LLMK_GROUPED(256, __nv_bfloat16);
 #undef LLMK_GROUPED
   return llmk_fail(-1, "gemm_tc_grouped: unsupported output kind %d", out_dtype);
+}
+
+// The same by row tile for few rows per group (a decode step's experts), in the swapped mode: row tiles of `tile` (16 or 32)
+// rows, the weights on the 128-row side of the MMA as a stream of TMA boxes with two CTAs per SM.  M a multiple of tile.
+LLMK_API int llmk_gemm_tc_grouped_few(const void* A, const void* W, void* C, int M, int N, int K, long long lda, long long ldw,
+                                      long long ldc, int out_dtype, int groups, const int* tile_group, const int* n_tiles, int act,
+                                      int tile, cudaStream_t stream) {
+  if (M == 0 || N == 0 || groups == 0) return 0;
+  LLMK_REQUIRE(llmk_gemm_tc_supported(A, W, M, N, K, lda, ldw), "gemm_tc_grouped_few: K=%d and the row pitches must be multiples of 8 and the bases 16-byte aligned", K);
+  LLMK_REQUIRE((tile == 16 || tile == 32) && M % tile == 0 && M / tile <= 65535 && tile_group && n_tiles,
+               "gemm_tc_grouped_few: tile %d (16 or 32) must divide M=%d, and the tile table must be given", tile, M);
+  LLMK_REQUIRE(act >= -1 && act <= 3, "gemm_tc_grouped_few: unknown activation %d", act);
+  int rc = ensure_err_flag();
+  if (rc) return rc;
+  CUtensorMap mp, mq;
+  if ((rc = get_map(&mp, W, (uint64_t)groups * N, K, ldw, BP))) return rc;
+  if ((rc = get_map(&mq, A, M, (uint64_t)K, lda, tile))) return rc;
+  const Grouping grp{2, 0, N, tile_group, n_tiles, act, nullptr, 0};
+  const int kb = (K + BK - 1) / BK;
+#define LLMK_GROUPED_FEW(BNQ, TOut) launch_cfg<BNQ, true, TOut, false>(mp, mq, C, ldc, 0, M, N, K, 1, kb, tile, stream, grp)
+  if (out_dtype == LLMK_F32) return tile == 16 ? LLMK_GROUPED_FEW(16, float) : LLMK_GROUPED_FEW(32, float);
+  if (out_dtype == LLMK_BF16) return tile == 16 ? LLMK_GROUPED_FEW(16, __nv_bfloat16) : LLMK_GROUPED_FEW(32, __nv_bfloat16);
+#undef LLMK_GROUPED_FEW
+  return llmk_fail(-1, "gemm_tc_grouped_few: unsupported output kind %d", out_dtype);
 }
 
 // Whether llmk_gemm_tc_qkv_rope takes these sizes and pointers.

@@ -184,73 +184,90 @@ lightning_chunk_state_kernel(const bf16* __restrict__ k, const bf16* __restrict_
   __syncthreads();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, half = (warp & 1) * HALF;
   float* dst = seg + ((size_t)blockIdx.x * heads + head) * dim * vdim;
-  for (int m0 = (warp >> 1) * 16; m0 < dim; m0 += WARPS / 2 * 16) {      // 16 rows of the state x HALF columns at a time
-    float acc[HALF / 8][4];
+  // a warp makes two tiles of 16 rows x HALF columns at a time, so that a piece of the values it loads serves both
+  for (int m0 = (warp >> 1) * 32; m0 < dim; m0 += WARPS / 2 * 32) {
+    const bool two = m0 + 16 < dim;
+    float acc[2][HALF / 8][4];
 #pragma unroll
-    for (int i = 0; i < HALF / 8; ++i)
+    for (int h = 0; h < 2; ++h)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+      for (int i = 0; i < HALF / 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[h][i][j] = 0.f;
 #pragma unroll
     for (int t0 = 0; t0 < CC; t0 += 16) {
-      uint32_t a[4];
-      ldsm4_t(a, k_s + (t0 + (lane & 7) + ((lane >> 4) << 3)) * kp + m0 + (((lane >> 3) & 1) << 3));
+      uint32_t a[2][4];
+      const bf16* at = k_s + (t0 + (lane & 7) + ((lane >> 4) << 3)) * kp + m0 + (((lane >> 3) & 1) << 3);
+      ldsm4_t(a[0], at);
+      ldsm4_t(a[1], two ? at + 16 : at);
 #pragma unroll
       for (int s = 0; s < 3; ++s)
 #pragma unroll
         for (int i = 0; i < HALF / 16; ++i) {
           uint32_t b[4];
           ldsm4_t(b, v_s + (s * CC + t0 + (lane & 15)) * VP + half + i * 16 + ((lane >> 4) << 3));
-          mma(acc[2 * i], a, b[0], b[1]);
-          mma(acc[2 * i + 1], a, b[2], b[3]);
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            mma(acc[h][2 * i], a[h], b[0], b[1]);
+            mma(acc[h][2 * i + 1], a[h], b[2], b[3]);
+          }
         }
     }
-    const int r = m0 + (lane >> 2);
 #pragma unroll
-    for (int i = 0; i < HALF / 8; ++i) {
-      const int c = col0 + half + i * 8 + 2 * (lane & 3);
-      if (c >= vdim) continue;
-      *reinterpret_cast<float2*>(dst + (size_t)r * vdim + c) = make_float2(acc[i][0], acc[i][1]);
-      *reinterpret_cast<float2*>(dst + (size_t)(r + 8) * vdim + c) = make_float2(acc[i][2], acc[i][3]);
+    for (int h = 0; h < 2; ++h) {
+      if (h && !two) break;
+      const int r = m0 + 16 * h + (lane >> 2);
+#pragma unroll
+      for (int i = 0; i < HALF / 8; ++i) {
+        const int c = col0 + half + i * 8 + 2 * (lane & 3);
+        if (c >= vdim) continue;
+        *reinterpret_cast<float2*>(dst + (size_t)r * vdim + c) = make_float2(acc[h][i][0], acc[h][i][1]);
+        *reinterpret_cast<float2*>(dst + (size_t)(r + 8) * vdim + c) = make_float2(acc[h][i][2], acc[h][i][3]);
+      }
     }
   }
 }
 
 // seg[chunk] holds the chunk's own contribution on entry and the state that enters the chunk on exit; the request's state
-// moves to the end of the entry.  A thread per four elements of the state; eight chunks' loads are issued together.
+// moves to the end of the entry.  A thread per two elements of the state; sixteen chunks' loads are issued together.
+constexpr int CHAIN = 16;
+
 __global__ void __launch_bounds__(256)
 lightning_chunk_chain_kernel(float* __restrict__ seg, const float* __restrict__ decay, float* __restrict__ state, long long slot_stride,
                              const int* __restrict__ state_slots, const int* __restrict__ cu_tokens, int heads, int dim, int vdim) {
   pdl_launch_dependents();
   pdl_wait();
-  const size_t per = (size_t)heads * dim * vdim / 4;
+  const size_t per = (size_t)heads * dim * vdim / 2;
   const size_t el = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (el >= per) return;
   const int entry = blockIdx.y;
   size_t first = 0;
   for (int e = 0; e < entry; ++e) first += (cu_tokens[e + 1] - cu_tokens[e] + CC - 1) / CC;
   const int len = cu_tokens[entry + 1] - cu_tokens[entry], chunks = (len + CC - 1) / CC;
-  const float d = decay[el / ((size_t)dim * vdim / 4)];
+  const float d = decay[el / ((size_t)dim * vdim / 2)];
   const float whole = powf(d, (float)CC), last = powf(d, (float)(len - (chunks - 1) * CC));
-  float4* S_g = reinterpret_cast<float4*>(state + (size_t)state_slots[entry] * slot_stride) + el;
-  float4* at = reinterpret_cast<float4*>(seg) + first * per + el;
-  float4 S = *S_g;
-  for (int c0 = 0; c0 < chunks; c0 += 8) {
-    float4 own[8];
+  float2* S_g = reinterpret_cast<float2*>(state + (size_t)state_slots[entry] * slot_stride) + el;
+  float2* at = reinterpret_cast<float2*>(seg) + first * per + el;
+  float2 S = *S_g;
+  for (int c0 = 0; c0 < chunks; c0 += CHAIN) {
+    float2 own[CHAIN];
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < CHAIN; ++i)
       if (c0 + i < chunks) own[i] = at[(size_t)(c0 + i) * per];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < CHAIN; ++i) {
       if (c0 + i >= chunks) break;
       at[(size_t)(c0 + i) * per] = S;
       const float w = c0 + i + 1 < chunks ? whole : last;
-      S.x = fmaf(w, S.x, own[i].x); S.y = fmaf(w, S.y, own[i].y); S.z = fmaf(w, S.z, own[i].z); S.w = fmaf(w, S.w, own[i].w);
+      S.x = fmaf(w, S.x, own[i].x); S.y = fmaf(w, S.y, own[i].y);
     }
   }
   *S_g = S;
 }
 
-// The outputs of a chunk: two warps per 16 tokens, each half of the columns.  Grid (chunks, heads, value tiles).
+// The outputs of a chunk: two warps per 16 tokens, each half of the columns.  Grid (chunks, heads, value tiles).  KD > 0: the
+// warp keeps its queries in registers (dim = 16 KD); 0: it reads them again where it needs them.
+template <int KD>
 __global__ void __launch_bounds__(THREADS)
 lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const bf16* __restrict__ q, const bf16* __restrict__ k,
                            const bf16* __restrict__ v, long long stride, const float* __restrict__ decay,
@@ -305,16 +322,27 @@ lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const 
   const int lane = threadIdx.x & 31, i0 = (threadIdx.x >> 6) * 16, half = ((threadIdx.x >> 5) & 1) * HALF;
   if (i0 >= n) return;
   const bf16* q_at = q_s + (i0 + (lane & 15)) * kp + ((lane >> 4) << 3);
+  const int kd = KD > 0 ? KD : dim / 16;
+  uint32_t qr[KD > 0 ? KD : 1][4];
+  if constexpr (KD > 0) {
+#pragma unroll
+    for (int x = 0; x < KD; ++x) ldsm4(qr[x], q_at + 16 * x);
+  }
+  auto query = [&](int x, uint32_t (&a)[4]) {
+    if constexpr (KD > 0) { a[0] = qr[x][0]; a[1] = qr[x][1]; a[2] = qr[x][2]; a[3] = qr[x][3]; }
+    else ldsm4(a, q_at + 16 * x);
+  };
   float o[HALF / 8][4];
 #pragma unroll
   for (int i = 0; i < HALF / 8; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
   // what the state that enters the chunk contributes: d^(i+1) S_0^T q_i
-#pragma unroll 2
-  for (int k0 = 0; k0 < dim; k0 += 16) {
+#pragma unroll KD > 0 ? KD : 2
+  for (int x = 0; x < kd; ++x) {
+    const int k0 = 16 * x;
     uint32_t a[4];
-    ldsm4(a, q_at + k0);
+    query(x, a);
 #pragma unroll
     for (int s = 0; s < 3; ++s)
 #pragma unroll
@@ -334,10 +362,11 @@ lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const 
   // the chunk's own tokens, 16 keys at a time up to the warp's last row
   for (int j0 = 0; j0 <= i0; j0 += 16) {
     float p[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-#pragma unroll 4
-    for (int k0 = 0; k0 < dim; k0 += 16) {
+#pragma unroll KD > 0 ? KD : 4
+    for (int x = 0; x < kd; ++x) {
+      const int k0 = 16 * x;
       uint32_t a[4], b[4];
-      ldsm4(a, q_at + k0);
+      query(x, a);
       ldsm4(b, k_s + (j0 + (lane & 7) + ((lane >> 4) << 3)) * kp + k0 + (((lane >> 3) & 1) << 3));
       mma(p[0], a, b[0], b[1]);
       mma(p[1], a, b[2], b[3]);
@@ -416,13 +445,15 @@ LLMK_API int llmk_lightning_chunks(float* out, long long out_stride, const void*
   const size_t smem1 = ((size_t)CC * (dim + PAD) + 3 * CC * VP) * sizeof(bf16);
   const size_t smem3 = ((size_t)2 * CC * (dim + PAD) + CC * VP + (size_t)3 * dim * VP) * sizeof(bf16);
   cudaFuncSetAttribute(lightning_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
-  cudaFuncSetAttribute(lightning_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
+  auto outputs = dim == 128 ? lightning_chunk_out_kernel<8> : dim == 64 ? lightning_chunk_out_kernel<4>
+               : dim == 32 ? lightning_chunk_out_kernel<2> : lightning_chunk_out_kernel<0>;
+  cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
   launch_kernel(lightning_chunk_state_kernel, dim3(chunks, heads, tiles), dim3(THREADS), smem1, stream, (const bf16*)k, (const bf16*)v, stride,
                 decay, cu_tokens, n_entries, heads, dim, vdim, seg);
-  const size_t per = (size_t)heads * dim * vdim / 4;
+  const size_t per = (size_t)heads * dim * vdim / 2;
   launch_kernel(lightning_chunk_chain_kernel, dim3((unsigned)((per + 255) / 256), n_entries), dim3(256), 0, stream, seg, decay, state,
                 slot_stride, state_slots, cu_tokens, heads, dim, vdim);
-  launch_kernel(lightning_chunk_out_kernel, dim3(chunks, heads, tiles), dim3(THREADS), smem3, stream, out, out_stride, (const bf16*)q,
+  launch_kernel(outputs, dim3(chunks, heads, tiles), dim3(THREADS), smem3, stream, out, out_stride, (const bf16*)q,
                 (const bf16*)k, (const bf16*)v, stride, decay, cu_tokens, n_entries, heads, dim, vdim, (const float*)seg);
   LLMK_LAUNCH_CHECK("lightning_chunks");
 }

@@ -897,6 +897,17 @@ GROUPED_PERSISTENT = os.environ.get("LLM_B200_GROUPED_PERSISTENT", "1") != "0"  
 MOE_TC_TILE = 128       # slots per tile of the tensor-core grouped products (the MMA's 128 rows)
 
 
+FEW_ROW_EXPERTS = True  # False: every step's experts run in tiles of 128 slots
+
+
+def moe_tc_tile(n_pairs: int, experts: int) -> int:
+    """Slots per tile of the tensor-core grouped products for a step of n_pairs (token, choice) pairs: with few rows per
+    expert 16 or 32 (the weights then take the MMA's 128-row side), else 128."""
+    if not FEW_ROW_EXPERTS or n_pairs > 24 * experts:
+        return MOE_TC_TILE
+    return 16 if n_pairs <= 10 * experts else 32
+
+
 def moe_max_tiles(n_pairs: int, experts: int, tile: int = 0) -> int:
     """Tiles that the grouped list of n_pairs (token, choice) pairs can take at most."""
     return _ceil_div(n_pairs, tile or moe_tile()) + min(experts, n_pairs)
@@ -959,16 +970,25 @@ def moe_gemm_tc_available(a: torch.Tensor, w: torch.Tensor) -> bool:
             and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def moe_gemm_tc(a: torch.Tensor, tile_expert, meta, w: torch.Tensor, out: torch.Tensor, max_tiles: int, act=None) -> None:
+def moe_gemm_tc(a: torch.Tensor, tile_expert, meta, w: torch.Tensor, out: torch.Tensor, max_tiles: int, act=None,
+                tile: int = MOE_TC_TILE) -> None:
     """out[slot] = act(a[slot] @ w[expert of the slot's tile].T) on the tensor cores: a [slots, K] in slot order
-    (tiles of 128 slots), w [experts, N, K], out bfloat16 or float32 [slots, N].  act "silu_gate": an expert's N rows
-    are N/2 gate rows followed by N/2 up rows and out [slots, N/2] bfloat16 = silu(gate) * up, made in the epilogue."""
+    (tiles of 128, 32 or 16 slots), w [experts, N, K], out bfloat16 or float32 [slots, N].  act "silu_gate": an expert's N rows
+    are N/2 gate rows followed by N/2 up rows and out [slots, N/2] bfloat16 = silu(gate) * up, made in the epilogue (tiles
+    of 128)."""
     _rows_contig(a, "a"); _rows_contig(out, "out")
     gated = act == "silu_gate"
     assert w.dim() == 3 and w.is_contiguous() and a.shape[1] == w.shape[2] and out.shape[1] == (w.shape[1] // 2 if gated else w.shape[1])
     assert not gated or (out.dtype == torch.bfloat16 and w.shape[1] % 2 == 0)
-    rows = max_tiles * MOE_TC_TILE
+    rows = max_tiles * tile
     assert a.shape[0] >= rows and out.shape[0] >= rows
+    if tile != MOE_TC_TILE:
+        assert not gated
+        _check_t(load_tensor().llmk_gemm_tc_grouped_few(
+            _ptr(a), _ptr(w), _ptr(out), c_int(rows), c_int(w.shape[1]), c_int(w.shape[2]), c_longlong(a.stride(0)),
+            c_longlong(w.shape[2]), c_longlong(out.stride(0)), c_int(_kind(out.dtype)), c_int(w.shape[0]), _ptr(tile_expert), _ptr(meta),
+            c_int(ACTIVATIONS[act] if act else -1), c_int(tile), _stream()))
+        return
     _check_t(load_tensor().llmk_gemm_tc_grouped(
         _ptr(a), _ptr(w), _ptr(out), c_int(rows), c_int(w.shape[1]), c_int(w.shape[2]), c_longlong(a.stride(0)),
         c_longlong(w.shape[2]), c_longlong(out.stride(0)), c_int(_kind(out.dtype)), c_int(2), c_int(w.shape[0]), c_int(0),

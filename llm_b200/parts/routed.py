@@ -118,17 +118,21 @@ class RoutedFFN(Part):
     def forward(self, x: torch.Tensor, ctx, allow_unsummed: bool = False):
         """With allow_unsummed (and no shared expert) the result is an ops.WeightedRows, else a tensor."""
         T, ws, top, E = ctx.n_tokens, ctx.workspace, self.top, self.experts
-        # bfloat16 runs the experts on the tensor cores (tiles of 128 slots, rows gathered into slot order
-        # first); float32, and shapes the tensor-core kernel refuses, on the CUDA cores (tiles of 64)
+        # bfloat16 runs the experts on the tensor cores (tiles of 128 slots, or of 16 or 32 where an expert gets few rows; rows
+        # gathered into slot order first); float32, and shapes the tensor-core kernel refuses, on the CUDA cores (tiles of 64)
         tensor = ops.moe_gemm_tc_available(x, self.w_up) and self.expert_size % 8 == 0
-        pairs, tile = T * top, (ops.MOE_TC_TILE if tensor else ops.moe_tile())
+        pairs = T * top
+        tile = ops.moe_tc_tile(pairs, E) if tensor else ops.moe_tile()
+        fused_gate = self.gated and not self.clamped and self.hidden_size >= FUSE_GATE_FROM_WIDTH and tile == ops.MOE_TC_TILE
         max_tiles = ops.moe_max_tiles(pairs, E, tile)                 # of this step: a function of T alone
         cap_pairs = ws.max_rows * top
-        cap_slots = ops.moe_max_tiles(cap_pairs, E, tile) * tile      # of any step: the buffers' sizes
+        # of any step, in tiles of the largest size: the buffers' sizes (the lists of smaller tiles are shorter)
+        cap_tile = ops.MOE_TC_TILE if tensor else tile
+        cap_slots = ops.moe_max_tiles(cap_pairs, E, cap_tile) * cap_tile
         i32, f32 = torch.int32, torch.float32
         ids, wts = ws.flat("moe_ids", cap_pairs, i32), ws.flat("moe_weights", cap_pairs, f32)
         pair_slot, meta = ws.flat("moe_pair_slot", cap_pairs, i32), ws.flat("moe_meta", 4, i32)
-        tile_expert, slot_src = ws.flat("moe_tile_expert", cap_slots // tile, i32), ws.flat("moe_slot_src", cap_slots, i32)
+        tile_expert, slot_src = ws.flat("moe_tile_expert", cap_slots // 16, i32), ws.flat("moe_slot_src", cap_slots, i32)
         act = ws.flat("moe_act", cap_slots * self.expert_size, self.dtype).view(cap_slots, self.expert_size)
         y = ws.flat("moe_y", cap_slots * self.hidden_size, f32).view(cap_slots, self.hidden_size)
 
@@ -140,12 +144,13 @@ class RoutedFFN(Part):
             # gated experts: a tile multiplies by its expert's gate rows and up rows and the epilogue makes silu(gate) * up
             rows = ws.flat("moe_rows", cap_slots * self.hidden_size, self.dtype).view(cap_slots, self.hidden_size)
             ops.moe_gather(rows, x, slot_src, meta, top, tile, max_tiles)
-            if self.gated and (self.clamped or self.hidden_size < FUSE_GATE_FROM_WIDTH):
+            if self.gated and not fused_gate:
                 up_out = ws.flat("moe_gate_up", cap_slots * 2 * self.expert_size, self.dtype).view(cap_slots, 2 * self.expert_size)
-                ops.moe_gemm_tc(rows, tile_expert, meta, self.w_up, up_out, max_tiles)
+                ops.moe_gemm_tc(rows, tile_expert, meta, self.w_up, up_out, max_tiles, tile=tile)
                 self._gate(act[:max_tiles * tile], up_out[:max_tiles * tile], max_tiles * tile)
             else:
-                ops.moe_gemm_tc(rows, tile_expert, meta, self.w_up, act, max_tiles, act="silu_gate" if self.gated else self.activation)
+                ops.moe_gemm_tc(rows, tile_expert, meta, self.w_up, act, max_tiles, act="silu_gate" if self.gated else self.activation,
+                                tile=tile)
         elif self.gated:
             # on the CUDA cores the up product leaves [gate, up] per slot and a row kernel makes silu(gate) * up of it
             up_out = ws.flat("moe_gate_up", cap_slots * 2 * self.expert_size, self.dtype).view(cap_slots, 2 * self.expert_size)
@@ -154,7 +159,7 @@ class RoutedFFN(Part):
         else:
             ops.moe_gemm(x, top, slot_src, tile_expert, meta, self.w_up, act, max_tiles, act=self.activation)
         if tensor:
-            ops.moe_gemm_tc(act, tile_expert, meta, self.w_down, y, max_tiles)
+            ops.moe_gemm_tc(act, tile_expert, meta, self.w_down, y, max_tiles, tile=tile)
         else:
             ops.moe_gemm(act, 0, slot_src, tile_expert, meta, self.w_down, y, max_tiles)
         if allow_unsummed and self.leaves_unsummed:

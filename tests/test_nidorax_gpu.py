@@ -120,6 +120,33 @@ def test_softmax_router_chooses_among_the_best_groups(E, top, count, keep):
     assert max_err(wts[clear], w_ref[clear]) < 1e-5 and max_err(wts.sum(dim=1), torch.ones(T)) < 1e-5
 
 
+@pytest.mark.parametrize("tile", [16, 32, 128])
+@pytest.mark.parametrize("T,top,E,W,F", [(1, 2, 4, 64, 72), (8, 4, 16, 256, 200), (40, 3, 5, 128, 96), (64, 2, 3, 72, 136), (5, 1, 1, 2048, 1408)])
+def test_expert_products_in_tiles_of_few_rows(tile, T, top, E, W, F):
+    """Rows sorted by expert into tiles of 16, 32 or 128 slots, an expert's run over several tiles among them: up-projection with
+    the squared relu in the epilogue, then the down-projection into float32."""
+    from llm_b200.csrc import ops
+    g = torch.Generator().manual_seed(T * 100 + tile)
+    x, up, down = bf(torch.randn(T, W, generator=g)), bf(torch.randn(E, F, W, generator=g) / math.sqrt(W)), bf(torch.randn(E, W, F, generator=g) / math.sqrt(F))
+    choice = torch.stack([torch.randperm(E, generator=g)[:top] for _ in range(T)])
+    pairs, max_tiles = T * top, ops.moe_max_tiles(T * top, E, tile)
+    z = lambda n: torch.zeros(n, dtype=torch.int32, device="cuda")
+    meta, tile_expert, slot_src, pair_slot = z(4), z(max_tiles), z(max_tiles * tile), z(pairs)
+    ops.moe_group(choice.flatten().to(torch.int32).cuda(), pairs, E, meta, tile_expert, slot_src, pair_slot, max_tiles, tile)
+    rows = torch.full((max_tiles * tile, W), float("nan"), device="cuda", dtype=torch.bfloat16)
+    act = torch.full((max_tiles * tile, F), float("nan"), device="cuda", dtype=torch.bfloat16)
+    y = torch.full((max_tiles * tile, W), float("nan"), device="cuda")
+    ops.moe_gather(rows, dev(x, "bfloat16"), slot_src, meta, top, tile, max_tiles)
+    ops.moe_gemm_tc(rows, tile_expert, meta, dev(up, "bfloat16"), act, max_tiles, act="relu2", tile=tile)
+    ops.moe_gemm_tc(act, tile_expert, meta, dev(down, "bfloat16"), y, max_tiles, tile=tile)
+    assert ops.gemm_tc_take_error() == 0
+    a = torch.stack([P.relu_squared(x[t].double() @ up[int(e)].double().T) for t in range(T) for e in choice[t]])
+    slots = pair_slot.cpu().long()
+    assert max_err(act[slots.cuda()], a) < KTOL["bfloat16"]
+    ref = torch.stack([bf(a[i].float()).double() @ down[int(e)].double().T for i, e in enumerate(choice.flatten())])
+    assert max_err(y[slots.cuda()], ref) < 2e-2
+
+
 def _lightning_inputs(T, H, D, V, seed):
     g = torch.Generator().manual_seed(seed)
     q, k, v = bf(torch.randn(T, H * D, generator=g)), bf(torch.randn(T, H * D, generator=g)), bf(torch.randn(T, H * V, generator=g))
