@@ -345,7 +345,7 @@ def decode_attention_sweep(args, peaks, torch, ops) -> int:
         q = torch.randn(batch, n_heads * hs, device=dev, dtype=torch.bfloat16)
         out = torch.empty_like(q)
         call = lambda i: ops.paged_attention_decode(out, q, k_pages, v_pages, tables[i % sets], kv_lens, batch, n_heads, n_kv,
-                                                    hs, 0, 1.0 / math.sqrt(hs), max_keys=ctx)
+                                                    hs, 0, 1.0 / math.sqrt(hs), max_keys=ctx, head_parts=args.head_parts)
         for i in range(3):
             call(i)
         torch.cuda.synchronize()
@@ -646,6 +646,7 @@ def main() -> int:
                          "tevudra, fopivik, norusun: that design beside Llama at equal layer sizes, prompt and decode, with every kernel's time; "
                          "potipel: the same beside Fopivik; nidorax: beside Tevudra")
     ap.add_argument("--latent", action="store_true", help="decode_attention: the key pages are the value pages too")
+    ap.add_argument("--head-parts", type=int, default=1, help="decode_attention: CTAs that the query heads of a kv head are split over")
     ap.add_argument("--sizes", default="", help="tevudra, fopivik, norusun, potipel, nidorax: which of the sizes to run (comma-separated; default all)")
     ap.add_argument("--ctx", type=int, default=0, help="decode_attention: the context length of the one case to run")
     ap.add_argument("--prompt-tokens", type=int, default=PREFILL_TOKENS, help="timeline_prefill: tokens of the prompt step")

@@ -11,7 +11,7 @@ template <bool FUSED>
 int launch_decode_mma(void* out, long long out_stride, const void* q, long long q_stride, const void* k_pages,
                       const void* v_pages, const int* block_table, int table_width, const int* kv_lens,
                       int n_entries, int n_heads, int n_kv, int head_dim, int page_size, float scale, int window,
-                      int splits, int max_keys, float* scratch, decode_mma::FusedQkv fused, cudaStream_t stream) {
+                      int splits, int max_keys, float* scratch, decode_mma::FusedQkv fused, cudaStream_t stream, int kv_share = 1) {
   dim3 grid(splits, n_kv, n_entries);
   const float scale_log2e = scale * 1.4426950408889634f;
   const int group_rows = n_heads / n_kv < decode_mma::ROWS ? n_heads / n_kv : decode_mma::ROWS;
@@ -66,11 +66,11 @@ int launch_decode_mma(void* out, long long out_stride, const void* q, long long 
     cfg.numAttrs = llmk_pdl_enabled() ? 2 : 1;
     cudaLaunchKernelEx(&cfg, kern, (__nv_bfloat16*)out, out_stride, scratch, (const __nv_bfloat16*)q, q_stride,
                        (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, block_table, table_width, kv_lens, n_heads,
-                       n_kv, page_size, window, scale_log2e, splits, fused);
+                       n_kv, page_size, window, scale_log2e, splits, fused, kv_share);
   } else {
     launch_kernel(kern, grid, dim3(decode_mma::THREADS), (size_t)stage_bytes, stream, (__nv_bfloat16*)out, out_stride, scratch,
                   (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, block_table,
-                  table_width, kv_lens, n_heads, n_kv, page_size, window, scale_log2e, splits, fused);
+                  table_width, kv_lens, n_heads, n_kv, page_size, window, scale_log2e, splits, fused, kv_share);
   }
   LLMK_LAUNCH_CHECK("attention_decode_mma");
 }
@@ -88,15 +88,18 @@ LLMK_API int llmk_paged_attention_decode_mma_supported(const void* q, long long 
 // As llmk_paged_attention_decode (same arguments, same scratch), on the warp-level tensor cores:
 // the query heads of a group as rows of the MMAs.  max_keys: an upper bound of kv_lens that the
 // host knows (0: what a row of the table holds); it only picks between variants of the kernel.
+// kv_share > 1: n_kv counts groups of query heads, of which kv_share neighbours read one of the n_kv / kv_share heads
+// that the pages hold.
 LLMK_API int llmk_paged_attention_decode_mma(void* out, long long out_stride, const void* q, long long q_stride,
                                              const void* k_pages, const void* v_pages, const int* block_table,
                                              int table_width, const int* kv_lens, int n_entries, int n_heads, int n_kv,
                                              int head_dim, int page_size, int window, float scale, int splits,
-                                             float* scratch, int dtype, int max_keys, cudaStream_t stream) {
+                                             float* scratch, int dtype, int max_keys, cudaStream_t stream, int kv_share) {
   if (n_entries == 0) return 0;
   LLMK_REQUIRE(llmk_paged_attention_decode_mma_supported(q, q_stride, head_dim, page_size, dtype),
                "attention_decode_mma: needs bfloat16, a head size of 64 or 128 (got %d) and pages of a power of two (got %d)",
                head_dim, page_size);
+  LLMK_REQUIRE(kv_share >= 1 && n_kv % kv_share == 0, "attention_decode_mma: %d groups do not share key heads by %d", n_kv, kv_share);
   LLMK_REQUIRE(n_kv > 0 && n_heads % n_kv == 0, "attention_decode_mma: %d query heads do not divide into %d kv heads", n_heads, n_kv);
   LLMK_REQUIRE(splits >= 1 && splits <= 64, "attention_decode_mma: splits %d must be 1 to 64", splits);
   LLMK_REQUIRE(n_kv <= 65535 && n_entries <= 65535, "attention_decode_mma: grid too large");
@@ -105,7 +108,7 @@ LLMK_API int llmk_paged_attention_decode_mma(void* out, long long out_stride, co
   LLMK_REQUIRE(window >= 0, "attention_decode_mma: bad window %d", window);
   return launch_decode_mma<false>(out, out_stride, q, q_stride, k_pages, v_pages, block_table, table_width, kv_lens,
                                   n_entries, n_heads, n_kv, head_dim, page_size, scale, window, splits, max_keys, scratch,
-                                  decode_mma::FusedQkv{}, stream);
+                                  decode_mma::FusedQkv{}, stream, kv_share);
 }
 
 // Whether the fused rotate-store-attend kernel takes these sizes and pointers.

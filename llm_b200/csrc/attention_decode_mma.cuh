@@ -112,7 +112,7 @@ decode_attention_mma_kernel(__nv_bfloat16* __restrict__ out, long long out_strid
                             __nv_bfloat16* __restrict__ k_pages, __nv_bfloat16* __restrict__ v_pages,
                             const int* __restrict__ block_table, int table_width, const int* __restrict__ kv_lens,
                             int n_heads, int n_kv, int page_size, int window, float scale_log2e, int splits,
-                            FusedQkv fused) {
+                            FusedQkv fused, int kv_share) {
   constexpr int KS = HS / 16;                  // k-steps of Q K^T
   constexpr int DT = HS / 8;                   // 8-wide tiles of the output row
   constexpr int CH = HS / 8;                   // 16-byte chunks of a row
@@ -141,6 +141,9 @@ decode_attention_mma_kernel(__nv_bfloat16* __restrict__ out, long long out_strid
   const int split = blockIdx.x, g = blockIdx.y, e = blockIdx.z;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int group = n_heads / n_kv;
+  // kv_share > 1: that many neighbouring groups of query heads read one key/value head (a group of many heads split over
+  // several CTAs, each with its own pass over the keys): the pages hold n_kv / kv_share heads
+  const int kv_heads = n_kv / kv_share, g_kv = g / kv_share;
   // a length beyond the entry's table row is cut to what the row can hold; an entry without keys
   // gets zeros (every range of it sees the same length and leaves here, so nobody waits for anybody)
   const int n_held = min(kv_lens[e], table_width * page_size);
@@ -168,7 +171,7 @@ decode_attention_mma_kernel(__nv_bfloat16* __restrict__ out, long long out_strid
   // cost more than the tile's arithmetic
   const int page_shift = __ffs(page_size) - 1;
   auto row_of = [&](int k) -> size_t {
-    return ((((size_t)table[k >> page_shift] * n_kv + g) << page_shift) + (k & (page_size - 1))) * HS;
+    return ((((size_t)table[k >> page_shift] * kv_heads + g_kv) << page_shift) + (k & (page_size - 1))) * HS;
   };
   uint8_t* w_buf = vbuf + warp * WARP_BYTES;                 // stage st: keys at st * 2 * V_BYTES, values V_BYTES further
   const uint32_t w_addr = (uint32_t)__cvta_generic_to_shared(w_buf);

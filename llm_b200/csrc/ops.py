@@ -1180,13 +1180,29 @@ def decode_splits(n_entries: int, n_kv: int, max_keys: int, sms: int = 0) -> int
     return 6 if s in (7, 8) else s
 
 
+def decode_head_parts(n_entries: int, n_heads: int, n_kv: int, splits: int, latent: bool, sms: int = 0) -> int:
+    """Over how many CTAs the query heads of one kv head are split, each with its own pass over the keys (from L2).  More than
+    16 heads per kv head (the rows of the kernel's MMAs) always are; over a latent cache, whose one head serves them all, so are
+    fewer, down to four heads a CTA, while the grid then still runs at once (measured, 128 channels, us a launch: 16 heads,
+    8 requests of 584 keys 12.1 -> 6.7, of 4,096 keys 19.6 -> 15.5; 32 heads 24.3 -> 9.2, 37.9 -> 22.4; at 64 requests one
+    CTA for 16 heads stays ahead, 15.7 against 23.1)."""
+    group, parts = n_heads // n_kv, 1
+    while group // parts > 16 and group % (2 * parts) == 0:
+        parts *= 2
+    limit = 2 * (sms or sm_count())
+    while latent and group % (2 * parts) == 0 and group // (2 * parts) >= 4 and n_entries * n_kv * splits * 2 * parts <= limit:
+        parts *= 2
+    return parts
+
+
 def paged_attention_decode(out: torch.Tensor, q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                            block_table: torch.Tensor, kv_lens: torch.Tensor, n_entries: int, n_heads: int,
                            n_kv: int, head_dim: int, window: int, scale: float, splits=None, max_keys: int = 0,
                            softcap: float = 0.0, sink: bool = False, keep_first: int = 0, sink_values=None, dist_bias=None,
-                           v_share: int = 1) -> None:
+                           v_share: int = 1, head_parts: int = 1) -> None:
     """One query token per entry (row e of q), attending to its request's kv_lens[e] keys.
-    max_keys: an upper bound of kv_lens, if the host knows one below the table's width.
+    max_keys: an upper bound of kv_lens, if the host knows one below the table's width.  head_parts: the query heads of a kv
+    head are split over so many CTAs (the tensor-core kernel only).
     softcap, sink, keep_first, dist_bias, v_share: as in paged_attention_generic (the CUDA-core kernel takes them)."""
     _rows_contig(out, "out"); _rows_contig(q, "q")
     assert block_table.dim() == 2 and block_table.is_contiguous() and block_table.dtype == torch.int32
@@ -1210,7 +1226,8 @@ def paged_attention_decode(out: torch.Tensor, q: torch.Tensor, k_pages: torch.Te
     extended = bool(softcap or sink or keep_first or dist_bias is not None or v_share > 1)
     if (not extended and q.dtype == torch.bfloat16 and head_dim in (64, 128) and page & (page - 1) == 0
             and q.stride(0) % 2 == 0 and q.data_ptr() % 4 == 0):
-        _check_t(load_tensor().llmk_paged_attention_decode_mma(*args, c_int(max_keys), _stream()))
+        args = args[:11] + (c_int(n_kv * head_parts),) + args[12:]
+        _check_t(load_tensor().llmk_paged_attention_decode_mma(*args, c_int(max_keys), _stream(), c_int(head_parts)))
     else:
         _check(load().llmk_paged_attention_decode_ex(*args, _stream(), c_float(softcap or 0.0), c_int(int(bool(sink))),
                                                      c_int(keep_first or 0), _ptr(sink_values), _ptr(r1), _ptr(r2), c_int(v_share)))
@@ -1383,9 +1400,10 @@ def paged_attention(out, qkv, k_pages, v_pages, group, ctx, n_heads: int, n_kv: 
         max_keys = min(ctx.kv_bucket or 1 << 30, group.block_table.shape[1] * k_pages.shape[2])
         if window:
             max_keys = min(max_keys, window)
+        splits = decode_splits(ctx.n_entries, n_kv, max_keys)
         paged_attention_decode(out, qkv, k_pages, v_pages, group.block_table, ctx.kv_lens, ctx.n_entries,
-                               n_heads, n_kv, head_dim, window, scale,
-                               splits=decode_splits(ctx.n_entries, n_kv, max_keys), max_keys=max_keys)
+                               n_heads, n_kv, head_dim, window, scale, splits=splits, max_keys=max_keys,
+                               head_parts=decode_head_parts(ctx.n_entries, n_heads, n_kv, splits, k_pages is v_pages))
         return
     if attention_tc_supported(qkv.dtype, n_heads, n_kv, head_dim, k_pages.shape[2]) and qkv.stride(0) % 8 == 0:
         attention_tc(out, qkv, k_pages, v_pages, group.block_table, ctx.cu_tokens, ctx.kv_lens, ctx.n_tokens,

@@ -120,6 +120,32 @@ def test_softmax_router_chooses_among_the_best_groups(E, top, count, keep):
     assert max_err(wts[clear], w_ref[clear]) < 1e-5 and max_err(wts.sum(dim=1), torch.ones(T)) < 1e-5
 
 
+@pytest.mark.parametrize("D,heads,parts", [(128, 16, 1), (128, 16, 4), (64, 24, 2), (128, 32, 2), (64, 40, 8), (128, 6, 3)])
+@pytest.mark.parametrize("splits", [1, 3, 12])
+def test_decode_attention_with_the_heads_of_a_latent_split_over_ctas(D, heads, parts, splits):
+    from llm_b200.csrc import ops
+    g = torch.Generator().manual_seed(D + heads)
+    page, lens, scale = 16, [333, 70, 16, 1], 0.15
+    c = bf(torch.randn(len(lens), max(lens), D, generator=g))
+    q = bf(torch.randn(len(lens), heads * D, generator=g))
+    per = -(-max(lens) // page)
+    perm = torch.randperm(len(lens) * per, generator=g).view(len(lens), per)
+    pages = torch.zeros(len(lens) * per, 1, page, D)
+    for e in range(len(lens)):
+        for t in range(lens[e]):
+            pages[perm[e, t // page], 0, t % page] = c[e, t]
+    ref = torch.zeros(len(lens), heads, D, dtype=torch.float64)
+    for e, n in enumerate(lens):
+        s = torch.softmax(q[e].view(heads, D).double() @ c[e, :n].double().T * scale, dim=1)
+        ref[e] = s @ c[e, :n].double()
+    out = torch.empty(len(lens), heads * D, device="cuda", dtype=torch.bfloat16)
+    pd = dev(pages, "bfloat16")
+    for _ in range(2):                      # the arrival counters are zero again after a launch
+        ops.paged_attention_decode(out, dev(q, "bfloat16"), pd, pd, perm.to(torch.int32).cuda().contiguous(), i32(lens), len(lens), heads, 1, D, 0,
+                                   scale, splits=splits, max_keys=max(lens), head_parts=parts)
+        assert max_err(out, ref.view(len(lens), -1)) < 1e-2
+
+
 @pytest.mark.parametrize("tile", [16, 32, 128])
 @pytest.mark.parametrize("T,top,E,W,F", [(1, 2, 4, 64, 72), (8, 4, 16, 256, 200), (40, 3, 5, 128, 96), (64, 2, 3, 72, 136), (5, 1, 1, 2048, 1408)])
 def test_expert_products_in_tiles_of_few_rows(tile, T, top, E, W, F):
