@@ -517,6 +517,8 @@ NIDORAX_SIZES = {
              tevudra_routed_config(4096, 4, 32, 128, 128, 128, 0, 32, 4, 2752, 0)),
     "1024-row64": (nidorax_config(1024, "nlnb", 2, 16, 64, 48, 16, 16, 64, 64, 8, 2, 1408),
                    tevudra_routed_config(1024, 8, 16, 64, 64, 64, 0, 8, 2, 1408, 0)),
+    "2048-row576": (nidorax_config(2048, "nlnb", 1, 16, 128, 512, 64, 16, 128, 128, 16, 4, 1408),
+                    tevudra_routed_config(2048, 4, 16, 128, 128, 512, 0, 16, 4, 1408, 0)),
 }
 
 

@@ -114,10 +114,10 @@ int launch(const void* A, const void* W, void* C, int M, int N, int K, long long
 
 // Few rows (a decode step): one warp per (product, output column).  The warp keeps its weight row in
 // registers (lane l holds k = l, l + 32, ...), dots every row of A with it and sums over the lanes in a
-// fixed order; the weights are read once, as a stream.  K up to 32 * GEMV_PER_LANE.
-constexpr int GEMV_PER_LANE = 16, GEMV_WARPS = 4;
+// fixed order; the weights are read once, as a stream.  K up to 32 * PER_LANE, which is 4, 8 or GEMV_PER_LANE.
+constexpr int GEMV_PER_LANE = 20, GEMV_WARPS = 4;
 
-template <typename T>
+template <typename T, int PER_LANE>
 __global__ void __launch_bounds__(GEMV_WARPS * 32)
 gemv_batched_kernel(const T* __restrict__ A, const T* __restrict__ W, T* __restrict__ C, int M, int N, int K, long long lda,
                     long long ldw, long long ldc, long long a_batch, long long w_batch, long long c_batch,
@@ -127,9 +127,9 @@ gemv_batched_kernel(const T* __restrict__ A, const T* __restrict__ W, T* __restr
   const int n = blockIdx.x * GEMV_WARPS + warp, z = blockIdx.y;
   if (n >= N) return;
   const T* w_row = W + (size_t)z * w_batch + (size_t)n * ldw;
-  float wr[GEMV_PER_LANE];
+  float wr[PER_LANE];
 #pragma unroll
-  for (int i = 0; i < GEMV_PER_LANE; ++i) {
+  for (int i = 0; i < PER_LANE; ++i) {
     const int k = lane + 32 * i;
     wr[i] = k < K ? to_f32(w_row[k]) : 0.f;          // the weights do not depend on the kernel before
   }
@@ -138,7 +138,7 @@ gemv_batched_kernel(const T* __restrict__ A, const T* __restrict__ W, T* __restr
     const T* a_row = A + (size_t)m * lda + (size_t)z * a_batch;
     float s = 0.f;
 #pragma unroll
-    for (int i = 0; i < GEMV_PER_LANE; ++i) {
+    for (int i = 0; i < PER_LANE; ++i) {
       const int k = lane + 32 * i;
       if (k < K) s = fmaf(to_f32(a_row[k]), wr[i], s);
     }
@@ -182,7 +182,8 @@ LLMK_API int llmk_gemm_simt_batched(const void* A, const void* W, void* C, int M
     // a decode step in bfloat16: the weights as a stream, one warp per output column (float32 keeps the tiled
     // kernel at every row count, so that its sums never depend on how many rows a step brings)
     using T = __nv_bfloat16;
-    launch_kernel(gemv_batched_kernel<T>, dim3((N + GEMV_WARPS - 1) / GEMV_WARPS, batches), dim3(GEMV_WARPS * 32), 0, stream,
+    auto kern = K <= 128 ? gemv_batched_kernel<T, 4> : K <= 256 ? gemv_batched_kernel<T, 8> : gemv_batched_kernel<T, GEMV_PER_LANE>;
+    launch_kernel(kern, dim3((N + GEMV_WARPS - 1) / GEMV_WARPS, batches), dim3(GEMV_WARPS * 32), 0, stream,
                   (const T*)A, (const T*)W, (T*)C, M, N, K, lda, ldw, ldc, a_batch, w_batch, c_batch, (const T*)gate, gate_stride);
     LLMK_LAUNCH_CHECK("gemv_batched");
   }

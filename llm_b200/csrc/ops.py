@@ -1150,6 +1150,7 @@ def sample_rows(out: torch.Tensor, logits: torch.Tensor, rows: int, temperature=
                                    c_int(logits.shape[1]), _ptr(temperature), _ptr(uniform), _stream()))
 
 
+_ATTN_COUNTER_WORDS = 4096       # arrival counters of the decode kernels, at the head of the scratch
 _ATTN_PARTIALS = {}
 _ATTN_PARTIALS_RETIRED = []      # outgrown buffers stay alive: captured graphs may still hold their addresses
 
@@ -1317,6 +1318,40 @@ def attention_tc_take_error() -> int:
     return int(load_tensor().llmk_attention_tc_take_error())
 
 
+ATTENTION_WIDE_WIDTHS = (192, 256, 320, 384, 512, 576, 640)      # cached rows that attention_wide takes
+ATTENTION_WIDE = True      # False: latents wider than 128 run on the general kernels
+
+
+def attention_wide(out: torch.Tensor, q: torch.Tensor, pages: torch.Tensor, block_table: torch.Tensor, cu_tokens: torch.Tensor,
+                   kv_lens: torch.Tensor, n_tokens: int, n_entries: int, n_heads: int, scale: float, decode: bool = False,
+                   max_keys: int = 0, splits: int = 0) -> None:
+    """Causal attention over a latent cache with wide rows (bfloat16; pages [pages, 1, page_size, W] serve as keys and values of
+    all heads): q and out [n_tokens, n_heads * W], arguments else as in attention_tc.  decode: every entry brings one token; the
+    keys are then split over ranges (splits, or by the batch and max_keys) and tiles of 16 rows serve up to 32 heads."""
+    width = pages.shape[3]
+    assert q.dtype == pages.dtype == out.dtype == torch.bfloat16 and pages.is_contiguous() and pages.shape[1] == 1
+    assert q.is_contiguous() and out.is_contiguous() and q.shape[1] == out.shape[1] == n_heads * width
+    assert block_table.dim() == 2 and block_table.is_contiguous() and block_table.dtype == cu_tokens.dtype == kv_lens.dtype == torch.int32
+    small = decode and n_heads <= 32
+    if not splits:
+        splits = 1
+        if decode:
+            tiles = n_entries * _ceil_div(n_heads, 16 if small else 64)
+            keys = max_keys or block_table.shape[1] * pages.shape[2]
+            splits = max(1, min(32, sm_count() // tiles, _ceil_div(keys, 128)))
+    part_o = part_ml = None
+    if splits > 1:
+        rows = n_tokens * n_heads
+        buf = _attn_partials(q.device, _ATTN_COUNTER_WORDS + rows * splits * (width + 2))
+        part_o = buf[_ATTN_COUNTER_WORDS:_ATTN_COUNTER_WORDS + rows * splits * width]      # the first words stay the arrival counters
+        part_ml = buf[_ATTN_COUNTER_WORDS + rows * splits * width:]
+        count_launches(1)
+    _check_t(load_tensor().llmk_attention_wide(
+        _ptr(out), _ptr(q), _ptr(pages), _ptr(block_table), c_int(block_table.shape[1]), _ptr(cu_tokens), _ptr(kv_lens), c_int(n_tokens),
+        c_int(n_entries), c_int(n_heads), c_int(width), c_int(pages.shape[2]), c_float(scale), c_int(int(small)), c_int(splits), _ptr(part_o),
+        _ptr(part_ml), _stream()))
+
+
 ATTENTION_FAST_OPTIONS = True      # False: the distance bias and shared values always run on the general kernel
 
 
@@ -1327,8 +1362,8 @@ def paged_attention(out, qkv, k_pages, v_pages, group, ctx, n_heads: int, n_kv: 
     """Attention of the step's tokens over their requests' pages; q is the first
     n_heads * head_dim columns of qkv.  Chooses the kernel for the batch: in bfloat16 the
     split-key decode kernel when every entry brings one token and the tcgen05 kernel otherwise,
-    where it takes the sizes; the general kernel for float32 and for all other sizes (head sizes
-    off the 16-grid among them).  value_dim, softcap, sink, keep_first: see paged_attention_generic, the kernel
+    where it takes the sizes; over latents wider than 128 channels attention_wide; the general kernel for float32 and for all
+    other sizes (head sizes off the 16-grid among them).  value_dim, softcap, sink, keep_first: see paged_attention_generic, the kernel
     that takes them in every combination.  sink_values (a learned score per head for the sink), chunk and sigmoid_bias (a
     chunked mask, sigmoid weights): the tcgen05 kernel for steps with prompt portions where it takes the sizes; else the
     split-key decode kernel (sink_values) or the general kernel, whose one warp per (token, head) walks at most one chunk.
@@ -1395,6 +1430,13 @@ def paged_attention(out, qkv, k_pages, v_pages, group, ctx, n_heads: int, n_kv: 
         paged_attention_generic(out, qkv, k_pages, v_pages, group.block_table, ctx.token_entry, ctx.positions,
                                 ctx.n_tokens, n_heads, n_kv, head_dim, window, scale, value_dim=value_dim,
                                 softcap=softcap, sink=sink, keep_first=keep_first, sink_values=sink_values)
+        return
+    if (ATTENTION_WIDE and k_pages is v_pages and n_kv == 1 and not window and qkv.dtype == torch.bfloat16
+            and head_dim in ATTENTION_WIDE_WIDTHS and qkv.is_contiguous() and out.is_contiguous()):
+        # a latent whose rows are wider than the tcgen05 kernel takes
+        attention_wide(out, qkv, k_pages, group.block_table, ctx.cu_tokens, ctx.kv_lens, ctx.n_tokens, ctx.n_entries, n_heads, scale,
+                       decode=ctx.decode_only,
+                       max_keys=min(ctx.kv_bucket or 1 << 30, group.block_table.shape[1] * k_pages.shape[2]))
         return
     if ctx.decode_only and qkv.dtype == torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 256:
         max_keys = min(ctx.kv_bucket or 1 << 30, group.block_table.shape[1] * k_pages.shape[2])

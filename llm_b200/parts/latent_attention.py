@@ -69,13 +69,13 @@ class LatentAttention(Part):
             raise ValueError(f"latent attention: {self.position.dims} turning channels do not fit a part of {self.rot_dim}")
         self.q_size = num_heads * (head_dim + self.rot_dim)
         rank = rank + self.rot_dim          # what a cached row holds: the turned key part, then the latent
-        # The width of a cached row.  The tensor-core attention kernels (bfloat16) take heads of 64 or 128: a
-        # smaller rank is padded up to the next of the two with zeros (in the cache rows and in the two per-head
-        # maps), which changes no score and no output and costs cache, not correctness.  Other ranks, and
-        # float32, keep their width and run on the general kernels.
+        # The width of a cached row.  The tensor-core attention kernels (bfloat16) take rows of 64, 128 and some wider sizes: a
+        # row is padded up to the next of them with zeros (in the cache rows and in the two per-head maps), which changes no
+        # score and no output and costs cache, not correctness.  Wider rows, and float32, keep their width and run on the
+        # general kernels.
         self.row_width = rank
-        if dtype == torch.bfloat16 and rank < 128 and rank != 64:
-            self.row_width = 64 if rank < 64 else 128
+        if dtype == torch.bfloat16:
+            self.row_width = next((w for w in (64, 128) + ops.ATTENTION_WIDE_WIDTHS if w >= rank), rank)
         self.w_in = None          # [q; down; gate] stacked: one product per step
         self.w_uk_t = None        # [heads, rank, dim]: the key map, transposed per head
         self.w_uv = None          # [heads, vdim, rank]

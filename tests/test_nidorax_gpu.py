@@ -120,6 +120,46 @@ def test_softmax_router_chooses_among_the_best_groups(E, top, count, keep):
     assert max_err(wts[clear], w_ref[clear]) < 1e-5 and max_err(wts.sum(dim=1), torch.ones(T)) < 1e-5
 
 
+@pytest.mark.parametrize("W,heads,page", [(192, 2, 16), (256, 6, 8), (320, 16, 32), (384, 1, 16), (512, 20, 16), (576, 16, 16), (640, 33, 64)])
+def test_attention_over_wide_latents(W, heads, page):
+    """Ragged portions behind cached tokens, beside single tokens; then single tokens alone with the keys in one range and in
+    several (an empty one among them); shuffled pages, unused rows poisoned.  One key a row stands far out."""
+    from llm_b200.csrc import ops
+    g = torch.Generator().manual_seed(W + heads)
+    held, new = [150, 65, 1, 300, 33], [150, 1, 1, 90, 32]
+    E, scale = len(held), 0.7 / math.sqrt(W)
+    c = bf(torch.randn(E, max(held), W, generator=g))
+    q = bf(torch.randn(sum(new), heads, W, generator=g))
+    for r in range(0, sum(new), 5):                                   # these rows ask for one key, at different distances
+        e = max(i for i in range(E) if sum(new[:i]) <= r)
+        pos = held[e] - new[e] + r - sum(new[:e])
+        q[r] = bf(3.0 * c[e, (r * 37) % (pos + 1)])
+    per = -(-max(held) // page)
+    perm = torch.randperm(E * per + 2, generator=g)[:E * per].view(E, per)
+    pages = torch.full((E * per + 2, 1, page, W), float("nan"))
+    for e in range(E):
+        for t in range(held[e]):
+            pages[perm[e, t // page], 0, t % page] = c[e, t]
+    ref, cu = [], [0]
+    for e in range(E):
+        for i in range(new[e]):
+            n = held[e] - new[e] + i + 1
+            s = torch.softmax(q[cu[e] + i].double() @ c[e, :n].double().T * scale, dim=1)
+            ref.append((s @ c[e, :n].double()).flatten())
+        cu.append(cu[-1] + new[e])
+    ref = torch.stack(ref)
+    pd, table, qd = dev(pages, "bfloat16"), perm.to(torch.int32).cuda().contiguous(), dev(q.view(-1, heads * W), "bfloat16")
+    out = torch.full_like(qd, float("nan"))
+    ops.attention_wide(out, qd, pd, table, i32(cu), i32(held), cu[-1], E, heads, scale)
+    assert max_err(out, ref) < 1.2e-2          # P is rounded to bfloat16 before the second product
+    last = [n - 1 for n in cu[1:]]
+    for splits in (1, 2, 7, 0):
+        out = torch.full((E, heads * W), float("nan"), device="cuda", dtype=torch.bfloat16)
+        ops.attention_wide(out, qd[last].contiguous(), pd, table, i32(list(range(E + 1))), i32(held), E, E, heads, scale, decode=True,
+                           max_keys=max(held), splits=splits)
+        assert max_err(out, ref[last]) < 1.2e-2
+
+
 @pytest.mark.parametrize("D,heads,parts", [(128, 16, 1), (128, 16, 4), (64, 24, 2), (128, 32, 2), (64, 40, 8), (128, 6, 3)])
 @pytest.mark.parametrize("splits", [1, 3, 12])
 def test_decode_attention_with_the_heads_of_a_latent_split_over_ctas(D, heads, parts, splits):
