@@ -143,7 +143,8 @@ decode_attention_mma_kernel(__nv_bfloat16* __restrict__ out, long long out_strid
   const int group = n_heads / n_kv;
   // kv_share > 1: that many neighbouring groups of query heads read one key/value head (a group of many heads split over
   // several CTAs, each with its own pass over the keys): the pages hold n_kv / kv_share heads
-  const int kv_heads = n_kv / kv_share, g_kv = g / kv_share;
+  // (not with FUSED, which stores a key per group: nothing is divided there)
+  const int kv_heads = FUSED ? n_kv : n_kv / kv_share, g_kv = FUSED ? g : g / kv_share;
   // a length beyond the entry's table row is cut to what the row can hold; an entry without keys
   // gets zeros (every range of it sees the same length and leaves here, so nobody waits for anybody)
   const int n_held = min(kv_lens[e], table_width * page_size);

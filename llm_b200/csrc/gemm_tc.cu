@@ -136,7 +136,8 @@ __device__ __forceinline__ float epilogue_act(float z, int kind) {
 // along blockIdx.z.  Instead of writing float32 partial results to global memory for a later
 // kernel to sum, each CTA hands its accumulator to the first CTA of the cluster through
 // distributed shared memory; that CTA adds them in the order of the splits and stores the result.
-template <int BNQ, bool SWAP, typename TOut, bool CLUSTER>
+// FEW: the swapped mode over row tiles by group (see Grouping, by_tile).
+template <int BNQ, bool SWAP, typename TOut, bool CLUSTER, bool FEW = false>
 __global__ void __launch_bounds__(THREADS, SWAP ? 2 : 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant__ CUtensorMap map_q,
                TOut* __restrict__ C, long long ldc, long long split_stride, int M, int N, int K,
@@ -167,7 +168,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
   if (grp.mode == 2) {
     // which tiles are in use is what the kernel before this one wrote: wait for it first
     pdl_wait();
-    const int row_tile = SWAP ? blockIdx.y : blockIdx.x;
+    const int row_tile = FEW ? blockIdx.y : blockIdx.x;
     if (row_tile >= *grp.n_tiles) return;
     group = grp.tile_group[row_tile];
   } else if (grp.mode == 1) {
@@ -321,7 +322,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
       }
       if (p >= p_limit) continue;
       const int q = q0 + c;
-      if (!CLUSTER && grp.act >= 0) {
+      if ((!SWAP || FEW) && grp.act >= 0) {
 #pragma unroll
         for (int j = 0; j < CHUNK; ++j) v[j] = epilogue_act(v[j], grp.act);
       }
@@ -948,11 +949,11 @@ int ensure_err_flag() {
   return 0;
 }
 
-template <int BNQ, bool SWAP, typename TOut, bool CLUSTER>
+template <int BNQ, bool SWAP, typename TOut, bool CLUSTER, bool FEW = false>
 int launch_cfg(const CUtensorMap& mp, const CUtensorMap& mq, void* C, long long ldc, long long split_stride, int M,
                int N, int K, int splits, int kb_per_split, int tile_q, cudaStream_t stream,
                const Grouping grp = Grouping{0, 0, 0, nullptr, nullptr, -1, nullptr, 0}) {
-  auto kern = gemm_tc_kernel<BNQ, SWAP, TOut, CLUSTER>;
+  auto kern = gemm_tc_kernel<BNQ, SWAP, TOut, CLUSTER, FEW>;
   constexpr int smem = smem_bytes_for(BNQ, SWAP);
   static bool configured = false;
   if (!configured) {
@@ -1242,7 +1243,7 @@ LLMK_API int llmk_gemm_tc_grouped_few(const void* A, const void* W, void* C, int
   if ((rc = get_map(&mq, A, M, (uint64_t)K, lda, tile))) return rc;
   const Grouping grp{2, 0, N, tile_group, n_tiles, act, nullptr, 0};
   const int kb = (K + BK - 1) / BK;
-#define LLMK_GROUPED_FEW(BNQ, TOut) launch_cfg<BNQ, true, TOut, false>(mp, mq, C, ldc, 0, M, N, K, 1, kb, tile, stream, grp)
+#define LLMK_GROUPED_FEW(BNQ, TOut) launch_cfg<BNQ, true, TOut, false, true>(mp, mq, C, ldc, 0, M, N, K, 1, kb, tile, stream, grp)
   if (out_dtype == LLMK_F32) return tile == 16 ? LLMK_GROUPED_FEW(16, float) : LLMK_GROUPED_FEW(32, float);
   if (out_dtype == LLMK_BF16) return tile == 16 ? LLMK_GROUPED_FEW(16, __nv_bfloat16) : LLMK_GROUPED_FEW(32, __nv_bfloat16);
 #undef LLMK_GROUPED_FEW
