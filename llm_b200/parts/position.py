@@ -63,7 +63,7 @@ class PairRotary(Part):
     scaling_kind "yarn" (scaling {factor, original, fast, slow}) blends by index instead of wavelength: with
     at(t) = dims ln(original / (2 pi t)) / (2 ln base), the (fractional) pair that makes t turns within the original length,
     f_i keeps its value below lo = max(floor(at(fast)), 0), is divided by factor above hi = min(ceil(at(slow)), dims - 1),
-    and runs linearly in i between; cos and sin are multiplied by `amplitude` = 0.1 ln(factor) + 1 (1 otherwise)."""
+    and runs linearly in i between; `amplitude`, 0.1 ln(factor) + 1 (1 without this scaling), goes on both cos and sin."""
 
     role = "position"
     SCALING_KEYS = {"wavelength": ("factor", "low", "high", "original"), "yarn": ("factor", "original", "fast", "slow")}
