@@ -648,6 +648,109 @@ class NidoraxConfig:
 
 
 @dataclass(frozen=True)
+class KepevikConfig:
+    """config.json of a Kepevik folder: a decoder with a norm before and after every sublayer and a learned scale on its
+    result, whose `layers` list gives every layer one by one.  Keys: `architecture`, `width`, `vocab`, `norm.eps`,
+    `embedding.scale`, and per layer `type`, `mixer`, `mlp` (`dense` with `ff`; `moe` with `expert.ff`, `router.{experts, top,
+    identity}` and `shared.ff`, the last two optional; or null).  Mixers:
+      mlstm     heads, dim, vdim, gate_cap
+      parallel  left  {heads, kv_heads, dim, vdim, scale, rot {dims, base}}      (attention, the keys being the values)
+                right {heads, kv_heads, dim, vdim, conv}                         (delta rule with a decay per channel)
+                left_scale, right_scale
+    The design has no length limit of its own: max_position (optional) bounds what the engine sizes its tables for."""
+
+    architecture: str
+    width: int
+    vocab: int
+    norm_eps: float
+    embedding_scale: float
+    layers: tuple                      # of dicts, validated
+    max_position: int = 131072
+    eos_token_id: Optional[int] = None
+
+    MIXERS = ("mlstm", "parallel")
+
+    @staticmethod
+    def _ints(d, keys, where):
+        out = {k: _take(d, k, int) for k in keys}
+        if min(out.values()) <= 0:
+            raise ConfigError(f"config.json: {where}: sizes must be positive")
+        return out
+
+    @classmethod
+    def _mixer(cls, kind: str, m: dict, where: str) -> dict:
+        if kind == "mlstm":
+            mixer = cls._ints(m, ("heads", "dim", "vdim"), where)
+            mixer["gate_cap"] = _take(m, "gate_cap", float)
+            if not mixer["gate_cap"] > 0:
+                raise ConfigError(f"config.json: {where}.gate_cap must be positive")
+            return mixer
+        if kind == "parallel":
+            left, right = _take(m, "left", dict), _take(m, "right", dict)
+            a = cls._ints(left, ("heads", "kv_heads", "dim", "vdim"), where + ".left")
+            a["scale"] = _take(left, "scale", float)
+            a["rot_dims"], a["rot_base"] = _rot_of(left, where + ".left", a["dim"])
+            b = cls._ints(right, ("heads", "kv_heads", "dim", "vdim", "conv"), where + ".right")
+            if a["heads"] % a["kv_heads"] or b["heads"] % b["kv_heads"]:
+                raise ConfigError(f"config.json: {where}: heads must be a multiple of kv_heads")
+            if a["vdim"] != a["dim"]:
+                raise ConfigError(f"config.json: {where}.left: the keys are the values, so vdim {a['vdim']} must equal dim {a['dim']}")
+            if b["conv"] > 16:
+                raise ConfigError(f"config.json: {where}.right: a convolution has at most 16 taps")
+            return {"left": a, "right": b, "left_scale": _take(m, "left_scale", float), "right_scale": _take(m, "right_scale", float)}
+        raise ConfigError(f"config.json: {where[:-6]}.type '{kind}' is not a mixer of this design {cls.MIXERS}")
+
+    @classmethod
+    def _mlp(cls, ff, where: str):
+        if ff is None:
+            return None
+        if not isinstance(ff, dict):
+            raise ConfigError(f"config.json: {where} must be an object or null")
+        kind = _take(ff, "kind", str)
+        if kind == "dense":
+            return dict(cls._ints(ff, ("ff",), where), kind="dense")
+        if kind == "moe":
+            router = _take(ff, "router", dict)
+            mlp = dict(cls._ints(router, ("experts", "top"), where + ".router"), kind="moe")
+            mlp["ff"] = cls._ints(_take(ff, "expert", dict), ("ff",), where + ".expert")["ff"]
+            mlp["identity"] = _take(router, "identity", int, 0)
+            shared = _take(ff, "shared", dict, None)
+            mlp["shared"] = cls._ints(shared, ("ff",), where + ".shared")["ff"] if shared is not None else 0
+            if mlp["identity"] < 0 or not (mlp["top"] <= mlp["experts"] + mlp["identity"] <= 256):
+                raise ConfigError(f"config.json: {where}.router: top {mlp['top']} of {mlp['experts']} + {mlp['identity']} experts "
+                                  f"(at most 256)")
+            return mlp
+        raise ConfigError(f"config.json: {where}.kind '{kind}' is not 'dense' or 'moe'")
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "KepevikConfig":
+        norm = _take(d, "norm", dict)
+        layers = _take(d, "layers", list)
+        if not layers:
+            raise ConfigError("config.json: 'layers' must list at least one layer")
+        out = []
+        for i, layer in enumerate(layers):
+            where = f"layers[{i}]"
+            if not isinstance(layer, dict):
+                raise ConfigError(f"config.json: {where} must be an object")
+            kind = _take(layer, "type", str)
+            out.append({"type": kind, "mixer": cls._mixer(kind, _take(layer, "mixer", dict), where + ".mixer"),
+                        "mlp": cls._mlp(layer.get("mlp"), where + ".mlp")})
+        eos = d.get("eos_token_id")
+        cfg = cls(architecture=_take(d, "architecture", str), width=_take(d, "width", int), vocab=_take(d, "vocab", int),
+                  norm_eps=_take(norm, "eps", float), embedding_scale=_take(_take(d, "embedding", dict), "scale", float),
+                  layers=tuple(out), max_position=_take(d, "max_position", int, 131072),
+                  eos_token_id=eos if isinstance(eos, int) else None)
+        if cfg.width <= 0 or cfg.vocab <= 0 or cfg.max_position <= 0:
+            raise ConfigError("config.json: width, vocab and max_position must be positive")
+        return cfg
+
+    @property
+    def max_position_embeddings(self) -> int:
+        return self.max_position
+
+
+@dataclass(frozen=True)
 class Architecture:
     """One registry entry: how to read the config and how to lay the model out."""
 

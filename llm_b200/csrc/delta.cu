@@ -5,6 +5,9 @@
 //   q_t, k_t unit vectors per head (x / sqrt(sum(x^2) + 1e-6)), q_t also times q_scale;
 //   beta_t = sigmoid(b_t),  g_t = exp(-exp(A_log) softplus(a_t + dt_bias))                   one number per head and token
 //
+// or, with a decay per key channel (CH), g_t = diag(exp(-exp(A_log) softplus(z_t + dt_bias))), z_t and dt_bias [dim] per head: the
+// rows of S decay each on its own, S^T k is taken over k times the decays, and everything else stays.
+//
 // Head h reads q/k head h / (heads / qk_heads).  The state is float32 and lives in the request's state slot (zero at
 // admission); it is read at the start of an entry's tokens and written back at their end, so a whole prompt, a portion and a
 // single token run the same arithmetic, in the same order, whatever else is in the batch.  Norms, beta, the decay, the
@@ -36,15 +39,15 @@ struct DeltaArgs {
   float* out; long long out_stride;                       // [T, heads * vdim] float32
   const void *q, *k; long long qk_stride;                 // [T, qk_heads * dim]
   const void* v; long long v_stride;                      // [T, heads * vdim]
-  const void *b, *a; long long ba_stride;                 // [T, heads] each
-  const float *a_log, *dt_bias;                           // [heads]
+  const void *b, *a; long long b_stride, a_stride;        // b [T, heads]; a [T, heads], or (CH) float32 [T, heads * dim]
+  const float *a_log, *dt_bias;                           // [heads]; (CH) dt_bias [heads * dim]
   float* state; long long slot_stride;                    // slot s at state + s * slot_stride: [heads, dim, vdim]
   const int *state_slots, *cu_tokens;
   int heads, qk_heads, dim, vdim;
   float q_scale, norm_eps;
 };
 
-template <typename T, int R>
+template <typename T, int R, bool CH>
 __global__ void __launch_bounds__(WARPS * 32)
 delta_scan_kernel(DeltaArgs a) {
   extern __shared__ __align__(16) float smem[];
@@ -59,6 +62,8 @@ delta_scan_kernel(DeltaArgs a) {
   float* g_s = o_s + CHUNK * VT;           // [CHUNK] decay, [CHUNK] beta, [CHUNK] k . q
   float* beta_s = g_s + CHUNK;
   float* kq_s = beta_s + CHUNK;
+  float* kd_s = kq_s + CHUNK;              // CH: [CHUNK][DP] the keys as they are (k_s and q_s then hold them times the decays)
+  float* gd_s = kd_s + CHUNK * DP;         // CH: [CHUNK][DP] the decays
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, tid = threadIdx.x;
   const int rl = lane & (ROW_LANES - 1), cl = lane >> 3;
   const int entry = blockIdx.z, head = blockIdx.y;
@@ -68,9 +73,15 @@ delta_scan_kernel(DeltaArgs a) {
   const int col0 = blockIdx.x * VT + wcol;
   const int t0 = a.cu_tokens[entry], t1 = a.cu_tokens[entry + 1];
   if (t0 >= t1) return;
-  const T *q = (const T*)a.q, *k = (const T*)a.k, *v = (const T*)a.v, *pb = (const T*)a.b, *pa = (const T*)a.a;
+  using A = typename std::conditional<CH, float, T>::type;
+  const T *q = (const T*)a.q, *k = (const T*)a.k, *v = (const T*)a.v, *pb = (const T*)a.b;
+  const A* pa = (const A*)a.a;
   float* S_g = a.state + (size_t)a.state_slots[entry] * a.slot_stride + ((size_t)head * dim) * vdim;
-  const float neg_a = -expf(a.a_log[head]), dt_b = a.dt_bias[head];
+  const float neg_a = -expf(a.a_log[head]), dt_b = CH ? 0.f : a.dt_bias[head];
+  float dt_c[CH ? PER : 1];                // CH: the bias of the channels that this lane stages
+  if (CH)
+#pragma unroll
+    for (int i = 0; i < PER; ++i) dt_c[CH ? i : 0] = lane + 32 * i < dim ? a.dt_bias[(size_t)head * dim + lane + 32 * i] : 0.f;
 
   float S[R][COLS];
 #pragma unroll
@@ -84,7 +95,8 @@ delta_scan_kernel(DeltaArgs a) {
   // its warp's tokens (warp, warp + WARPS, ...) of q and k, PER channels a lane; lane j's b and a of the warp's j-th token;
   // and its share of the chunk's values.
   constexpr int TOK = CHUNK / WARPS, VREGS = CHUNK * VT / (WARPS * 32);
-  T q_r[TOK][PER], k_r[TOK][PER], v_r[VREGS], b_r = T(), a_r = T();
+  T q_r[TOK][PER], k_r[TOK][PER], v_r[VREGS], b_r = T();
+  A a_r = A(), z_r[CH ? TOK : 1][CH ? PER : 1];
   auto fetch = [&](int c0) {
     const int n = min(CHUNK, t1 - c0);
 #pragma unroll
@@ -94,12 +106,16 @@ delta_scan_kernel(DeltaArgs a) {
 #pragma unroll
       for (int i = 0; i < PER; ++i) {
         const int d = lane + 32 * i;
-        if (c < n && d < dim) { q_r[j][i] = q[at + d]; k_r[j][i] = k[at + d]; }
+        if (c < n && d < dim) {
+          q_r[j][i] = q[at + d]; k_r[j][i] = k[at + d];
+          if (CH) z_r[CH ? j : 0][CH ? i : 0] = pa[(size_t)(c0 + c) * a.a_stride + (size_t)head * dim + d];
+        }
       }
     }
     if (lane < TOK && warp + lane * WARPS < n) {
-      const size_t ba = (size_t)(c0 + warp + lane * WARPS) * a.ba_stride + head;
-      b_r = pb[ba]; a_r = pa[ba];
+      const size_t t = (size_t)(c0 + warp + lane * WARPS);
+      b_r = pb[t * a.b_stride + head];
+      if (!CH) a_r = pa[t * a.a_stride + head];
     }
 #pragma unroll
     for (int i = 0; i < VREGS; ++i) {
@@ -145,14 +161,21 @@ delta_scan_kernel(DeltaArgs a) {
         for (int i = 0; i < PER; ++i) {
           const int d = lane + 32 * i;
           if (d < ROW_LANES * R) {
-            q_s[c * DP + (d / R) * PITCH + d % R] = qv[j][i] * rq;
-            k_s[c * DP + (d / R) * PITCH + d % R] = kv[j][i] * rk;
+            const int at = c * DP + (d / R) * PITCH + d % R;
+            float g = 1.f;
+            if (CH) {
+              g = d < dim ? expf(neg_a * softplus_d(to_f32(z_r[CH ? j : 0][CH ? i : 0]) + dt_c[CH ? i : 0])) : 0.f;
+              kd_s[at] = kv[j][i] * rk;
+              gd_s[at] = g;
+            }
+            q_s[at] = qv[j][i] * rq * g;
+            k_s[at] = kv[j][i] * rk * g;
           }
         }
         if (lane == j) {
           kq_s[c] = red[j][2] * rq * rk;
           beta_s[c] = 1.f / (1.f + expf(-to_f32(b_r)));
-          g_s[c] = expf(neg_a * softplus_d(to_f32(a_r) + dt_b));
+          if (!CH) g_s[c] = expf(neg_a * softplus_d(to_f32(a_r) + dt_b));
         }
       }
     }
@@ -165,7 +188,7 @@ delta_scan_kernel(DeltaArgs a) {
     if (c0 + CHUNK < t1) fetch(c0 + CHUNK);
 #pragma unroll WALK_UNROLL
     for (int c = 0; c < n; ++c) {
-      const float g = g_s[c], beta = beta_s[c], kq = kq_s[c];
+      const float g = CH ? 1.f : g_s[c], beta = beta_s[c], kq = kq_s[c];      // CH: the decays are in k_s and q_s
       float kd[R];
       float pk[COLS][2], pq[COLS][2];          // two partial sums each: the chains of multiply-adds are half as long
 #pragma unroll
@@ -203,10 +226,23 @@ delta_scan_kernel(DeltaArgs a) {
         u[cc] = beta * (vv[cc] - g * sk[cc]);
         o2[cc] = fmaf(u[cc], kq, g * sq[cc]);
       }
+      if (CH) {
 #pragma unroll
-      for (int i = 0; i < R; ++i)
+        for (int i = 0; i < R; i += 4) {
+          const float4 k4 = *reinterpret_cast<const float4*>(kd_s + c * DP + rl * PITCH + i);
+          const float4 g4 = *reinterpret_cast<const float4*>(gd_s + c * DP + rl * PITCH + i);
+          const float kr[4] = {k4.x, k4.y, k4.z, k4.w}, gr[4] = {g4.x, g4.y, g4.z, g4.w};
 #pragma unroll
-        for (int cc = 0; cc < COLS; ++cc) S[i][cc] = fmaf(kd[i], u[cc], g * S[i][cc]);
+          for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int cc = 0; cc < COLS; ++cc) S[i + j][cc] = fmaf(kr[j], u[cc], gr[j] * S[i + j][cc]);
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < R; ++i)
+#pragma unroll
+          for (int cc = 0; cc < COLS; ++cc) S[i][cc] = fmaf(kd[i], u[cc], g * S[i][cc]);
+      }
       if (rl == 0) *reinterpret_cast<float2*>(o_s + c * VT + wcol) = make_float2(o2[0], o2[1]);
     }
     __syncthreads();
@@ -225,13 +261,21 @@ delta_scan_kernel(DeltaArgs a) {
   }
 }
 
-template <typename T, int R>
+template <typename T, int R, bool CH>
 int launch_delta(const DeltaArgs& a, int n_entries, cudaStream_t stream) {
-  const size_t smem = ((size_t)2 * CHUNK * ROW_LANES * (R + 4) + 2 * CHUNK * VT + 3 * CHUNK) * sizeof(float);
-  if (smem > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<T, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const size_t smem = ((size_t)(CH ? 4 : 2) * CHUNK * ROW_LANES * (R + 4) + 2 * CHUNK * VT + 3 * CHUNK) * sizeof(float);
+  if (smem > 48 * 1024) cudaFuncSetAttribute(delta_scan_kernel<T, R, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   const dim3 grid((a.vdim + VT - 1) / VT, a.heads, n_entries);
-  launch_kernel(delta_scan_kernel<T, R>, grid, dim3(WARPS * 32), smem, stream, a);
+  launch_kernel(delta_scan_kernel<T, R, CH>, grid, dim3(WARPS * 32), smem, stream, a);
   LLMK_LAUNCH_CHECK("delta_scan");
+}
+
+template <typename T, bool CH>
+int launch_delta_of(const DeltaArgs& a, int n_entries, cudaStream_t stream) {
+  if (a.dim <= 32) return launch_delta<T, 4, CH>(a, n_entries, stream);
+  if (a.dim <= 64) return launch_delta<T, 8, CH>(a, n_entries, stream);
+  if (a.dim <= 128) return launch_delta<T, 16, CH>(a, n_entries, stream);
+  return launch_delta<T, 32, CH>(a, n_entries, stream);
 }
 
 // ---- prompts: the rule chunk by chunk ---------------------------------------------------------------------------
@@ -250,18 +294,26 @@ int launch_delta(const DeltaArgs& a, int n_entries, cudaStream_t stream) {
 // tiles of 16 to 32 sums a thread, the state's tile in registers from chunk to chunk and mirrored in shared memory for the
 // products that read all of it.  What is left of the chain from token to token is one step per chunk.  All of it float32;
 // the sums of a token are grouped by where its chunk begins, which moves results by rounding only.
-constexpr int CC = 32;
+//
+// With a decay per key channel (CH) L_t is a vector over the channels and the decays stand inside the Gram matrices,
+//     A_ts = beta_t sum_d exp(L_td - L_sd) k_td k_sd,    B_ts alike with q_t,
+// while Y, the scaled q and k and the end decay take them channel by channel and the walk stays as it is.  exp(L_t) and
+// exp(-L_s) cannot be taken apart (the second overflows), but within reach of a token r between s and t both exp(L_t - L_r) and
+// exp(L_r - L_s) are at most one: the chunk is cut into blocks of CB tokens, the Gram entries of two different blocks are
+// plain products of rows scaled to the last token before the later block, and only those within a block take an exponential
+// for every channel and pair.
+constexpr int CC = 32, CB = 8;
 
 struct PrepArgs {
   const void *q, *k; long long qk_stride;
   const void* v; long long v_stride;
-  const void *b, *a; long long ba_stride;
+  const void *b, *a; long long b_stride, a_stride;
   const float *a_log, *dt_bias;
   const int* cu_tokens; int n_entries;
   int heads, qk_heads, dim, vdim;
   float q_scale, norm_eps;
   // per chunk c and head h, at (c * heads + h) * size: YQ [dim][2 CC] (Y's tokens, then the scaled q's), K [CC][dim],
-  // W [CC][vdim], B [CC][CC], G [1] (the chunk's whole decay)
+  // W [CC][vdim], B [CC][CC], G [1] (the chunk's whole decay; CH: [dim])
   float *YQ, *K, *W, *B, *G;
 };
 
@@ -275,7 +327,7 @@ __device__ __forceinline__ bool chunk_of(const int* cu_tokens, int n_entries, in
   return false;
 }
 
-template <typename T>
+template <typename T, bool CH>
 __global__ void __launch_bounds__(256)
 delta_prepare_kernel(PrepArgs a) {
   extern __shared__ __align__(16) float smem[];
@@ -290,10 +342,14 @@ delta_prepare_kernel(PrepArgs a) {
   float* qn = kn + CC * pitch;             // [CC][dim + 1]
   float* A_s = qn + CC * pitch;            // [CC][CC + 1]
   float* beta_s = A_s + CC * (CC + 1);     // [CC]
-  float* L_s = beta_s + CC;                // [CC]: log g, then its running sum
+  float* L_s = beta_s + CC;                // [CC]: log g, then its running sum; CH: [CC][dim + 1]
+  float* kr_s = L_s + CC * pitch;          // CH: [CC - CB][dim + 1] keys scaled to the token before a block
+  float* xr_s = kr_s + (CC - CB) * pitch;  // CH: [2][CB][dim + 1] the block's k and q scaled from that token
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const T *q = (const T*)a.q, *k = (const T*)a.k, *v = (const T*)a.v, *pb = (const T*)a.b, *pa = (const T*)a.a;
-  const float neg_a = -expf(a.a_log[head]), dt_b = a.dt_bias[head];
+  const T *q = (const T*)a.q, *k = (const T*)a.k, *v = (const T*)a.v, *pb = (const T*)a.b;
+  using A = typename std::conditional<CH, float, T>::type;
+  const A* pa = (const A*)a.a;
+  const float neg_a = -expf(a.a_log[head]), dt_b = CH ? 0.f : a.dt_bias[head];
   // unit q and k, beta and log g: a warp per token
   for (int t = warp; t < CC; t += 8) {
     const size_t at = (size_t)(c0 + t) * a.qk_stride + (size_t)qk_head * dim;
@@ -307,35 +363,102 @@ delta_prepare_kernel(PrepArgs a) {
     for (int d = lane; d < dim; d += 32) {
       qn[t * pitch + d] = t < n ? to_f32(q[at + d]) * rq : 0.f;
       kn[t * pitch + d] = t < n ? to_f32(k[at + d]) * rk : 0.f;
+      if (CH)
+        L_s[t * pitch + d] = t < n ? neg_a * softplus_d(to_f32(pa[(size_t)(c0 + t) * a.a_stride + (size_t)head * dim + d]) +
+                                                        a.dt_bias[(size_t)head * dim + d]) : 0.f;
     }
     if (lane == 0) {
-      const size_t ba = (size_t)(c0 + t) * a.ba_stride + head;
-      beta_s[t] = t < n ? 1.f / (1.f + expf(-to_f32(pb[ba]))) : 0.f;
-      L_s[t] = t < n ? neg_a * softplus_d(to_f32(pa[ba]) + dt_b) : 0.f;      // log g: the decay without its exponential
+      beta_s[t] = t < n ? 1.f / (1.f + expf(-to_f32(pb[(size_t)(c0 + t) * a.b_stride + head]))) : 0.f;
+      if (!CH) L_s[t] = t < n ? neg_a * softplus_d(to_f32(pa[(size_t)(c0 + t) * a.a_stride + head]) + dt_b) : 0.f;      // log g: the decay without its exponential
     }
   }
   __syncthreads();
-  if (tid == 0) {
+  if (CH) {
+    for (int d = tid; d < dim; d += 256) {
+      float run = 0.f;
+      for (int t = 0; t < CC; ++t) { run += L_s[t * pitch + d]; L_s[t * pitch + d] = run; }
+    }
+  } else if (tid == 0) {
     float run = 0.f;
     for (int t = 0; t < CC; ++t) { run += L_s[t]; L_s[t] = run; }
   }
   __syncthreads();
-  // the two Gram matrices with their decays
-  for (int idx = tid; idx < CC * CC; idx += 256) {
-    const int t = idx / CC, s2 = idx % CC;
-    float kk = 0.f, qk = 0.f;
-    if (s2 <= t && t < n) {
-      for (int d = 0; d < dim; ++d) {
-        const float ks = kn[s2 * pitch + d];
-        kk = fmaf(kn[t * pitch + d], ks, kk);
-        qk = fmaf(qn[t * pitch + d], ks, qk);
-      }
-      const float e = expf(L_s[t] - L_s[s2]);
-      kk *= e * beta_s[t];
-      qk *= e;
+  if (CH) {
+    for (int idx = tid; idx < CC * CC; idx += 256) {          // beyond the diagonal
+      const int t = idx / CC, s2 = idx % CC;
+      if (s2 > t) { A_s[t * (CC + 1) + s2] = 0.f; a.B[unit * CC * CC + idx] = 0.f; }
     }
-    A_s[t * (CC + 1) + s2] = s2 < t ? kk : 0.f;
-    a.B[unit * CC * CC + idx] = (s2 <= t && t < n) ? qk : 0.f;
+    // pairs within a block: four threads a pair, an exponential for every channel
+    constexpr int PAIRS = CB * (CB + 1) / 2;
+    for (int w = tid / 4; w < CC / CB * PAIRS; w += 64) {
+      const int blk = w / PAIRS;
+      int i = 0, left = w % PAIRS;
+      while (left > i) { left -= i + 1; ++i; }                // the pair (i, left), left <= i, of the block's lower triangle
+      const int t = blk * CB + i, s2 = blk * CB + left;
+      float kk = 0.f, qk = 0.f;
+      for (int d = tid % 4; d < dim; d += 4) {
+        const float x = expf(L_s[t * pitch + d] - L_s[s2 * pitch + d]) * kn[s2 * pitch + d];
+        kk = fmaf(kn[t * pitch + d], x, kk);
+        qk = fmaf(qn[t * pitch + d], x, qk);
+      }
+      static_assert(CC / CB * PAIRS % 8 == 0, "a warp's eight pairs are all there or none");
+      kk += __shfl_xor_sync(0xffffffffu, kk, 1); kk += __shfl_xor_sync(0xffffffffu, kk, 2);
+      qk += __shfl_xor_sync(0xffffffffu, qk, 1); qk += __shfl_xor_sync(0xffffffffu, qk, 2);
+      if (tid % 4 == 0) {
+        A_s[t * (CC + 1) + s2] = s2 < t ? kk * beta_s[t] : 0.f;
+        a.B[unit * CC * CC + t * CC + s2] = t < n ? qk : 0.f;
+      }
+    }
+    // pairs of two blocks, one later block at a time
+    for (int t0 = CB; t0 < CC && t0 < n; t0 += CB) {
+      const float* ref = L_s + (t0 - 1) * pitch;
+      for (int idx = tid; idx < t0 * dim; idx += 256) {
+        const int s2 = idx / dim, d = idx % dim;
+        kr_s[s2 * pitch + d] = expf(ref[d] - L_s[s2 * pitch + d]) * kn[s2 * pitch + d];
+      }
+      for (int idx = tid; idx < CB * dim; idx += 256) {
+        const int i = idx / dim, d = idx % dim;
+        const float e = expf(L_s[(t0 + i) * pitch + d] - ref[d]);
+        xr_s[i * pitch + d] = e * kn[(t0 + i) * pitch + d];
+        xr_s[(CB + i) * pitch + d] = e * qn[(t0 + i) * pitch + d];
+      }
+      __syncthreads();
+      for (int idx = tid; idx < CB * t0; idx += 256) {
+        const int i = idx % CB, s2 = idx / CB, t = t0 + i;
+        float kk = 0.f, qk = 0.f;
+        for (int d = 0; d < dim; ++d) {
+          const float x = kr_s[s2 * pitch + d];
+          kk = fmaf(xr_s[i * pitch + d], x, kk);
+          qk = fmaf(xr_s[(CB + i) * pitch + d], x, qk);
+        }
+        A_s[t * (CC + 1) + s2] = kk * beta_s[t];
+        a.B[unit * CC * CC + t * CC + s2] = t < n ? qk : 0.f;
+      }
+      __syncthreads();
+    }
+    // blocks behind the chunk's last token
+    for (int idx = tid; idx < CC * CC; idx += 256) {
+      const int t = idx / CC, s2 = idx % CC;
+      if (t / CB * CB >= n && t >= CB && s2 < t / CB * CB) { A_s[t * (CC + 1) + s2] = 0.f; a.B[unit * CC * CC + idx] = 0.f; }
+    }
+  } else {
+    // the two Gram matrices with their decays
+    for (int idx = tid; idx < CC * CC; idx += 256) {
+      const int t = idx / CC, s2 = idx % CC;
+      float kk = 0.f, qk = 0.f;
+      if (s2 <= t && t < n) {
+        for (int d = 0; d < dim; ++d) {
+          const float ks = kn[s2 * pitch + d];
+          kk = fmaf(kn[t * pitch + d], ks, kk);
+          qk = fmaf(qn[t * pitch + d], ks, qk);
+        }
+        const float e = expf(L_s[t] - L_s[s2]);
+        kk *= e * beta_s[t];
+        qk *= e;
+      }
+      A_s[t * (CC + 1) + s2] = s2 < t ? kk : 0.f;
+      a.B[unit * CC * CC + idx] = (s2 <= t && t < n) ? qk : 0.f;
+    }
   }
   __syncthreads();
   // forward substitution: a thread per column of [beta V | beta exp(L) K], the column in registers
@@ -348,7 +471,7 @@ delta_prepare_kernel(PrepArgs a) {
       float r = 0.f;
       if (t < n)
         r = is_v ? beta_s[t] * to_f32(v[(size_t)(c0 + t) * a.v_stride + (size_t)head * vdim + col])
-                 : beta_s[t] * expf(L_s[t]) * kn[t * pitch + d];
+                 : beta_s[t] * expf(CH ? L_s[t * pitch + d] : L_s[t]) * kn[t * pitch + d];
       x[t] = r;
     }
 #pragma unroll
@@ -368,16 +491,19 @@ delta_prepare_kernel(PrepArgs a) {
     }
   }
   // q and k with the decays that the walk needs: to the token from the chunk's start, from the token to the chunk's end
-  const float L_end = L_s[n - 1];
   for (int idx = tid; idx < CC * dim; idx += 256) {
     const int t = idx % CC, d = idx / CC;
-    a.YQ[(unit * dim + d) * (2 * CC) + CC + t] = t < n ? expf(L_s[t]) * qn[t * pitch + d] : 0.f;
+    a.YQ[(unit * dim + d) * (2 * CC) + CC + t] = t < n ? expf(CH ? L_s[t * pitch + d] : L_s[t]) * qn[t * pitch + d] : 0.f;
   }
   for (int idx = tid; idx < CC * dim; idx += 256) {
     const int t = idx / dim, d = idx % dim;
-    a.K[(unit * CC + t) * dim + d] = t < n ? expf(L_end - L_s[t]) * kn[t * pitch + d] : 0.f;
+    const float rest = CH ? L_s[(n - 1) * pitch + d] - L_s[t * pitch + d] : L_s[n - 1] - L_s[t];
+    a.K[(unit * CC + t) * dim + d] = t < n ? expf(rest) * kn[t * pitch + d] : 0.f;
   }
-  if (tid == 0) a.G[unit] = expf(L_end);
+  if (CH)
+    for (int d = tid; d < dim; d += 256) a.G[unit * dim + d] = expf(L_s[(n - 1) * pitch + d]);
+  else if (tid == 0)
+    a.G[unit] = expf(L_s[n - 1]);
 }
 
 struct WalkArgs {
@@ -401,7 +527,7 @@ static_assert(2 * CC % TYN == 0 && CC % TYN == 0, "rows of the products divide a
 
 // RT: rows of the state a thread keeps (a head's rows / 32, rounded up to 1, 2, 4 or 8).  STAGES chunks of operands lie in
 // shared memory (2: the next chunk's copies run under this chunk's arithmetic; 1 where two do not fit).
-template <int RT, int STAGES>
+template <int RT, int STAGES, bool CH>
 __global__ void __launch_bounds__(WT)
 delta_chunk_walk_kernel(WalkArgs a) {
   extern __shared__ __align__(16) float smem[];
@@ -465,7 +591,14 @@ delta_chunk_walk_kernel(WalkArgs a) {
   int at_stage = 0;
   for (int c0 = t0; c0 < t1; c0 += CC, ++chunk) {
     const int n = min(CC, t1 - c0);
-    const float g_end = a.G[(size_t)chunk * a.heads + head];
+    float g_end[CH ? RT : 1];
+    if (CH) {
+#pragma unroll
+      for (int i = 0; i < RT; ++i)
+        g_end[CH ? i : 0] = ty * RT + i < dim ? a.G[((size_t)chunk * a.heads + head) * dim + ty * RT + i] : 0.f;
+    } else {
+      g_end[0] = a.G[(size_t)chunk * a.heads + head];
+    }
     const float* st = smem + at_stage * STAGE;
     const float *yq_s = st, *k_s = st + DPAD * 2 * CC, *w_s = k_s + CC * DPAD, *b_s = w_s + CC * WV;
     const bool more = c0 + CC < t1;
@@ -556,7 +689,7 @@ delta_chunk_walk_kernel(WalkArgs a) {
 #pragma unroll
     for (int i = 0; i < RT; ++i)
 #pragma unroll
-      for (int c = 0; c < 4; ++c) S[i][c] *= g_end;
+      for (int c = 0; c < 4; ++c) S[i][c] *= g_end[CH ? i : 0];
     {
       float4 ua, ub;
       float ka[RT], kb[RT];
@@ -609,72 +742,75 @@ delta_chunk_walk_kernel(WalkArgs a) {
   }
 }
 
-template <int RT>
+template <int RT, bool CH>
 int launch_walk(const WalkArgs& a, int n_entries, cudaStream_t stream) {
   constexpr int STAGES = RT <= 4 ? 2 : 1;      // two stages of a head of 256 rows exceed an SM's shared memory
   constexpr int DPAD = TYN * RT;
   const size_t stage = (size_t)DPAD * 2 * CC + CC * DPAD + CC * WV + CC * (CC + 4);
   const size_t smem = (STAGES * stage + DPAD * WV + 2 * CC * WV) * sizeof(float);
   if (smem > 48 * 1024)
-    cudaFuncSetAttribute(delta_chunk_walk_kernel<RT, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  launch_kernel(delta_chunk_walk_kernel<RT, STAGES>, dim3((a.vdim + WV - 1) / WV, a.heads, n_entries), dim3(WT), smem, stream, a);
+    cudaFuncSetAttribute(delta_chunk_walk_kernel<RT, STAGES, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  launch_kernel(delta_chunk_walk_kernel<RT, STAGES, CH>, dim3((a.vdim + WV - 1) / WV, a.heads, n_entries), dim3(WT), smem, stream, a);
   LLMK_LAUNCH_CHECK("delta_chunk_walk");
+}
+
+template <bool CH>
+int launch_chunks(const PrepArgs& p, WalkArgs w, int n_tokens, int dtype, cudaStream_t stream) {
+  const int chunks = n_tokens / CC + p.n_entries;
+  const size_t own = CH ? (size_t)(CC + CC - CB + 2 * CB) * (p.dim + 1) : (size_t)CC;
+  const size_t smem = ((size_t)2 * CC * (p.dim + 1) + CC * (CC + 1) + CC + own) * sizeof(float);
+  int rc = dispatch_dtype(dtype, [&](auto* tag) {
+    using T = LLMK_ELEM(tag);
+    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prepare_kernel<T, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_kernel(delta_prepare_kernel<T, CH>, dim3(chunks, p.heads), dim3(256), smem, stream, p);
+    LLMK_LAUNCH_CHECK("delta_prepare");
+  });
+  if (rc) return rc;
+  if (p.dim <= 32) return launch_walk<1, CH>(w, p.n_entries, stream);
+  if (p.dim <= 64) return launch_walk<2, CH>(w, p.n_entries, stream);
+  if (p.dim <= 128) return launch_walk<4, CH>(w, p.n_entries, stream);
+  return launch_walk<8, CH>(w, p.n_entries, stream);
 }
 
 }  // namespace
 
-// q, k [T, qk_heads * dim] (one row stride), v [T, heads * vdim], b and a [T, heads] (one row stride), all in the
-// projections' kind; a_log, dt_bias float32 [heads]; state float32, slot s at state + s * slot_stride holding
-// [heads, dim, vdim]; out float32 [T, heads * vdim].  q is scaled by q_scale after its unit norm; norm_eps is added to the
-// sums of squares.
+// q, k [T, qk_heads * dim] (one row stride), v [T, heads * vdim] and b [T, heads] in the projections' kind; per_channel 0: a
+// [T, heads] of the same kind, dt_bias float32 [heads]; else a float32 [T, heads * dim], dt_bias [heads * dim]; a_log float32
+// [heads]; state float32, slot s at state + s * slot_stride holding [heads, dim, vdim]; out float32 [T, heads * vdim].  q is
+// scaled by q_scale after its unit norm; norm_eps is added to the sums of squares.
 LLMK_API int llmk_delta_scan(float* out, long long out_stride, const void* q, const void* k, long long qk_stride, const void* v,
-                             long long v_stride, const void* b, const void* a, long long ba_stride, const float* a_log,
-                             const float* dt_bias, float* state, long long slot_stride, const int* state_slots,
+                             long long v_stride, const void* b, long long b_stride, const void* a, long long a_stride,
+                             const float* a_log, const float* dt_bias, float* state, long long slot_stride, const int* state_slots,
                              const int* cu_tokens, int n_entries, int heads, int qk_heads, int dim, int vdim, float q_scale,
-                             float norm_eps, int dtype, cudaStream_t stream) {
+                             float norm_eps, int per_channel, int dtype, cudaStream_t stream) {
   if (n_entries == 0) return 0;
   LLMK_REQUIRE(dim > 0 && dim <= 256, "delta_scan: key size %d (1 to 256)", dim);
   LLMK_REQUIRE(qk_heads > 0 && heads % qk_heads == 0 && vdim > 0, "delta_scan: %d heads do not divide into %d key heads", heads, qk_heads);
   LLMK_REQUIRE(n_entries <= 65535 && heads <= 65535, "delta_scan: too many entries or heads for one launch");
-  DeltaArgs args = {out, out_stride, q, k, qk_stride, v, v_stride, b, a, ba_stride, a_log, dt_bias, state, slot_stride,
+  DeltaArgs args = {out, out_stride, q, k, qk_stride, v, v_stride, b, a, b_stride, a_stride, a_log, dt_bias, state, slot_stride,
                     state_slots, cu_tokens, heads, qk_heads, dim, vdim, q_scale, norm_eps};
   return dispatch_dtype(dtype, [&](auto* tag) {
     using T = LLMK_ELEM(tag);
-    if (dim <= 32) return launch_delta<T, 4>(args, n_entries, stream);
-    if (dim <= 64) return launch_delta<T, 8>(args, n_entries, stream);
-    if (dim <= 128) return launch_delta<T, 16>(args, n_entries, stream);
-    return launch_delta<T, 32>(args, n_entries, stream);
+    return per_channel ? launch_delta_of<T, true>(args, n_entries, stream) : launch_delta_of<T, false>(args, n_entries, stream);
   });
 }
 
 // The same rule for a step with prompt portions, chunk by chunk (see delta_prepare_kernel).  n_tokens: the step's tokens.
 // Float32 scratch for n_tokens / 32 + n_entries chunks of every head: YQ (dim * 64 floats a chunk and head), K (32 * dim),
-// W (32 * vdim), B (32 * 32), G (1).
+// W (32 * vdim), B (32 * 32), G (1; per_channel: dim).
 LLMK_API int llmk_delta_chunk_scan(float* out, long long out_stride, const void* q, const void* k, long long qk_stride,
-                                   const void* v, long long v_stride, const void* b, const void* a, long long ba_stride,
-                                   const float* a_log, const float* dt_bias, float* state, long long slot_stride,
+                                   const void* v, long long v_stride, const void* b, long long b_stride, const void* a,
+                                   long long a_stride, const float* a_log, const float* dt_bias, float* state, long long slot_stride,
                                    const int* state_slots, const int* cu_tokens, int n_entries, int n_tokens, int heads,
-                                   int qk_heads, int dim, int vdim, float q_scale, float norm_eps, float* YQ, float* K, float* W,
-                                   float* B, float* G, int dtype, cudaStream_t stream) {
+                                   int qk_heads, int dim, int vdim, float q_scale, float norm_eps, int per_channel, float* YQ, float* K,
+                                   float* W, float* B, float* G, int dtype, cudaStream_t stream) {
   if (n_entries == 0 || n_tokens == 0) return 0;
   LLMK_REQUIRE(dim > 0 && dim <= 256, "delta_chunk_scan: key size %d (1 to 256)", dim);
   LLMK_REQUIRE(qk_heads > 0 && heads % qk_heads == 0 && vdim > 0, "delta_chunk_scan: %d heads do not divide into %d key heads", heads, qk_heads);
   LLMK_REQUIRE(n_entries <= 65535 && heads <= 65535, "delta_chunk_scan: too many entries or heads for one launch");
   LLMK_REQUIRE(YQ && K && W && B && G, "delta_chunk_scan: the scratch is missing");
-  PrepArgs p = {q, k, qk_stride, v, v_stride, b, a, ba_stride, a_log, dt_bias, cu_tokens, n_entries, heads, qk_heads, dim, vdim,
-                q_scale, norm_eps, YQ, K, W, B, G};
-  const int chunks = n_tokens / CC + n_entries;
-  const size_t smem = ((size_t)2 * CC * (dim + 1) + CC * (CC + 1) + 2 * CC) * sizeof(float);
-  int rc = dispatch_dtype(dtype, [&](auto* tag) {
-    using T = LLMK_ELEM(tag);
-    if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_kernel(delta_prepare_kernel<T>, dim3(chunks, heads), dim3(256), smem, stream, p);
-    LLMK_LAUNCH_CHECK("delta_prepare");
-  });
-  if (rc) return rc;
-  WalkArgs w = {out, out_stride, YQ, K, W, B, G, state, slot_stride, state_slots, cu_tokens, heads, dim, vdim};
-  if (dim <= 32) return launch_walk<1>(w, n_entries, stream);
-  if (dim <= 64) return launch_walk<2>(w, n_entries, stream);
-  if (dim <= 128) return launch_walk<4>(w, n_entries, stream);
-  return launch_walk<8>(w, n_entries, stream);
+  const PrepArgs p = {q, k, qk_stride, v, v_stride, b, a, b_stride, a_stride, a_log, dt_bias, cu_tokens, n_entries, heads, qk_heads, dim,
+                      vdim, q_scale, norm_eps, YQ, K, W, B, G};
+  const WalkArgs w = {out, out_stride, YQ, K, W, B, G, state, slot_stride, state_slots, cu_tokens, heads, dim, vdim};
+  return per_channel ? launch_chunks<true>(p, w, n_tokens, dtype, stream) : launch_chunks<false>(p, w, n_tokens, dtype, stream);
 }

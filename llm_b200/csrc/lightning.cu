@@ -16,7 +16,7 @@
 // every float32 operand of a product (the state, the decayed scores, the decayed values) enters it as the sum of three bfloat16
 // numbers, which hold its 24 bits, and every sum is float32.  The products are warp-level MMAs (mma.sync): their operands are
 // made in registers by the warp that uses them, and a tile is 64 rows.
-#include "common.cuh"
+#include "warp_mma.cuh"
 
 namespace {
 
@@ -105,43 +105,6 @@ __device__ __forceinline__ bool chunk_of(const int* cu_tokens, int n_entries, in
   return false;
 }
 
-__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void cp_async16(void* smem_dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(smem_dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory"); }
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
-}
-__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
-}
-__device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// Two float32 numbers as three pairs of bfloat16 numbers whose sums they are (to the last of their 24 bits or so).
-__device__ __forceinline__ void split3(float x, float y, uint32_t (&p)[3]) {
-#pragma unroll
-  for (int i = 0; i < 3; ++i) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-    p[i] = *reinterpret_cast<const uint32_t*>(&h);
-    x -= __low2float(h); y -= __high2float(h);
-  }
-}
-
-// rows [0, n) of a [.., cols] tensor into shared memory with pitch `pitch`, zeros in rows n .. CC and columns up to `cols_pad`
-// (cols a multiple of 8, cols_pad of 8)
-__device__ __forceinline__ void bring_rows(bf16* dst, int pitch, const bf16* src, long long stride, int n, int cols, int cols_pad) {
-  const int per = cols_pad / 8;
-  for (int i = threadIdx.x; i < CC * per; i += THREADS) {
-    const int r = i / per, c = (i % per) * 8;
-    bf16* at = dst + r * pitch + c;
-    if (r < n && c < cols) cp_async16(at, src + (size_t)r * stride + c);
-    else *reinterpret_cast<uint4*>(at) = make_uint4(0, 0, 0, 0);
-  }
-}
-
 // seg[chunk, head] [dim, vdim] = sum_j d^(n-1-j) k_j v_j^T.  Grid (chunks, heads, value tiles).
 __global__ void __launch_bounds__(THREADS)
 lightning_chunk_state_kernel(const bf16* __restrict__ k, const bf16* __restrict__ v, long long stride, const float* __restrict__ decay,
@@ -155,7 +118,7 @@ lightning_chunk_state_kernel(const bf16* __restrict__ k, const bf16* __restrict_
   const int head = blockIdx.y, col0 = blockIdx.z * VT, kp = dim + PAD;
   bf16* k_s = reinterpret_cast<bf16*>(smem_raw);          // [CC][dim + PAD]
   bf16* v_s = k_s + CC * kp;                              // [3][CC][VP]: the decayed values in three pieces
-  bring_rows(k_s, kp, k + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
+  bring_rows<CC, THREADS>(k_s, kp, k + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
   // a thread's eight-column pieces of the values: requested first, scaled and split when the powers of the decay are there
   constexpr int PIECES = CC * (VT / 8) / THREADS;
   const bf16* src = v + (size_t)c0 * stride + (size_t)head * vdim + col0;
@@ -299,9 +262,9 @@ lightning_chunk_out_kernel(float* __restrict__ out, long long out_stride, const 
     }
   };
   fetch(0);
-  bring_rows(q_s, kp, q + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
-  bring_rows(k_s, kp, k + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
-  bring_rows(v_s, VP, v + (size_t)c0 * stride + (size_t)head * vdim + col0, stride, n, min(VT, vdim - col0), VT);
+  bring_rows<CC, THREADS>(q_s, kp, q + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
+  bring_rows<CC, THREADS>(k_s, kp, k + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
+  bring_rows<CC, THREADS>(v_s, VP, v + (size_t)c0 * stride + (size_t)head * vdim + col0, stride, n, min(VT, vdim - col0), VT);
   if (threadIdx.x <= CC) pw[threadIdx.x] = powf(decay[head], (float)threadIdx.x);
   for (int i0 = 0; i0 < dim * (VT / 8); i0 += BATCH * THREADS) {
     if (i0) fetch(i0);

@@ -35,6 +35,13 @@ class PartialSum:
         return self.rows * self.cols
 
 
+class BiasedRows:
+    """Rows (a tensor or a PartialSum) to which `bias` (float32 [cols]) is still to be added by the kernel that reads them."""
+
+    def __init__(self, rows, bias: torch.Tensor):
+        self.rows, self.bias = rows, bias
+
+
 class WeightedRows:
     """The result of a routed feed-forward before its last sum: row t is sum_j weights[t, j] * y[pair_slot[t, j]] for y
     float32 [slots, cols] (a slot of -1 counts nothing).  The norm behind the residual sum takes it as it is (sum_rmsnorm);
@@ -240,6 +247,29 @@ def add_layernorm(resid: torch.Tensor, delta, post, mult: float, pre, out, rows:
                                      c_int(rows), c_int(hidden), c_float(eps), c_int(_kind(ref.dtype)), _stream()))
 
 
+def add_rmsnorms(resid: torch.Tensor, delta, post, mult: float, pre, out, rows: int, eps: float, delta_bias=None) -> None:
+    """RMS norms on both sides of the residual sum: resid[:rows] += mult * rms(delta + delta_bias) * post where delta (a tensor
+    or a PartialSum) is given (post None: mult * delta); out[:rows] = rms(resid) * pre where out is given.  delta_bias: float32
+    [hidden] or None."""
+    assert resid.dtype == torch.float32 and resid.is_contiguous()
+    hidden = resid.shape[-1]
+    ref = out if out is not None else delta
+    if ref is None:
+        return
+    for w in (post, pre, delta_bias):
+        assert w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == hidden)
+    if isinstance(delta, PartialSum):
+        assert delta.cols == hidden and delta.rows == rows
+    elif delta is not None:
+        assert delta.is_contiguous() and delta.shape[-1] == hidden
+    if out is not None:
+        assert pre is not None and out.is_contiguous() and out.shape[-1] == hidden
+        assert delta is None or delta.dtype == out.dtype
+    d, parts, splits, stride = _split_args(delta)
+    _check(load().llmk_add_rmsnorms(_ptr(resid), d, parts, splits, stride, _ptr(delta_bias), _ptr(post), c_float(mult), _ptr(pre),
+                                    _ptr(out), c_int(rows), c_int(hidden), c_float(eps), c_int(_kind(ref.dtype)), _stream()))
+
+
 def softcap(x: torch.Tensor, rows: int, cap: float) -> None:
     """x[:rows] = cap * tanh(x / cap), float32 in place."""
     assert x.dtype == torch.float32 and x.is_contiguous()
@@ -266,6 +296,27 @@ def head_rmsnorm_gate(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, gate,
         assert gate.dtype == out.dtype and gate.shape[1] == x.shape[-1]
     _check(load().llmk_head_rmsnorm_gate(_ptr(out), _ptr(x), _ptr(w), _ptr(gate), c_longlong(gate.stride(0) if gate is not None else 0),
                                          c_int(rows), c_int(heads), c_int(n), c_float(eps), c_int(_kind(out.dtype)), _stream()))
+
+
+def head_rmsnorm_sigmoid(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, gate, gate_col: int, rows: int, heads: int,
+                         eps: float) -> None:
+    """out[t, h] = x[t, h] / sqrt(mean(x[t, h]^2) + eps) * w * sigmoid(gate[t, gate_col + h*n ..]) per head of x float32
+    [rows, heads * n]; w float32 [n], shared by the heads, or [heads * n]; gate a tensor (unit column stride) or a PartialSum, of
+    out's dtype or float32."""
+    n = x.shape[-1] // heads
+    assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and out.shape[-1] == x.shape[-1] == n * heads
+    assert w.dtype == torch.float32 and w.is_contiguous() and w.numel() in (n, n * heads)
+    if isinstance(gate, PartialSum):
+        assert gate.cols >= gate_col + n * heads and gate.rows == rows
+        gate_stride = gate.cols
+    else:
+        _rows_contig(gate, "gate")
+        assert gate.shape[1] >= gate_col + n * heads
+        gate_stride = gate.stride(0)
+    d, parts, splits, stride = _split_args(gate)
+    _check(load().llmk_head_rmsnorm_sigmoid(_ptr(out), _ptr(x), _ptr(w), c_int(int(w.numel() != n)), d, parts, splits, stride,
+                                            c_longlong(gate_stride), c_longlong(gate_col), c_int(rows), c_int(heads), c_int(n),
+                                            c_float(eps), c_int(_kind(out.dtype)), c_int(_kind(gate.dtype)), _stream()))
 
 
 def rope_pairs_kv_write(qkv, freqs, positions: torch.Tensor, slot_map, k_pages, v_pages, n_tokens: int, n_heads: int,
@@ -347,6 +398,19 @@ def act_rows(out: torch.Tensor, x, rows: int, kind: str) -> None:
     d, parts, splits, stride = _split_args(x)
     _check(load().llmk_act_rows(_ptr(out), d, parts, splits, stride, c_longlong(rows * cols), c_int(ACTIVATIONS[kind]),
                                 c_int(_kind(out.dtype)), _stream()))
+
+
+def bias_act_rows(out: torch.Tensor, x, bias: torch.Tensor, rows: int, kind: str) -> None:
+    """out[:rows] = act(x + bias), bias float32 [cols]; x a tensor or a PartialSum (then float32 until the activation)."""
+    cols = out.shape[-1]
+    assert out.is_contiguous() and bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == cols
+    if isinstance(x, PartialSum):
+        assert x.cols == cols and x.rows == rows
+    else:
+        assert x.is_contiguous() and x.shape[-1] == cols and x.dtype == out.dtype
+    d, parts, splits, stride = _split_args(x)
+    _check(load().llmk_bias_act_rows(_ptr(out), d, parts, splits, stride, _ptr(bias), c_int(rows), c_int(cols),
+                                     c_int(ACTIVATIONS[kind]), c_int(_kind(out.dtype)), _stream()))
 
 
 HEADS_ON_TENSOR_CORES = True
@@ -697,57 +761,144 @@ def lightning_chunks(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: tor
     count_launches(2)
 
 
+def _delta_operands(out, q, k, v, b, a, a_log, dt_bias, state, heads: int, qk_heads: int, dim: int, vdim: int, per_channel: bool) -> None:
+    for t in (out, q, k, v, b, a, state):
+        _rows_contig(t, "delta rule operand")
+    assert q.stride(0) == k.stride(0) and q.dtype == k.dtype == v.dtype == b.dtype
+    assert q.shape[1] == k.shape[1] == qk_heads * dim and v.shape[1] == out.shape[1] == heads * vdim
+    per = dim if per_channel else 1
+    assert b.shape[1] == heads and a.shape[1] == heads * per and a.dtype == (torch.float32 if per_channel else b.dtype)
+    assert out.dtype == state.dtype == torch.float32 and state.shape[1] >= heads * dim * vdim
+    for t, n in ((a_log, heads), (dt_bias, heads * per)):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n
+
+
 def delta_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b: torch.Tensor, a: torch.Tensor,
                a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, ctx, heads: int, qk_heads: int, dim: int,
-               vdim: int, q_scale: float, norm_eps: float = 1e-6) -> None:
+               vdim: int, q_scale: float, norm_eps: float = 1e-6, per_channel: bool = False) -> None:
     """The gated delta rule (delta.cu): S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q per head, with q and k
     made unit vectors per head (q also times q_scale), beta = sigmoid(b), g = exp(-exp(a_log) softplus(a + dt_bias)).
-    q, k [T, qk_heads*dim] (equal row strides), v [T, heads*vdim], b, a [T, heads] (equal row strides), all in the compute
-    dtype; a_log, dt_bias float32 [heads]; state float32 [slots, >= heads*dim*vdim]; out float32 [T, heads*vdim]."""
-    for t in (out, q, k, v, b, a, state):
-        _rows_contig(t, "delta_scan operand")
-    assert q.stride(0) == k.stride(0) and b.stride(0) == a.stride(0) and q.dtype == k.dtype == v.dtype == b.dtype == a.dtype
-    assert q.shape[1] == k.shape[1] == qk_heads * dim and v.shape[1] == out.shape[1] == heads * vdim
-    assert b.shape[1] == a.shape[1] == heads and out.dtype == state.dtype == torch.float32 and state.shape[1] >= heads * dim * vdim
-    for t in (a_log, dt_bias):
-        assert t.dtype == torch.float32 and t.is_contiguous() and t.numel() == heads
+    q, k [T, qk_heads*dim] (equal row strides), v [T, heads*vdim], b, a [T, heads], all in the compute dtype; a_log, dt_bias
+    float32 [heads]; state float32 [slots, >= heads*dim*vdim]; out float32 [T, heads*vdim].  per_channel: a decay per key
+    channel, a float32 [T, heads*dim] and dt_bias [heads*dim]; g then scales the rows of S."""
+    _delta_operands(out, q, k, v, b, a, a_log, dt_bias, state, heads, qk_heads, dim, vdim, per_channel)
     _check(load().llmk_delta_scan(_ptr(out), c_longlong(out.stride(0)), _ptr(q), _ptr(k), c_longlong(q.stride(0)), _ptr(v),
-                                  c_longlong(v.stride(0)), _ptr(b), _ptr(a), c_longlong(b.stride(0)), _ptr(a_log), _ptr(dt_bias),
-                                  _ptr(state), c_longlong(state.stride(0)), _ptr(ctx.state_slots), _ptr(ctx.cu_tokens),
-                                  c_int(ctx.n_entries), c_int(heads), c_int(qk_heads), c_int(dim), c_int(vdim), c_float(q_scale),
-                                  c_float(norm_eps), c_int(_kind(q.dtype)), _stream()))
+                                  c_longlong(v.stride(0)), _ptr(b), c_longlong(b.stride(0)), _ptr(a), c_longlong(a.stride(0)),
+                                  _ptr(a_log), _ptr(dt_bias), _ptr(state), c_longlong(state.stride(0)), _ptr(ctx.state_slots),
+                                  _ptr(ctx.cu_tokens), c_int(ctx.n_entries), c_int(heads), c_int(qk_heads), c_int(dim), c_int(vdim),
+                                  c_float(q_scale), c_float(norm_eps), c_int(int(per_channel)), c_int(_kind(q.dtype)), _stream()))
 
 
 DELTA_CHUNK = 32       # tokens that the chunk-wise delta rule solves together (delta.cu)
 
 
-def delta_chunk_scratch(n_chunks: int, heads: int, dim: int, vdim: int):
+def delta_chunk_scratch(n_chunks: int, heads: int, dim: int, vdim: int, per_channel: bool = False):
     """Float32 element counts of the chunk-wise delta rule's five scratch buffers for n_chunks chunks."""
     c = DELTA_CHUNK
-    return [n_chunks * heads * n for n in (dim * 2 * c, c * dim, c * vdim, c * c, 1)]
+    return [n_chunks * heads * n for n in (dim * 2 * c, c * dim, c * vdim, c * c, dim if per_channel else 1)]
 
 
 def delta_chunk_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b: torch.Tensor, a: torch.Tensor,
                      a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, ctx, heads: int, qk_heads: int, dim: int,
-                     vdim: int, q_scale: float, norm_eps: float, scratch) -> None:
+                     vdim: int, q_scale: float, norm_eps: float, scratch, per_channel: bool = False) -> None:
     """delta_scan for a step with prompt portions: the rule chunk by chunk (32 tokens solved together, chunks chained through
     the state; see delta.cu).  scratch: five flat float32 tensors of at least delta_chunk_scratch(ctx.n_tokens // 32 +
     ctx.n_entries, ...) elements."""
-    for t in (out, q, k, v, b, a, state):
-        _rows_contig(t, "delta_chunk_scan operand")
-    assert q.stride(0) == k.stride(0) and b.stride(0) == a.stride(0) and q.dtype == k.dtype == v.dtype == b.dtype == a.dtype
-    assert q.shape[1] == k.shape[1] == qk_heads * dim and v.shape[1] == out.shape[1] == heads * vdim
-    assert b.shape[1] == a.shape[1] == heads and out.dtype == state.dtype == torch.float32 and state.shape[1] >= heads * dim * vdim
+    _delta_operands(out, q, k, v, b, a, a_log, dt_bias, state, heads, qk_heads, dim, vdim, per_channel)
     T = ctx.n_tokens
-    for t, numel in zip(scratch, delta_chunk_scratch(T // DELTA_CHUNK + ctx.n_entries, heads, dim, vdim)):
+    for t, numel in zip(scratch, delta_chunk_scratch(T // DELTA_CHUNK + ctx.n_entries, heads, dim, vdim, per_channel)):
         assert t.dtype == torch.float32 and t.is_contiguous() and t.numel() >= numel
     _check(load().llmk_delta_chunk_scan(_ptr(out), c_longlong(out.stride(0)), _ptr(q), _ptr(k), c_longlong(q.stride(0)), _ptr(v),
-                                        c_longlong(v.stride(0)), _ptr(b), _ptr(a), c_longlong(b.stride(0)), _ptr(a_log),
-                                        _ptr(dt_bias), _ptr(state), c_longlong(state.stride(0)), _ptr(ctx.state_slots),
+                                        c_longlong(v.stride(0)), _ptr(b), c_longlong(b.stride(0)), _ptr(a), c_longlong(a.stride(0)),
+                                        _ptr(a_log), _ptr(dt_bias), _ptr(state), c_longlong(state.stride(0)), _ptr(ctx.state_slots),
                                         _ptr(ctx.cu_tokens), c_int(ctx.n_entries), c_int(T), c_int(heads), c_int(qk_heads),
-                                        c_int(dim), c_int(vdim), c_float(q_scale), c_float(norm_eps), *[_ptr(t) for t in scratch],
-                                        c_int(_kind(q.dtype)), _stream()))
+                                        c_int(dim), c_int(vdim), c_float(q_scale), c_float(norm_eps), c_int(int(per_channel)),
+                                        *[_ptr(t) for t in scratch], c_int(_kind(q.dtype)), _stream()))
     count_launches(1)
+
+
+# ---- matrix memory with exponential gates (mlstm.cu) ----------------------------------------
+
+MLSTM_CHUNK = 64       # tokens per chunk of a prompt portion
+MLSTM_COLS = 64        # value columns per block: the normaliser and the running maximum are kept once per block of a head
+
+
+def mlstm_state(heads: int, dim: int, vdim: int):
+    """(offset of n, offset of m, length) of a request's state row [S | n | m], in float32 elements (see mlstm.cu)."""
+    pad4 = lambda n: (n + 3) // 4 * 4
+    blocks = _ceil_div(vdim, MLSTM_COLS)
+    n_off = pad4(heads * dim * vdim)
+    m_off = pad4(n_off + heads * blocks * dim)
+    return n_off, m_off, pad4(m_off + heads * blocks)
+
+
+def mlstm_single_available(dim: int, vdim: int, state: torch.Tensor) -> bool:
+    """Whether the single-token kernel takes these sizes."""
+    return dim <= 512 and vdim % 4 == 0 and state.stride(0) % 4 == 0 and state.data_ptr() % 16 == 0
+
+
+def _mlstm_gates(i_bias, f_bias, cap: float, q_scale: float, heads: int):
+    for t in (i_bias, f_bias):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.numel() == heads
+    return _ptr(i_bias), _ptr(f_bias), c_float(cap), c_float(q_scale)
+
+
+def _mlstm_state_args(state, ctx, heads: int, dim: int, vdim: int):
+    _rows_contig(state, "state")
+    n_off, m_off, size = mlstm_state(heads, dim, vdim)
+    assert state.dtype == torch.float32 and state.shape[1] >= size
+    return (_ptr(state), c_longlong(state.stride(0)), c_longlong(n_off), c_longlong(m_off), _ptr(ctx.state_slots), _ptr(ctx.cu_tokens))
+
+
+def mlstm_scan(out: torch.Tensor, proj, gate_col: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, q_scale: float,
+               state: torch.Tensor, ctx, heads: int, dim: int, vdim: int, single: bool = False) -> None:
+    """The recurrence of mlstm.cu token by token: proj float32 rows [q | k | v | .. | at gate_col: i | f] (a tensor; with
+    single, one token per entry, also a PartialSum of a float32 product); out float32 [T, heads*vdim]."""
+    _rows_contig(out, "out")
+    assert proj.dtype == out.dtype == torch.float32 and out.shape[1] == heads * vdim and gate_col >= heads * (2 * dim + vdim)
+    if isinstance(proj, PartialSum):
+        assert single and proj.rows == ctx.n_tokens and proj.cols >= gate_col + 2 * heads
+        stride = proj.cols
+    else:
+        _rows_contig(proj, "proj")
+        assert proj.shape[1] >= gate_col + 2 * heads
+        stride = proj.stride(0)
+    assert not single or ctx.n_tokens == ctx.n_entries
+    d, parts, splits, split_stride = _split_args(proj)
+    _check(load().llmk_mlstm_scan(_ptr(out), c_longlong(out.stride(0)), d, parts, splits, split_stride, c_longlong(stride),
+                                  c_longlong(gate_col), *_mlstm_gates(i_bias, f_bias, cap, q_scale, heads),
+                                  *_mlstm_state_args(state, ctx, heads, dim, vdim), c_int(ctx.n_entries), c_int(heads), c_int(dim),
+                                  c_int(vdim), c_int(int(single)), _stream()))
+
+
+def mlstm_chunks_available(dtype, dim: int, vdim: int, stride: int, heads: int) -> bool:
+    """Whether the chunk-wise kernels take these sizes (bfloat16 operands on the 16-byte grid)."""
+    return (dtype == torch.bfloat16 and dim % 16 == 0 and dim <= 256 and vdim % 8 == 0 and stride % 8 == 0)
+
+
+def mlstm_chunk_scratch(n_chunks: int, heads: int, dim: int, vdim: int):
+    """Float32 element counts of the chunk-wise form's three scratch buffers for n_chunks chunks."""
+    return [n_chunks * heads * n for n in (dim * vdim, dim, 4)]
+
+
+def mlstm_chunks(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, i_bias: torch.Tensor,
+                 f_bias: torch.Tensor, cap: float, q_scale: float, state: torch.Tensor, ctx, heads: int, dim: int, vdim: int,
+                 scratch) -> None:
+    """mlstm_scan for entries of any length on the tensor cores, chunk by chunk: q, k, v bfloat16 (one row stride), z float32
+    [T, >= 2 heads] the gates' pre-activations [i | f].  scratch: three flat float32 tensors of at least
+    mlstm_chunk_scratch(n_tokens // 64 + n_entries, ...) elements."""
+    for t in (out, q, k, v, z):
+        _rows_contig(t, "mlstm_chunks operand")
+    assert q.stride(0) == k.stride(0) == v.stride(0) and q.dtype == k.dtype == v.dtype == torch.bfloat16
+    assert q.shape[1] == k.shape[1] == heads * dim and v.shape[1] == out.shape[1] == heads * vdim
+    assert out.dtype == z.dtype == torch.float32 and z.shape[1] >= 2 * heads
+    for t, numel in zip(scratch, mlstm_chunk_scratch(ctx.n_tokens // MLSTM_CHUNK + ctx.n_entries, heads, dim, vdim)):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.numel() >= numel
+    _check(load().llmk_mlstm_chunks(_ptr(out), c_longlong(out.stride(0)), _ptr(q), _ptr(k), _ptr(v), c_longlong(q.stride(0)), _ptr(z),
+                                    c_longlong(z.stride(0)), *_mlstm_gates(i_bias, f_bias, cap, q_scale, heads),
+                                    *_mlstm_state_args(state, ctx, heads, dim, vdim), c_int(ctx.n_entries), c_int(ctx.n_tokens),
+                                    c_int(heads), c_int(dim), c_int(vdim), *[_ptr(t) for t in scratch], _stream()))
+    count_launches(2)
 
 
 def group_rmsnorm_gate(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, rows: int, groups: int,
@@ -853,12 +1004,14 @@ def latent_rope_norm_store(x: torch.Tensor, q_gain, q_rank: int, cq_out, gain: t
 
 
 def norm_rope_kv_write(qkv, q_gain, k_gain, eps: float, freqs, halves: bool, positions: torch.Tensor, slot_map, k_pages, v_pages,
-                       n_tokens: int, n_heads: int, n_kv: int, dim: int, vdim: int, q_out=None, amp: float = 1.0) -> torch.Tensor:
+                       n_tokens: int, n_heads: int, n_kv: int, dim: int, vdim: int, q_out=None, amp: float = 1.0,
+                       v_from_k: bool = False) -> torch.Tensor:
     """As rope_pairs_kv_write, with the RMS norm of the token's whole q projection (weights q_gain, float32
     [n_heads * dim]) and whole k projection (k_gain [n_kv * dim]) first, either None for none, and the choice of pairs:
-    halves turns channel i against channel i + len(freqs), else 2i against 2i + 1.  Returns the tensor that holds q."""
-    assert positions.dtype == torch.int32
-    width = n_heads * dim + n_kv * (dim + vdim)
+    halves turns channel i against channel i + len(freqs), else 2i against 2i + 1.  v_from_k: the row has no v columns, the
+    values are the keys as projected, before norm and rotation.  Returns the tensor that holds q."""
+    assert positions.dtype == torch.int32 and (not v_from_k or vdim == dim)
+    width = n_heads * dim + n_kv * (dim if v_from_k else dim + vdim)
     if isinstance(qkv, PartialSum):
         assert q_out is not None and qkv.cols >= width
         src_stride = qkv.cols
@@ -883,7 +1036,7 @@ def norm_rope_kv_write(qkv, q_gain, k_gain, eps: float, freqs, halves: bool, pos
                                           _ptr(q_gain), _ptr(k_gain), c_float(eps), _ptr(freqs), c_int(pairs), c_int(int(halves)),
                                           _ptr(positions), _ptr(slot_map), _ptr(k_pages), _ptr(v_pages), c_int(n_tokens),
                                           c_int(n_heads), c_int(n_kv), c_int(dim), c_int(vdim), c_int(page), c_int(_kind(qkv.dtype)),
-                                          _stream(), c_float(amp)))
+                                          _stream(), c_float(amp), c_int(int(v_from_k))))
     return q_out
 
 
@@ -915,15 +1068,18 @@ def moe_max_tiles(n_pairs: int, experts: int, tile: int = 0) -> int:
 
 def moe_route(h: torch.Tensor, w: torch.Tensor, bias, logits: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
               n_tokens: int, top: int, over_all: bool = False, groups=None, softmax: bool = False, group_max: bool = False,
-              renorm_eps: float = -1.0) -> None:
+              renorm_eps: float = -1.0, gate_out=None) -> None:
     """Router (over_all: the weights are the chosen experts' shares of the softmax over all experts, not
     renormalised): logits = h @ w.T with float32 accumulation (the tensor-core product in bfloat16 where it takes the
     shape, the CUDA-core product otherwise) into `logits` (float32 [>= n_tokens, experts]); plus bias, the `top`
-    largest per token (ids, falling) and the softmax over those alone (weights)."""
+    largest per token (ids, falling) and the softmax over those alone (weights).  gate_out (float32 [>= n_tokens], with groups
+    only): w has one row more than there are experts, and the sigmoid of its logit goes there."""
     _rows_contig(h, "h")
-    experts = w.shape[0]
+    assert gate_out is None or (groups is not None and gate_out.dtype == torch.float32 and gate_out.is_contiguous())
+    stride_ = w.shape[0]
+    experts = stride_ - (1 if gate_out is not None else 0)
     assert w.is_contiguous() and w.dtype == h.dtype and w.shape[1] == h.shape[1]
-    assert logits.dtype == torch.float32 and logits.is_contiguous() and logits.shape[1] == experts and logits.shape[0] >= n_tokens
+    assert logits.dtype == torch.float32 and logits.is_contiguous() and logits.shape[1] == stride_ and logits.shape[0] >= n_tokens
     assert ids.dtype == torch.int32 and weights.dtype == torch.float32 and ids.is_contiguous() and weights.is_contiguous()
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == experts)
     if gemm_fast_available(h, w, logits, n_tokens):
@@ -939,7 +1095,7 @@ def moe_route(h: torch.Tensor, w: torch.Tensor, bias, logits: torch.Tensor, ids:
         count, keep = groups
         _check(load().llmk_moe_topk_grouped(d, parts, splits, stride, _ptr(bias), _ptr(ids), _ptr(weights), c_int(n_tokens),
                                             c_int(experts), c_int(top), c_int(count), c_int(keep), c_int(int(softmax)),
-                                            c_int(int(group_max)), c_float(renorm_eps), _stream()))
+                                            c_int(int(group_max)), c_float(renorm_eps), c_int(stride_), _ptr(gate_out), _stream()))
         return
     _check(load().llmk_moe_topk(d, parts, splits, stride, _ptr(bias), _ptr(ids), _ptr(weights), c_int(n_tokens),
                                 c_int(experts), c_int(top), c_int(int(over_all)), _stream()))
@@ -1009,12 +1165,20 @@ def moe_gemm(a: torch.Tensor, gather_div: int, slot_src, tile_expert, meta, w: t
                                 c_int(ACTIVATIONS[act] if act else -1), c_int(_kind(a.dtype)), c_int(_kind(out.dtype)), _stream()))
 
 
-def moe_combine(out: torch.Tensor, y: torch.Tensor, pair_slot, weights, shared, n_tokens: int, top: int) -> None:
-    """out[t] = shared[t] (a tensor, a PartialSum or None) + sum_j weights[t, j] * y[pair_slot[t, j]]."""
+def moe_combine(out: torch.Tensor, y: torch.Tensor, pair_slot, weights, shared, n_tokens: int, top: int, shared_gate=None,
+                ids=None, first_identity: int = 0, x=None) -> None:
+    """out[t] = shared[t] (a tensor, a PartialSum or None; times shared_gate[t], float32, if given) + sum_j weights[t, j] *
+    y[pair_slot[t, j]].  With ids (int32 [n_tokens * top]) a choice of index first_identity or more counts the row x[t] itself."""
     assert out.is_contiguous() and y.dtype == torch.float32 and y.is_contiguous() and y.shape[1] == out.shape[1]
+    assert shared_gate is None or (shared_gate.dtype == torch.float32 and shared_gate.is_contiguous() and shared_gate.numel() >= n_tokens)
+    if ids is not None:
+        _rows_contig(x, "x")
+        assert ids.dtype == torch.int32 and ids.is_contiguous() and x.dtype == out.dtype and x.shape[1] == out.shape[1]
     d, parts, splits, stride = _split_args(shared)
     _check(load().llmk_moe_combine(_ptr(out), _ptr(y), _ptr(pair_slot), _ptr(weights), d, parts, splits, stride,
-                                   c_int(n_tokens), c_int(top), c_int(out.shape[1]), c_int(_kind(out.dtype)), _stream()))
+                                   c_int(n_tokens), c_int(top), c_int(out.shape[1]), c_int(_kind(out.dtype)), _ptr(ids),
+                                   c_int(first_identity), _ptr(x), c_longlong(x.stride(0) if x is not None else 0),
+                                   _ptr(shared_gate), _stream()))
 
 
 def gather_rows(out: torch.Tensor, resid: torch.Tensor, delta, rows: torch.Tensor, n_rows: int) -> None:

@@ -178,14 +178,15 @@ rope_pairs_kv_write_kernel(MaybePartial<T> src, long long src_stride, T* __restr
 // (n_heads * dim numbers at once, weights q_gain) and of its whole k projection (n_kv * dim, weights k_gain) before they
 // are split into heads (either gain null: that side is not normed), turns the first 2 * rot_pairs channels of every q and k
 // head by position * freqs[i], channel i against channel i + rot_pairs (halves) or 2i against 2i + 1 (neighbours), and
-// stores k and v at the token's slot.  The row is held in shared memory as float32.
+// stores k and v at the token's slot.  The row is held in shared memory as float32.  v_from_k: the row has no v columns, and
+// the values are the keys as projected, before norm and rotation (vdim = dim).
 template <typename T>
 __global__ void __launch_bounds__(256)
 norm_rope_kv_write_kernel(MaybePartial<T> src, long long src_stride, T* __restrict__ q_out, long long q_out_stride,
                           const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
                           const float* __restrict__ freqs, int rot_pairs, int halves, const int* __restrict__ positions,
                           const int* __restrict__ slot_map, T* __restrict__ k_pages, T* __restrict__ v_pages,
-                          int n_heads, int n_kv, int dim, int vdim, int page_size, float amp) {
+                          int n_heads, int n_kv, int dim, int vdim, int page_size, float amp, int v_from_k) {
   extern __shared__ float row_s[];            // [(n_heads + n_kv) * dim]
   __shared__ float red[32];
   pdl_launch_dependents();
@@ -239,7 +240,7 @@ norm_rope_kv_write_kernel(MaybePartial<T> src, long long src_stride, T* __restri
   const size_t v = row + (size_t)(qn + kn);
   for (int idx = threadIdx.x; idx < n_kv * vdim; idx += blockDim.x) {
     const int g = idx / vdim, d = idx % vdim;
-    v_pages[v_base + (size_t)g * page_size * vdim + d] = from_f32<T>(src.at(v + idx));
+    v_pages[v_base + (size_t)g * page_size * vdim + d] = from_f32<T>(v_from_k ? row_s[qn + idx] : src.at(v + idx));
   }
 }
 
@@ -307,16 +308,19 @@ LLMK_API int llmk_rope_pairs_kv_write(const void* qkv, const float* partials, in
 }
 
 // As llmk_rope_pairs_kv_write, with the RMS norm of the whole q and k projections first (gains float32 [n_heads * dim] and
-// [n_kv * dim], each may be null) and the choice of the pairs: halves != 0 turns channel i against i + rot_pairs.
+// [n_kv * dim], each may be null) and the choice of the pairs: halves != 0 turns channel i against i + rot_pairs.  v_from_k: a row
+// is n_heads * dim | n_kv * dim numbers and the values stored are the keys before norm and rotation.
 LLMK_API int llmk_norm_rope_kv_write(const void* qkv, const float* partials, int splits, long long split_stride,
                                      long long src_stride, void* q_out, long long q_out_stride, const float* q_gain,
                                      const float* k_gain, float eps, const float* freqs, int rot_pairs, int halves,
                                      const int* positions, const int* slot_map, void* k_pages, void* v_pages, int n_tokens,
-                                     int n_heads, int n_kv, int dim, int vdim, int page_size, int dtype, cudaStream_t stream, float amp) {
+                                     int n_heads, int n_kv, int dim, int vdim, int page_size, int dtype, cudaStream_t stream, float amp,
+                                     int v_from_k) {
   if (n_tokens == 0) return 0;
   LLMK_REQUIRE((qkv != nullptr) != (partials != nullptr), "norm_rope_kv_write: give qkv or partials");
   LLMK_REQUIRE(rot_pairs >= 0 && 2 * rot_pairs <= dim, "norm_rope_kv_write: %d pairs do not fit a head of %d", rot_pairs, dim);
   LLMK_REQUIRE(rot_pairs == 0 || freqs != nullptr, "norm_rope_kv_write: frequencies are missing");
+  LLMK_REQUIRE(!v_from_k || vdim == dim, "norm_rope_kv_write: keys that are values have one size, not %d and %d", dim, vdim);
   const size_t smem = (size_t)(n_heads + n_kv) * dim * sizeof(float);
   LLMK_REQUIRE(smem <= 200 * 1024, "norm_rope_kv_write: a projection of %d numbers does not fit shared memory", (n_heads + n_kv) * dim);
   return dispatch_dtype(dtype, [&](auto* tag) {
@@ -326,7 +330,7 @@ LLMK_API int llmk_norm_rope_kv_write(const void* qkv, const float* partials, int
       cudaFuncSetAttribute(norm_rope_kv_write_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_kernel(norm_rope_kv_write_kernel<T>, dim3(n_tokens), dim3(256), smem, stream, src, src_stride, (T*)q_out,
                   q_out_stride, q_gain, k_gain, eps, freqs, rot_pairs, halves, positions, slot_map, (T*)k_pages, (T*)v_pages,
-                  n_heads, n_kv, dim, vdim, page_size, amp);
+                  n_heads, n_kv, dim, vdim, page_size, amp, v_from_k);
     LLMK_LAUNCH_CHECK("norm_rope_kv_write");
   });
 }

@@ -12,7 +12,8 @@
 //   products C[slot] = act(A[row of slot] . W[expert of the slot's tile]^T), float32 accumulation in a
 //            fixed k order per element, so a pair's result does not depend on its slot or on what
 //            else is in the batch.
-//   combine  out[t] = shared[t] + sum_j weight[t, j] * y[slot of (t, j)], summed in the order of j.
+//   combine  out[t] = shared[t] + sum_j weight[t, j] * y[slot of (t, j)], summed in the order of j; an identity expert's
+//            y is the input row, and shared may be scaled by a gate of one number per token.
 #include "common.cuh"
 
 namespace {
@@ -87,21 +88,23 @@ topk_kernel(MaybePartial<float> z, const float* __restrict__ bias, int* __restri
 // The experts form `groups` equal runs of neighbours; a group's score is the sum of its two largest choice scores (of its one,
 // in groups of one), or (group_max) its largest; only experts of the `keep` best groups can be chosen: the others are struck
 // out (minus infinity, since choice scores may be negative).  Ties go to the lower index, for groups and for experts.  One
-// warp per token.
+// warp per token.  A row of logits is `stride` long; with gate_out its column `experts` is one more number, whose sigmoid goes to
+// gate_out[t] (the gate of a shared expert, which then costs no product of its own).
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 topk_grouped_kernel(MaybePartial<float> z, const float* __restrict__ correction, int* __restrict__ ids,
                     float* __restrict__ weights, int n_tokens, int experts, int top, int groups, int keep, int softmax,
-                    int group_max, float renorm_eps) {
+                    int group_max, float renorm_eps, int stride, float* __restrict__ gate_out) {
   __shared__ float c_s[ROUTE_WARPS][MAX_EXPERTS], s_s[ROUTE_WARPS][MAX_EXPERTS], g_s[ROUTE_WARPS][MAX_EXPERTS];
   pdl_launch_dependents();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * ROUTE_WARPS + warp;
   if (t >= n_tokens) return;
+  if (gate_out && lane == 0) gate_out[t] = 1.f / (1.f + expf(-z.at((size_t)t * stride + experts)));
   if (softmax) {
     float mx = -INFINITY, sum = 0.f;
     for (int e = lane; e < experts; e += 32) {
-      const float v = z.at((size_t)t * experts + e);
+      const float v = z.at((size_t)t * stride + e);
       s_s[warp][e] = v;
       mx = fmaxf(mx, v);
     }
@@ -119,7 +122,7 @@ topk_grouped_kernel(MaybePartial<float> z, const float* __restrict__ correction,
     }
   } else {
     for (int e = lane; e < experts; e += 32) {
-      const float sc = 1.f / (1.f + expf(-z.at((size_t)t * experts + e)));
+      const float sc = 1.f / (1.f + expf(-z.at((size_t)t * stride + e)));
       s_s[warp][e] = sc;
       c_s[warp][e] = sc + (correction ? correction[e] : 0.f);
     }
@@ -326,10 +329,20 @@ grouped_gemm_kernel(const T* __restrict__ A, long long lda, int gather_div, cons
   }
 }
 
+// What a token's choices beyond the experts with tensors count, and what scales the shared expert: the pair of an expert with an
+// index of `first` or more (an identity expert) has no slot and counts weight * x[t]; gate [t] (or null) multiplies `shared`.
+template <typename T>
+struct CombineMore {
+  const int* ids; int first;            // ids null: no identity experts
+  const T* x; long long x_stride;
+  const float* gate;
+};
+
 // four columns per thread where the rows allow 16-byte loads
 template <typename T>
 __global__ void combine4_kernel(T* __restrict__ out, const float* __restrict__ y, const int* __restrict__ pair_slot,
-                                const float* __restrict__ weights, MaybePartial<T> shared, int top, int width, size_t total4) {
+                                const float* __restrict__ weights, MaybePartial<T> shared, int top, int width, size_t total4,
+                                CombineMore<T> more) {
   pdl_launch_dependents();
   pdl_wait();
   const int per_row = width / 4;
@@ -339,14 +352,21 @@ __global__ void combine4_kernel(T* __restrict__ out, const float* __restrict__ y
     float s[4] = {0.f, 0.f, 0.f, 0.f};
     for (int j = 0; j < top; ++j) {
       const int slot = pair_slot[t * top + j];
-      if (slot < 0) continue;
       const float w = weights[t * top + j];
+      if (slot < 0) {
+        if (more.ids && more.ids[t * top + j] >= more.first) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k) s[k] = fmaf(w, to_f32(more.x[t * more.x_stride + c + k]), s[k]);
+        }
+        continue;
+      }
       const float4 v = *reinterpret_cast<const float4*>(y + (size_t)slot * width + c);
       s[0] = fmaf(w, v.x, s[0]); s[1] = fmaf(w, v.y, s[1]); s[2] = fmaf(w, v.z, s[2]); s[3] = fmaf(w, v.w, s[3]);
     }
     if (shared.present()) {
+      const float g = more.gate ? more.gate[t] : 1.f;
 #pragma unroll
-      for (int k = 0; k < 4; ++k) s[k] += shared.at(t * width + c + k);
+      for (int k = 0; k < 4; ++k) s[k] = fmaf(g, shared.at(t * width + c + k), s[k]);
     }
 #pragma unroll
     for (int k = 0; k < 4; ++k) out[t * width + c + k] = from_f32<T>(s[k]);
@@ -355,7 +375,8 @@ __global__ void combine4_kernel(T* __restrict__ out, const float* __restrict__ y
 
 template <typename T>
 __global__ void combine_kernel(T* __restrict__ out, const float* __restrict__ y, const int* __restrict__ pair_slot,
-                               const float* __restrict__ weights, MaybePartial<T> shared, int top, int width, size_t total) {
+                               const float* __restrict__ weights, MaybePartial<T> shared, int top, int width, size_t total,
+                               CombineMore<T> more) {
   pdl_launch_dependents();
   pdl_wait();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
@@ -365,8 +386,9 @@ __global__ void combine_kernel(T* __restrict__ out, const float* __restrict__ y,
     for (int j = 0; j < top; ++j) {
       const int slot = pair_slot[t * top + j];
       if (slot >= 0) s = fmaf(weights[t * top + j], y[(size_t)slot * width + c], s);
+      else if (more.ids && more.ids[t * top + j] >= more.first) s = fmaf(weights[t * top + j], to_f32(more.x[t * more.x_stride + c]), s);
     }
-    if (shared.present()) s += shared.at(i);
+    if (shared.present()) s = fmaf(more.gate ? more.gate[t] : 1.f, shared.at(i), s);
     out[i] = from_f32<T>(s);
   }
 }
@@ -392,19 +414,22 @@ LLMK_API int llmk_moe_topk(const float* logits, const float* partials, int split
 
 // The router with groups (see topk_grouped_kernel): correction float32 [experts] or null; groups divides experts;
 // 1 <= keep <= groups; softmax 0: sigmoid scores; group_max 0: a group's score is the sum of its two largest; renorm_eps < 0:
-// the weights are the chosen scores as they are.
+// the weights are the chosen scores as they are; stride and gate_out: see the kernel (gate_out may be null).
 LLMK_API int llmk_moe_topk_grouped(const float* logits, const float* partials, int splits, long long split_stride,
                                    const float* correction, int* ids, float* weights, int n_tokens, int experts, int top,
-                                   int groups, int keep, int softmax, int group_max, float renorm_eps, cudaStream_t stream) {
+                                   int groups, int keep, int softmax, int group_max, float renorm_eps, int stride, float* gate_out,
+                                   cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   LLMK_REQUIRE((logits != nullptr) != (partials != nullptr), "moe_topk_grouped: give logits or partials");
   LLMK_REQUIRE(experts > 0 && experts <= MAX_EXPERTS, "moe_topk_grouped: %d experts (1 to %d)", experts, MAX_EXPERTS);
   LLMK_REQUIRE(top > 0 && top <= experts, "moe_topk_grouped: top %d of %d experts", top, experts);
   LLMK_REQUIRE(groups > 0 && experts % groups == 0 && keep > 0 && keep <= groups,
                "moe_topk_grouped: %d experts in %d groups of which %d are kept", experts, groups, keep);
+  LLMK_REQUIRE(stride >= experts + (gate_out ? 1 : 0), "moe_topk_grouped: rows of %d logits for %d experts", stride, experts);
   MaybePartial<float> z{logits, partials, splits, split_stride};
   launch_kernel(topk_grouped_kernel, dim3((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), 0, stream, z,
-                correction, ids, weights, n_tokens, experts, top, groups, keep, softmax, group_max, renorm_eps);
+                correction, ids, weights, n_tokens, experts, top, groups, keep, softmax, group_max, renorm_eps,
+                stride, gate_out);
   LLMK_LAUNCH_CHECK("moe_topk_grouped");
 }
 
@@ -455,10 +480,12 @@ LLMK_API int llmk_moe_gemm(const void* A, long long lda, int gather_div, const i
 }
 
 // out [n_tokens, width] of the element kind = shared (a tensor, partial results, or nothing) + the
-// weighted sum of the pairs' rows of y (float32 [slots, width]).
+// weighted sum of the pairs' rows of y (float32 [slots, width]).  ids (int32 [n_tokens, top], or null), first, x: experts from
+// `first` on are the input row itself; shared_gate float32 [n_tokens] (or null) multiplies shared.
 LLMK_API int llmk_moe_combine(void* out, const float* y, const int* pair_slot, const float* weights, const void* shared,
                               const float* partials, int splits, long long split_stride, int n_tokens, int top, int width,
-                              int dtype, cudaStream_t stream) {
+                              int dtype, const int* ids, int first, const void* x, long long x_stride, const float* shared_gate,
+                              cudaStream_t stream) {
   const size_t total = (size_t)n_tokens * width;
   if (total == 0) return 0;
   LLMK_REQUIRE(!(shared && partials), "moe_combine: give shared or partials, not both");
@@ -467,12 +494,13 @@ LLMK_API int llmk_moe_combine(void* out, const float* y, const int* pair_slot, c
   return dispatch_dtype(dtype, [&](auto* tag) {
     using T = LLMK_ELEM(tag);
     MaybePartial<T> s{(const T*)shared, partials, splits, split_stride};
+    const CombineMore<T> more{ids, first, (const T*)x, x_stride, shared_gate};
     if (width % 4 == 0 && (uintptr_t)y % 16 == 0) {
       size_t b4 = (total / 4 + 255) / 256;
       if (b4 > (size_t)llmk_sm_count() * 16) b4 = (size_t)llmk_sm_count() * 16;
-      launch_kernel(combine4_kernel<T>, dim3((unsigned)b4), dim3(256), 0, stream, (T*)out, y, pair_slot, weights, s, top, width, total / 4);
+      launch_kernel(combine4_kernel<T>, dim3((unsigned)b4), dim3(256), 0, stream, (T*)out, y, pair_slot, weights, s, top, width, total / 4, more);
     } else {
-      launch_kernel(combine_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (T*)out, y, pair_slot, weights, s, top, width, total);
+      launch_kernel(combine_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (T*)out, y, pair_slot, weights, s, top, width, total, more);
     }
     LLMK_LAUNCH_CHECK("moe_combine");
   });

@@ -21,7 +21,8 @@ no normalisation over the keys (weights="sigmoid").  Further still: a sink whose
 (sink="learned", tensor `sink`); a bias that grows with the distance, r1_h ln(1 + r2_h (i - j)) taken off the capped score
 (dist_bias, tensors `r1`, `r2`); a short causal convolution over time on every channel of the projected (and biased) q, k, v
 (qkv_conv = taps, tensors `<projection>.conv` [channels, taps]; the last taps - 1 projected rows are the request's state); and
-biases on q, k, v without one on the output (out_bias=False).
+biases on q, k, v without one on the output (out_bias=False); and values that are the keys as projected, before rotation
+(keys_as_values: no value projection).
 """
 from __future__ import annotations
 
@@ -45,8 +46,8 @@ class PagedAttention(Part):
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, position=None,
                  window=None, scale=None, shares_cache: bool = False, bias: bool = False, value_dim=None, softcap=None,
                  sink: bool = False, keep_first: int = 0, names=None, chunk=None, weights: str = "softmax", qk_norm=None,
-                 norm_eps: float = 1e-6, out_bias=None, qkv_conv: int = 0, dist_bias: bool = False, prefix: str = "",
-                 dtype=None, device=None):
+                 norm_eps: float = 1e-6, out_bias=None, qkv_conv: int = 0, dist_bias: bool = False,
+                 keys_as_values: bool = False, prefix: str = "", dtype=None, device=None):
         super().__init__(prefix, dtype, device)
         if num_heads % num_kv_heads:
             raise ValueError(f"attention: {num_heads} heads do not divide into {num_kv_heads} kv heads")
@@ -80,7 +81,10 @@ class PagedAttention(Part):
             raise ValueError("attention: sigmoid weights take no sink and no soft cap")
         # the options above, and pair rotation, run on the path that rotates and stores with one kernel and
         # attends with a kernel that takes them (see forward)
-        self.extended = bool(self.value_dim != head_dim or self.softcap or self.sink or self.keep_first or self.qkv_conv
+        self.keys_as_values = bool(keys_as_values)
+        if self.keys_as_values and (self.value_dim != head_dim or bias or self.qkv_conv or shares_cache):
+            raise ValueError("attention: keys that serve as values have the values' size, no bias, no convolution and pages of their own")
+        self.extended = bool(self.keys_as_values or self.value_dim != head_dim or self.softcap or self.sink or self.keep_first or self.qkv_conv
                              or self.dist_bias or self.chunk or self.sigmoid or self.qk_norm
                              or (self.position is not None and hasattr(self.position, "frequencies")))
         self.out_bias = bool(bias) if out_bias is None else bool(out_bias)
@@ -89,7 +93,7 @@ class PagedAttention(Part):
                              "without a bias on the output")
         self.q_size = num_heads * head_dim
         self.kv_size = 0 if shares_cache else num_kv_heads * head_dim
-        self.v_size = 0 if shares_cache else num_kv_heads * self.value_dim
+        self.v_size = 0 if shares_cache or self.keys_as_values else num_kv_heads * self.value_dim
         self.bias = bool(bias)        # q/k/v and o projections carry bias vectors (model/modules/Attention.h:16-19)
         self.w_qkv = None
         self.w_o = None
@@ -104,6 +108,7 @@ class PagedAttention(Part):
         p = {n("q"): ParamInfo((self.q_size, self.hidden_size))}
         if not self.shares_cache:
             p[n("k")] = ParamInfo((self.kv_size, self.hidden_size))
+        if self.v_size:
             p[n("v")] = ParamInfo((self.v_size, self.hidden_size))
         p[n("o")] = ParamInfo((self.hidden_size, self.num_heads * self.value_dim))
         if self.sigmoid:
@@ -133,7 +138,7 @@ class PagedAttention(Part):
         n = lambda k: tensors[self.name(self.names[k])]
         parts = [n("q")]
         if not self.shares_cache:
-            parts += [n("k"), n("v")]
+            parts += [n("k")] if self.keys_as_values else [n("k"), n("v")]
         self.w_qkv = torch.cat(parts, dim=0).contiguous() if len(parts) > 1 else parts[0].contiguous()
         self.w_o = n("o").contiguous()
         if self.sigmoid:
@@ -250,10 +255,10 @@ class PagedAttention(Part):
         halves = getattr(self.position, "layout", "pairs") == "halves"
         amp = getattr(self.position, "amplitude", 1.0)
         q_out = ws.get("q_rot", T, self.q_size, self.dtype) if isinstance(qkv, ops.PartialSum) else None
-        if self.qk_norm or halves:
+        if self.qk_norm or halves or self.keys_as_values:
             q = ops.norm_rope_kv_write(qkv, self.q_gain, self.k_gain, self.norm_eps, freqs, halves, ctx.positions,
                                        view.group.slot_map, k_pages, v_pages, T, H, 0 if self.shares_cache else n_kv, D, V,
-                                       q_out=q_out, amp=amp)
+                                       q_out=q_out, amp=amp, v_from_k=self.keys_as_values)
         else:
             q = ops.rope_pairs_kv_write(qkv, freqs, ctx.positions, view.group.slot_map, k_pages, v_pages, T, H,
                                         0 if self.shares_cache else n_kv, D, V, q_out=q_out, amp=amp)

@@ -82,12 +82,15 @@ class SandwichBlock:
             if self.parts[r] is not None and not hasattr(self.parts[r], "attach"):
                 raise ValueError(f"sandwich block: the norm '{part_specs[r].kind}' cannot stand behind a sublayer (no attach)")
         self.mixer, self.ffn = self.parts["mixer"], self.parts["ffn"]
+        # a feed-forward whose last bias the norm behind it can add leaves it to that norm
+        self.biased = ({"allow_biased": True} if getattr(self.ffn, "leaves_bias", False)
+                       and getattr(self.parts["post2"], "takes_bias", False) else {})
 
     def forward(self, stream: ResidualStream, ctx, view) -> None:
         p = self.parts
         p["post1"].attach(stream, self.mixer.forward(p["norm1"].forward(stream, ctx), ctx, view), self.mult)
         if self.ffn is not None:
-            p["post2"].attach(stream, self.ffn.forward(p["norm2"].forward(stream, ctx), ctx), self.mult)
+            p["post2"].attach(stream, self.ffn.forward(p["norm2"].forward(stream, ctx), ctx, **self.biased), self.mult)
 
 
 register_part("block", "sandwich", SandwichBlock)

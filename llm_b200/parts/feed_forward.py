@@ -58,15 +58,15 @@ class SwiGLU(Part):
             self.b_gate_up = torch.cat([n("gate_bias"), n("up_bias")]).contiguous()
             self.b_down = n("down_bias").contiguous()
 
-    def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, ctx, tag: str = "ffn") -> torch.Tensor:
         T, ws = ctx.n_tokens, ctx.workspace
-        act = ws.get("ffn_act", T, self.intermediate_size, self.dtype)
+        act = ws.get(tag + "_act", T, self.intermediate_size, self.dtype)
         # with many rows the product's epilogue makes the activation; with few rows, or biases, the row kernel
         if self.bias or not linear_swiglu(x, self.w_gate_up, act, T, self.activation):
             gate_up = linear(x, self.w_gate_up, ws.get("gate_up", T, 2 * self.intermediate_size, self.dtype), T,
                              allow_partial=FUSE_PARTIALS, bias=self.b_gate_up)
             ops.silu_mul(act, gate_up, T, self.activation)
-        return linear(act, self.w_down, ws.get("ffn_out", T, self.hidden_size, self.dtype), T, allow_partial=FUSE_PARTIALS,
+        return linear(act, self.w_down, ws.get(tag + "_out", T, self.hidden_size, self.dtype), T, allow_partial=FUSE_PARTIALS,
                       bias=self.b_down)
 
 
@@ -76,30 +76,49 @@ register_part("ffn", "swiglu", SwiGLU)
 class ActMLP(Part):
     """down(act(up(x))): a feed-forward with one up-projection and an element-wise activation
     ("relu2": the square of relu, "gelu": erf, "gelu_tanh", "silu").  Tensors `<prefix>.up` and
-    `<prefix>.down` unless other names are given."""
+    `<prefix>.down` unless other names are given; with bias also `<up>.b` and `<down>.b`, of which the first is added in the
+    activation's kernel and the second, where the caller allows it, by the kernel that reads the result (ops.BiasedRows)."""
 
     role = "ffn"
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "relu2", up_name: str = "up",
-                 down_name: str = "down", prefix: str = "", dtype=None, device=None):
+                 down_name: str = "down", bias: bool = False, prefix: str = "", dtype=None, device=None):
         super().__init__(prefix, dtype, device)
         if activation not in ops.ACTIVATIONS:
             raise ValueError(f"feed-forward: unknown activation '{activation}'; known: {sorted(ops.ACTIVATIONS)}")
         self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
-        self.up_name, self.down_name = up_name, down_name
-        self.w_up = self.w_down = None
+        self.up_name, self.down_name, self.bias = up_name, down_name, bool(bias)
+        self.w_up = self.w_down = self.b_up = self.b_down = None
+
+    @property
+    def leaves_bias(self) -> bool:
+        return self.bias
 
     def parameters(self):
-        return {self.name(self.up_name): ParamInfo((self.intermediate_size, self.hidden_size)),
-                self.name(self.down_name): ParamInfo((self.hidden_size, self.intermediate_size))}
+        p = {self.name(self.up_name): ParamInfo((self.intermediate_size, self.hidden_size)),
+             self.name(self.down_name): ParamInfo((self.hidden_size, self.intermediate_size))}
+        if self.bias:
+            p[self.name(self.up_name + ".b")] = ParamInfo((self.intermediate_size,), kind="gain", init="normal")
+            p[self.name(self.down_name + ".b")] = ParamInfo((self.hidden_size,), kind="gain", init="normal")
+        return p
 
     def bind(self, tensors):
         self.w_up = tensors[self.name(self.up_name)].contiguous()
         self.w_down = tensors[self.name(self.down_name)].contiguous()
+        if self.bias:
+            self.b_up = tensors[self.name(self.up_name + ".b")].contiguous()
+            self.b_down = tensors[self.name(self.down_name + ".b")].contiguous()
 
-    def forward(self, x: torch.Tensor, ctx, tag: str = "ffn") -> torch.Tensor:
+    def forward(self, x: torch.Tensor, ctx, tag: str = "ffn", allow_biased: bool = False):
         T, ws = ctx.n_tokens, ctx.workspace
         act = ws.get(tag + "_act", T, self.intermediate_size, self.dtype)
+        if self.bias:
+            up = linear(x, self.w_up, ws.get(tag + "_up", T, self.intermediate_size, self.dtype), T, allow_partial=FUSE_PARTIALS)
+            ops.bias_act_rows(act, up, self.b_up, T, self.activation)
+            out = ws.get(tag + "_out", T, self.hidden_size, self.dtype)
+            if allow_biased:
+                return ops.BiasedRows(linear(act, self.w_down, out, T, allow_partial=FUSE_PARTIALS), self.b_down)
+            return linear(act, self.w_down, out, T, bias=self.b_down)
         if not linear_act(x, self.w_up, act, T, self.activation):      # many rows: the activation in the product's epilogue
             up = linear(x, self.w_up, ws.get(tag + "_up", T, self.intermediate_size, self.dtype), T, allow_partial=FUSE_PARTIALS)
             ops.act_rows(act, up, T, self.activation)

@@ -16,21 +16,27 @@ from .base import ParamInfo, Part, ResidualStream, register_part
 class RMSNorm(Part):
     role = "norm"
 
-    def __init__(self, size: int, eps: float, weight_name: str = "weight", centred: bool = False, prefix: str = "", dtype=None,
-                 device=None):
+    def __init__(self, size: int, eps: float, weight_name: str = "weight", centred: bool = False, scale_name: str = None,
+                 prefix: str = "", dtype=None, device=None):
         super().__init__(prefix, dtype, device)
         self.size = size
         self.eps = float(eps)
         self.weight_name = weight_name        # "": the gain is the tensor named like the part
         self.centred = bool(centred)          # the stored weight is the gain's distance from one
+        self.scale_name = scale_name          # a second vector on the result (a layer scale): part of the gain
         self.gain = None
 
     def parameters(self):
-        return {self.name(self.weight_name): ParamInfo((self.size,), kind="gain", init="normal" if self.centred else "ones_normal")}
+        p = {self.name(self.weight_name): ParamInfo((self.size,), kind="gain", init="normal" if self.centred else "ones_normal")}
+        if self.scale_name is not None:
+            p[self.name(self.scale_name)] = ParamInfo((self.size,), kind="gain", init="ones_normal")
+        return p
 
     def bind(self, tensors):
         w = tensors[self.name(self.weight_name)]
         self.gain = (w + 1.0).contiguous() if self.centred else w
+        if self.scale_name is not None:
+            self.gain = (self.gain * tensors[self.name(self.scale_name)]).contiguous()
 
     def close(self, stream: ResidualStream, y, alpha: float, ctx) -> None:
         """The norm behind a residual sum: x <- rms(alpha * x + y) * gain, in float32 on the stream, with a copy of the new
@@ -45,9 +51,33 @@ class RMSNorm(Part):
 
     def forward(self, stream: ResidualStream, ctx, tag: str = "normed") -> torch.Tensor:
         out = ctx.workspace.get(tag, stream.rows, self.size, self.dtype)
+        if stream.pending_post is not None:
+            self._add_posted(stream, self.gain, out)
+            return out
         ops.add_rmsnorm(stream.resid, stream.pending, self.gain, out, stream.rows, self.eps)
         stream.pending = None
         return out
+
+    takes_bias = True      # attach() takes ops.BiasedRows
+
+    def attach(self, stream: ResidualStream, y, mult: float = 1.0) -> None:
+        """A sublayer's output left pending, to be normed by this part and scaled by `mult` before it joins the residual: x +=
+        mult * rms(y) * gain.  The norm that comes next (or fold) does both in one pass over the row."""
+        stream.pending, stream.pending_post = y, (self, float(mult))
+
+    def _add_posted(self, stream: ResidualStream, pre, out) -> None:
+        part, mult = stream.pending_post
+        if not isinstance(part, RMSNorm) or part.eps != self.eps:
+            raise ValueError("a pending term that another kind of norm is to treat cannot be folded by this one")
+        y, bias = stream.pending, None
+        if isinstance(y, ops.BiasedRows):
+            y, bias = y.rows, y.bias
+        ops.add_rmsnorms(stream.resid, y, part.gain, mult, pre, out, stream.rows, self.eps, delta_bias=bias)
+        stream.pending = stream.pending_post = None
+
+    def fold(self, stream: ResidualStream, ctx) -> None:
+        """resid += mult * rms(pending) * gain: the stream made whole without a norm after it."""
+        self._add_posted(stream, None, None)
 
     def forward_rows(self, rows_f32: torch.Tensor, n_rows: int, out: torch.Tensor) -> torch.Tensor:
         """Norm of float32 rows that are not a stream (the gathered rows before the head)."""

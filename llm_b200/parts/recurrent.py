@@ -7,7 +7,7 @@
   hgrn2          a forget gate with a lower bound that also decides what is written: S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T,
                  o_t = S_t^T silu(q_t); no key
   gated_delta    the gated delta rule: S <- g_t S; u = beta_t (v_t - S^T k_t); S <- S + k_t u^T; o_t = S^T q_t with unit q, k
-                 behind a short convolution and silu, one decay and one beta per head
+                 behind a short convolution and silu, one decay (or one per key channel) and one beta per head
   conv_input     a wrapper: the inner mixer (or feed-forward) reads h + conv(h), a short causal convolution per channel
   parallel       a wrapper: two mixers read the same rows; the result is the mean of their RMS-normed outputs, or a sum of
                  the two with fixed scales
@@ -269,14 +269,19 @@ class GatedDeltaRule(Part):
     convolution, then silu); b, a [H, W] (beta = sigmoid(b h), decay = exp(-exp(A_log) softplus(a h + dt_bias))); A_log,
     dt_bias [H]; g [H*V, W] (the output gate, silu); norm [V] (shared by the heads); o [W, H*V].  q and k become unit vectors
     per head and q is scaled by D^(-1/2).  Head h reads q/k head h // (H / G).  State row: [the convolution's last
-    taps - 1 inputs | S: H * D * V]."""
+    taps - 1 inputs | S: H * D * V].
+
+    channel_decay: a decay per head and key channel through a low rank, softplus(a2 (a1 h) + dt_bias) with a1 [rank, W],
+    a2 [H*D, rank] and dt_bias [H*D] in place of a and dt_bias [H].  low_rank_gate: the output gate is sigmoid(g2 (g1 h)), g1
+    [rank, W], g2 [H*V, rank], in place of g.  The ranks are the checkpoint's."""
 
     role = "mixer"
 
     def __init__(self, hidden_size: int, num_heads: int, num_qk_heads: int, head_dim: int, value_dim: int, taps: int, eps: float,
-                 unit_eps: float = 1e-6, prefix: str = "", dtype=None, device=None):
+                 unit_eps: float = 1e-6, channel_decay: bool = False, low_rank_gate: bool = False, rank: int = 16, prefix: str = "",
+                 dtype=None, device=None):
         super().__init__(prefix, dtype, device)
-        if min(hidden_size, num_heads, num_qk_heads, head_dim, value_dim) <= 0 or not (1 <= taps <= 16):
+        if min(hidden_size, num_heads, num_qk_heads, head_dim, value_dim, rank) <= 0 or not (1 <= taps <= 16):
             raise ValueError("gated delta rule: sizes must be positive and taps 1 to 16")
         if num_heads % num_qk_heads:
             raise ValueError(f"gated delta rule: {num_heads} heads do not divide into {num_qk_heads} key heads")
@@ -285,25 +290,52 @@ class GatedDeltaRule(Part):
         self.hidden_size, self.num_heads, self.num_qk_heads = int(hidden_size), int(num_heads), int(num_qk_heads)
         self.head_dim, self.value_dim, self.taps = int(head_dim), int(value_dim), int(taps)
         self.eps, self.unit_eps = float(eps), float(unit_eps)
+        self.channel_decay, self.low_rank_gate, self.rank = bool(channel_decay), bool(low_rank_gate), int(rank)
         self.qk_size, self.v_size = self.num_qk_heads * self.head_dim, self.num_heads * self.value_dim
         self.conv_channels = 2 * self.qk_size + self.v_size
         self.conv_cols = _pad4((self.taps - 1) * self.conv_channels)
-        self.w_in = self.w_conv = self.a_log = self.dt_bias = self.gain = self.w_o = None
+        self.w_in = self.w_conv = self.a_log = self.dt_bias = self.gain = self.w_o = self.w_a2 = self.w_g2 = None
+        self.cols = {}            # column range of the input product by local name
 
     def parameters(self):
-        n, W, H = self.name, self.hidden_size, self.num_heads
+        n, W, H, R = self.name, self.hidden_size, self.num_heads, self.rank
         p = {n("q"): ParamInfo((self.qk_size, W)), n("k"): ParamInfo((self.qk_size, W)), n("v"): ParamInfo((self.v_size, W)),
-             n("b"): ParamInfo((H, W)), n("a"): ParamInfo((H, W)), n("g"): ParamInfo((self.v_size, W)),
-             n("A_log"): ParamInfo((H,), kind="gain", init="normal"), n("dt_bias"): ParamInfo((H,), kind="gain", init="normal"),
+             n("b"): ParamInfo((H, W)), n("A_log"): ParamInfo((H,), kind="gain", init="normal"),
              n("norm"): ParamInfo((self.value_dim,), kind="gain", init="ones_normal"), n("o"): ParamInfo((W, self.v_size))}
+        if self.channel_decay:
+            p.update({n("a1"): ParamInfo((R, W), free_dims=(0,)), n("a2"): ParamInfo((H * self.head_dim, R), free_dims=(1,)),
+                      n("dt_bias"): ParamInfo((H * self.head_dim,), kind="gain", init="normal")})
+        else:
+            p.update({n("a"): ParamInfo((H, W)), n("dt_bias"): ParamInfo((H,), kind="gain", init="normal")})
+        if self.low_rank_gate:
+            p.update({n("g1"): ParamInfo((R, W), free_dims=(0,)), n("g2"): ParamInfo((self.v_size, R), free_dims=(1,))})
+        else:
+            p[n("g")] = ParamInfo((self.v_size, W))
         for m, c in (("q", self.qk_size), ("k", self.qk_size), ("v", self.v_size)):
             p[n(m + ".conv")] = ParamInfo((c, self.taps), kind="gain", init="normal")
         return p
 
     def bind(self, tensors):
         t = lambda local: tensors[self.name(local)]
-        # one product for everything the mixer reads from h: [q | k | v | gate | b | a]
-        self.w_in = torch.cat([t("q"), t("k"), t("v"), t("g"), t("b"), t("a")], dim=0).contiguous()
+        # one product for everything the mixer reads from h: [q | k | v | gate | b | decay]; with low ranks every range behind
+        # the convolution's starts on a multiple of 8 columns and is as wide, so that it can be a product's operand in turn
+        grid = 8 if self.channel_decay or self.low_rank_gate else 1
+        rows, at = [t("q"), t("k"), t("v")], self.conv_channels
+        for local in ("g1" if self.low_rank_gate else "g", "b", "a1" if self.channel_decay else "a"):
+            w = t(local)
+            before, behind = -at % grid, -w.shape[0] % grid
+            rows += [w.new_zeros(before, w.shape[1]), w, w.new_zeros(behind, w.shape[1])]
+            self.cols[local] = slice(at + before, at + before + w.shape[0] + (behind if local in ("a1", "g1") else 0))
+            at += before + w.shape[0] + behind
+        self.w_in = torch.cat(rows, dim=0).contiguous()
+
+        def second(local, first):
+            w = t(local)
+            if w.shape[1] != t(first).shape[0]:
+                raise ValueError(f"{self.prefix}: {first} and {local} disagree on their rank ({t(first).shape[0]} and {w.shape[1]})")
+            return torch.nn.functional.pad(w, (0, -w.shape[1] % grid)).contiguous()
+        self.w_a2 = second("a2", "a1") if self.channel_decay else None
+        self.w_g2 = second("g2", "g1") if self.low_rank_gate else None
         self.w_conv = torch.cat([t("q.conv"), t("k.conv"), t("v.conv")], dim=0).t().contiguous()      # [taps, channels]
         self.a_log, self.dt_bias = t("A_log").contiguous(), t("dt_bias").contiguous()
         self.gain, self.w_o = t("norm").contiguous(), t("o").contiguous()
@@ -318,23 +350,31 @@ class GatedDeltaRule(Part):
         T, ws = ctx.n_tokens, ctx.workspace
         QK, VS, C, H = self.qk_size, self.v_size, self.conv_channels, self.num_heads
         conv_state, S = view.state[:, :self.conv_cols], view.state[:, self.conv_cols:]
-        proj = linear(x, self.w_in, ws.get("delta_in", T, C + VS + 2 * H, self.dtype), T)
+        proj = linear(x, self.w_in, ws.get("delta_in", T, self.w_in.shape[0], self.dtype), T)
         qkv = ws.get("delta_qkv", T, C, self.dtype)
         ops.short_conv(qkv, proj[:, :C], self.w_conv, None, conv_state, ctx, silu=True)
         o = ws.get("delta_o", T, VS, torch.float32)
-        operands = (o, qkv[:, :QK], qkv[:, QK:2 * QK], qkv[:, 2 * QK:], proj[:, C + VS:C + VS + H], proj[:, C + VS + H:],
+        if self.channel_decay:      # the decays' pre-activation in float32; bias, softplus and exponentials are the kernel's
+            a = linear(proj[:, self.cols["a1"]], self.w_a2, ws.get("delta_z", T, H * self.head_dim, torch.float32), T)
+        else:
+            a = proj[:, self.cols["a"]]
+        operands = (o, qkv[:, :QK], qkv[:, QK:2 * QK], qkv[:, 2 * QK:], proj[:, self.cols["b"]], a,
                     self.a_log, self.dt_bias, S, ctx, H, self.num_qk_heads, self.head_dim, self.value_dim, self.head_dim ** -0.5,
                     self.unit_eps)
         if CHUNKED_DELTA and not ctx.decode_only and T >= 4 * SEGMENT:
             # a step with prompt portions: chunks of 32 tokens solved together, chained through the state
             cap = ws.max_rows // ops.DELTA_CHUNK + ctx.cu_tokens.numel()          # chunks of any step: the buffers' sizes
-            scratch = [ws.flat("delta_chunk_" + tag, numel, torch.float32)
-                       for tag, numel in zip(("yq", "k", "w", "b", "g"), ops.delta_chunk_scratch(cap, H, self.head_dim, self.value_dim))]
-            ops.delta_chunk_scan(*operands, scratch)
+            sizes = ops.delta_chunk_scratch(cap, H, self.head_dim, self.value_dim, self.channel_decay)
+            scratch = [ws.flat("delta_chunk_" + tag, numel, torch.float32) for tag, numel in zip(("yq", "k", "w", "b", "g"), sizes)]
+            ops.delta_chunk_scan(*operands, scratch, per_channel=self.channel_decay)
         else:
-            ops.delta_scan(*operands)
+            ops.delta_scan(*operands, per_channel=self.channel_decay)
         normed = ws.get("delta_normed", T, VS, self.dtype)
-        ops.head_rmsnorm_gate(normed, o, self.gain, proj[:, C:C + VS], T, H, self.eps)
+        if self.low_rank_gate:
+            gate = linear(proj[:, self.cols["g1"]], self.w_g2, ws.get("delta_gate", T, VS, self.dtype), T, allow_partial=FUSE_PARTIALS)
+            ops.head_rmsnorm_sigmoid(normed, o, self.gain, gate, 0, T, H, self.eps)
+        else:
+            ops.head_rmsnorm_gate(normed, o, self.gain, proj[:, self.cols["g"]], T, H, self.eps)
         return linear(normed, self.w_o, ws.get("delta_out", T, self.hidden_size, self.dtype), T, allow_partial=FUSE_PARTIALS)
 
 

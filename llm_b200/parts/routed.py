@@ -10,7 +10,10 @@ the chosen weights do not sum to one); router "sigmoid_groups", where the scores
 s + correction (a learned vector, `<prefix>.correction`), the experts form `groups` equal runs of neighbours of which only the
 `keep_groups` best (by the sum of their two largest choice scores) can be chosen from, and the weights are the chosen s,
 not renormalised; "softmax_groups", the same with s = softmax(z) over all experts, a group counted by its largest choice score
-alone, and the chosen s divided by their sum + weight_eps; gated experts, down_e(act(gate_e(h)) * up_e(h)), with act silu or the clamped unit
+alone, and the chosen s divided by their sum + weight_eps; "softmax_corrected", the same without groups and with the weights as
+they are; identity experts behind the others (`identity` more outputs of the router), whose output is the input row; a shared
+expert that is gated like the others, down_s(silu(gate_s(h)) * up_s(h)) (shared_gated), and multiplied by sigmoid(Wsg h), one number
+per token (shared_gate, tensor `<prefix>.shared.sg`), which is made as one more row of the router's product; gated experts, down_e(act(gate_e(h)) * up_e(h)), with act silu or the clamped unit
 g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit) (activation "clamped").
 
 On the device: the router kernel writes each token's choices and weights; the (token, choice)
@@ -27,7 +30,7 @@ import torch
 
 from ..csrc import ops
 from .base import ParamInfo, Part, register_part
-from .feed_forward import ActMLP
+from .feed_forward import ActMLP, SwiGLU
 
 
 # Gated experts on the tensor cores: from this width on the grouped product applies silu(gate) * up in its epilogue;
@@ -45,14 +48,16 @@ class RoutedFFN(Part):
     def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, activation: str = "gelu",
                  router_bias: bool = True, shared_size: int = 0, shared_activation: str = None, gated: bool = False,
                  router: str = "softmax_chosen", groups: int = 1, keep_groups: int = 1, limit: float = 0.0, alpha: float = 1.702,
-                 weight_eps: float = 1e-20, prefix: str = "", dtype=None, device=None):
+                 weight_eps: float = 1e-20, identity: int = 0, shared_gated: bool = False, shared_gate: bool = False,
+                 prefix: str = "", dtype=None, device=None):
         super().__init__(prefix, dtype, device)
-        if not (0 < top <= experts <= 256):
-            raise ValueError(f"routed feed-forward: top {top} of {experts} experts (1 <= top <= experts <= 256)")
+        self.identity, self.outputs = int(identity), experts + int(identity)      # outputs of the router
+        if not (0 < top <= self.outputs <= 256) or experts <= 0 or identity < 0:
+            raise ValueError(f"routed feed-forward: top {top} of {experts} + {identity} experts (1 <= top <= experts <= 256)")
         if activation not in ops.ACTIVATIONS and activation != "clamped":
             raise ValueError(f"routed feed-forward: unknown activation '{activation}'")
         self.hidden_size, self.experts, self.top, self.expert_size = hidden_size, experts, top, expert_size
-        if router not in ("softmax_chosen", "softmax_all", "sigmoid_groups", "softmax_groups"):
+        if router not in ("softmax_chosen", "softmax_all", "sigmoid_groups", "softmax_groups", "softmax_corrected"):
             raise ValueError(f"routed feed-forward: unknown router '{router}'")
         if gated and activation not in ("silu", "clamped") or (activation == "clamped" and not gated):
             raise ValueError("routed feed-forward: gated experts take the silu activation or the clamped unit, and only they the latter")
@@ -69,21 +74,34 @@ class RoutedFFN(Part):
             if router == "softmax_groups":
                 self.route_options = {"softmax": True, "group_max": True, "renorm_eps": float(weight_eps)}
             router_bias = False
+        elif router == "softmax_corrected":
+            self.groups, self.route_options, router_bias = (1, 1), {"softmax": True}, False
+        self.shared_gate = bool(shared_gate and shared_size)
+        if (self.identity or self.shared_gate) and (self.groups is None or self.groups[0] > 1):
+            raise ValueError("routed feed-forward: identity experts and a gate on the shared expert go with the corrected router without groups")
         self.activation, self.router_bias = activation, bool(router_bias)
         self.gated, self.over_all = bool(gated), router == "softmax_all"
-        self.shared = (ActMLP(hidden_size, shared_size, shared_activation or activation, prefix=self.name("shared"),
-                              dtype=dtype, device=device) if shared_size else None)
+        if not shared_size:
+            self.shared = None
+        elif shared_gated:
+            self.shared = SwiGLU(hidden_size, shared_size, names={"gate": "gate", "up": "up", "down": "down"}, prefix=self.name("shared"),
+                                 dtype=dtype, device=device)
+        else:
+            self.shared = ActMLP(hidden_size, shared_size, shared_activation or activation, prefix=self.name("shared"),
+                                 dtype=dtype, device=device)
         self.w_router = self.b_router = self.w_up = self.w_down = None
 
     def children(self):
         return [self.shared] if self.shared is not None else []
 
     def parameters(self):
-        p = {self.name("router"): ParamInfo((self.experts, self.hidden_size))}
+        p = {self.name("router"): ParamInfo((self.outputs, self.hidden_size))}
+        if self.shared_gate:
+            p[self.name("shared.sg")] = ParamInfo((1, self.hidden_size))
         if self.router_bias:
             p[self.name("router.b")] = ParamInfo((self.experts,), kind="gain", init="normal")
         if self.groups:
-            p[self.name("correction")] = ParamInfo((self.experts,), kind="gain", init="normal")
+            p[self.name("correction")] = ParamInfo((self.outputs,), kind="gain", init="normal")
         for e in range(self.experts):
             if self.gated:
                 p[self.name(f"e{e}.gate")] = ParamInfo((self.expert_size, self.hidden_size))
@@ -93,6 +111,8 @@ class RoutedFFN(Part):
 
     def bind(self, tensors):
         self.w_router = tensors[self.name("router")].contiguous()
+        if self.shared_gate:
+            self.w_router = torch.cat([self.w_router, tensors[self.name("shared.sg")]], dim=0).contiguous()
         self.b_router = tensors[self.name("router.b")].contiguous() if self.router_bias else None
         if self.groups:
             self.b_router = tensors[self.name("correction")].contiguous()      # enters the choice, not the weights
@@ -113,7 +133,7 @@ class RoutedFFN(Part):
     @property
     def leaves_unsummed(self) -> bool:
         """Whether the weighted sum of a token's experts can be left to the kernel that reads it (no shared expert beside it)."""
-        return self.shared is None
+        return self.shared is None and not self.identity
 
     def forward(self, x: torch.Tensor, ctx, allow_unsummed: bool = False):
         """With allow_unsummed (and no shared expert) the result is an ops.WeightedRows, else a tensor."""
@@ -136,9 +156,10 @@ class RoutedFFN(Part):
         act = ws.flat("moe_act", cap_slots * self.expert_size, self.dtype).view(cap_slots, self.expert_size)
         y = ws.flat("moe_y", cap_slots * self.hidden_size, f32).view(cap_slots, self.hidden_size)
 
-        logits = ws.get("moe_logits", T, E, f32)
+        logits = ws.get("moe_logits", T, self.w_router.shape[0], f32)
+        gate = ws.flat("moe_shared_gate", ws.max_rows, f32) if self.shared_gate else None
         ops.moe_route(x, self.w_router, self.b_router, logits, ids, wts, T, top, over_all=self.over_all,
-                      groups=self.groups, **self.route_options)
+                      groups=self.groups, gate_out=gate, **self.route_options)
         ops.moe_group(ids, pairs, E, meta, tile_expert, slot_src, pair_slot, max_tiles, tile)
         if tensor:
             # gated experts: a tile multiplies by its expert's gate rows and up rows and the epilogue makes silu(gate) * up
@@ -166,7 +187,8 @@ class RoutedFFN(Part):
             return ops.WeightedRows(y, pair_slot, wts, top, T)
         shared = self.shared.forward(x, ctx, tag="ffn_shared") if self.shared is not None else None
         out = ws.get("ffn_out", T, self.hidden_size, self.dtype)
-        ops.moe_combine(out, y, pair_slot, wts, shared, T, top)
+        more = {"ids": ids, "first_identity": E, "x": x} if self.identity else {}
+        ops.moe_combine(out, y, pair_slot, wts, shared, T, top, shared_gate=gate, **more)
         return out
 
 
