@@ -522,9 +522,32 @@ NIDORAX_SIZES = {
 }
 
 
+def kepevik_config(width, repeats, heads, kv_heads, dim, lstm_heads, lstm_dim, lstm_vdim, delta_heads, delta_kv, ff, experts, top,
+                   expert_ff, shared_ff, vocab=32000):
+    """Layers alternate between the matrix memory with a dense feed-forward and attention beside the channel-decayed delta rule
+    with a routed one (two identity experts, a gated shared expert)."""
+    lstm = {"heads": lstm_heads, "dim": lstm_dim, "vdim": lstm_vdim, "gate_cap": 15.0}
+    par = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"dims": dim // 2, "base": 1e6}},
+           "right": {"heads": delta_heads, "kv_heads": delta_kv, "dim": dim, "vdim": dim, "conv": 4},
+           "left_scale": 0.8, "right_scale": 0.9}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "identity": 2, "top": top}, "shared": {"ff": shared_ff}}
+    ls = [{"type": "mlstm", "mixer": lstm, "mlp": {"kind": "dense", "ff": ff}}, {"type": "parallel", "mixer": par, "mlp": moe}] * repeats
+    return {"architecture": "Kepevik", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "embedding": {"scale": 4.0}, "layers": ls,
+            "max_position": 4096}
+
+
+# name -> (Kepevik config, Potipel config of the same width, depth, heads and experts: the design here that also sets attention beside
+# a delta rule and routes every other feed-forward; Kepevik's dense feed-forward is not gated and half as wide again)
+KEPEVIK_SIZES = {
+    "2048": (kepevik_config(2048, 4, 16, 4, 128, 16, 128, 128, 8, 4, 8448, 16, 4, 1408, 1408), POTIPEL_SIZES["2048"][0]),
+    "4096": (kepevik_config(4096, 2, 32, 8, 128, 16, 128, 256, 16, 8, 16512, 32, 4, 2752, 2752), POTIPEL_SIZES["4096"][0]),
+    "1024-head64": (kepevik_config(1024, 4, 16, 4, 64, 16, 64, 64, 8, 4, 4224, 8, 2, 1408, 1408), POTIPEL_SIZES["1024-head64"][0]),
+}
+
+
 def design_comparison(args, peaks, design: str = "tevudra") -> int:
     """Prefill and decode throughput of a design (Tevudra, Fopivik or Norusun) beside Llama at equal layer sizes, of Potipel
-    beside Fopivik, or of Nidorax beside Tevudra (random weights, bfloat16), with the device time of every kernel of one prompt step and one decode step.
+    beside Fopivik, of Nidorax beside Tevudra, or of Kepevik beside Potipel (random weights, bfloat16), with the device time of every kernel of one prompt step and one decode step.
     One JSON line per size."""
     import collections
 
@@ -613,8 +636,9 @@ def design_comparison(args, peaks, design: str = "tevudra") -> int:
         torch.cuda.empty_cache()
         return out
 
-    table = {"fopivik": FOPIVIK_SIZES, "norusun": NORUSUN_SIZES, "potipel": POTIPEL_SIZES, "nidorax": NIDORAX_SIZES}.get(design, DESIGN_SIZES)
-    beside = {"potipel": "fopivik", "nidorax": "tevudra"}.get(design, "llama")
+    table = {"fopivik": FOPIVIK_SIZES, "norusun": NORUSUN_SIZES, "potipel": POTIPEL_SIZES, "nidorax": NIDORAX_SIZES,
+             "kepevik": KEPEVIK_SIZES}.get(design, DESIGN_SIZES)
+    beside = {"potipel": "fopivik", "nidorax": "tevudra", "kepevik": "potipel"}.get(design, "llama")
     sizes = [s for s in table if not args.sizes or s in args.sizes.split(",")]
     for name in sizes:
         tev, lla = table[name]
@@ -640,16 +664,16 @@ def main() -> int:
                     help="skip the runs at the Llama-2-7B and Llama-3-8B shapes, the many-request load and the 32-bit check")
     ap.add_argument("--mode", default="all",
                     choices=["all", "decode", "prefill", "timeline", "timeline_prefill", "decode_attention", "tevudra", "fopivik", "norusun",
-                             "potipel", "nidorax"],
+                             "potipel", "nidorax", "kepevik"],
                     help="decode / prefill: only that measurement, for small profiling runs (not the benchmark line); "
                          "timeline: the kernels of one decode layer with their start and end inside the step's CUDA graph; "
                          "decode_attention: the decode attention kernel alone over batches and context lengths "
                          "(--batch with --ctx: that one case); "
                          "tevudra, fopivik, norusun: that design beside Llama at equal layer sizes, prompt and decode, with every kernel's time; "
-                         "potipel: the same beside Fopivik; nidorax: beside Tevudra")
+                         "potipel: the same beside Fopivik; nidorax: beside Tevudra; kepevik: beside Potipel")
     ap.add_argument("--latent", action="store_true", help="decode_attention: the key pages are the value pages too")
     ap.add_argument("--head-parts", type=int, default=1, help="decode_attention: CTAs that the query heads of a kv head are split over")
-    ap.add_argument("--sizes", default="", help="tevudra, fopivik, norusun, potipel, nidorax: which of the sizes to run (comma-separated; default all)")
+    ap.add_argument("--sizes", default="", help="tevudra, fopivik, norusun, potipel, nidorax, kepevik: which of the sizes to run (comma-separated; default all)")
     ap.add_argument("--ctx", type=int, default=0, help="decode_attention: the context length of the one case to run")
     ap.add_argument("--prompt-tokens", type=int, default=PREFILL_TOKENS, help="timeline_prefill: tokens of the prompt step")
     ap.add_argument("--heads", default="32,4,64", help="decode_attention: query heads, kv heads, head size")
@@ -672,7 +696,7 @@ def main() -> int:
     peaks = load_peaks()
     if args.mode == "decode_attention":
         return decode_attention_sweep(args, peaks, torch, ops)
-    if args.mode in ("tevudra", "fopivik", "norusun", "potipel", "nidorax"):
+    if args.mode in ("tevudra", "fopivik", "norusun", "potipel", "nidorax", "kepevik"):
         return design_comparison(args, peaks, args.mode)
     cfg = dict(MODEL, num_hidden_layers=args.layers)
     if args.mode != "all":
