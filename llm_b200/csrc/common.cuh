@@ -128,6 +128,31 @@ template <> struct Vec8<__nv_bfloat16> {
   }
 };
 
+// Four consecutive elements as float32 (one 16-byte access of float32, one of 8 bytes of bfloat16).
+template <typename T> struct Vec4;
+template <> struct Vec4<float> {
+  static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  }
+  static __device__ __forceinline__ void store(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+};
+template <> struct Vec4<__nv_bfloat16> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[4]) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) { v[2 * i] = __low2float(h[i]); v[2 * i + 1] = __high2float(h[i]); }
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[4]) {
+    uint2 u;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    *reinterpret_cast<uint2*>(p) = u;
+  }
+};
+
 // A value that is either an element of a tensor of T or the sum, in the order s = 0, 1, ...,
 // of `splits` float32 partial results laid out [split][row][col] (split-K products).
 template <typename T>
@@ -176,6 +201,31 @@ struct MaybePartial {
       return;
     }
     Vec8<T>::load(direct + idx, v);
+  }
+  // four consecutive values starting at idx (idx a multiple of 4, the bases 16-byte aligned)
+  __device__ __forceinline__ void at4(size_t idx, float (&v)[4]) const {
+    if (parts) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[i] = 0.f;
+      int s = 0;
+      for (; s + 4 <= splits; s += 4) {              // the loads of four splits in flight, sums in split order
+        float t[4][4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) Vec4<float>::load(parts + (size_t)(s + u) * split_stride + idx, t[u]);
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) v[i] += t[u][i];
+      }
+      for (; s < splits; ++s) {
+        float t[4];
+        Vec4<float>::load(parts + (size_t)s * split_stride + idx, t);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[i] += t[i];
+      }
+      return;
+    }
+    Vec4<T>::load(direct + idx, v);
   }
   __host__ bool vector_ok() const {
     return ((uintptr_t)direct % 16 == 0) && ((uintptr_t)parts % 16 == 0) && (split_stride % 4 == 0);

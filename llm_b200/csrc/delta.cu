@@ -328,7 +328,7 @@ __device__ __forceinline__ bool chunk_of(const int* cu_tokens, int n_entries, in
 }
 
 template <typename T, bool CH>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, CH ? 2 : 1)
 delta_prepare_kernel(PrepArgs a) {
   extern __shared__ __align__(16) float smem[];
   pdl_launch_dependents();

@@ -650,6 +650,7 @@ struct RopeStore {
   __nv_bfloat16* v_pages;
   int n_heads, n_kv, head_dim, page_size;
   int act_plus1;      // EPI_PLAIN only: 0 = store the product; else activation act_plus1 - 1 (see epilogue_act) on the accumulator
+  const float* bias;  // EPI_PLAIN with an activation only: added to the accumulator before it (float32 [N] or null)
 };
 enum : int { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_ROPE = 2 };
 
@@ -818,6 +819,10 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_cons
 #pragma unroll
               for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
               if (rs.act_plus1) {
+                if (rs.bias) {                   // every lane of the warp reads the same numbers
+#pragma unroll
+                  for (int j = 0; j < 32; ++j) v[j] += q0 + c + j < N ? __ldg(rs.bias + q0 + c + j) : 0.f;
+                }
 #pragma unroll
                 for (int j = 0; j < 32; ++j) v[j] = epilogue_act(v[j], rs.act_plus1 - 1);
               }
@@ -1169,6 +1174,25 @@ LLMK_API int llmk_gemm_tc(const void* A, const void* W, void* C, int M, int N, i
   if (out_dtype == LLMK_F32) return launch_out<float>(swap != 0, tile, cluster != 0, mp, mq, C, ldc, split_stride, M, N, K, splits, kblocks_per_split, stream);
   if (out_dtype == LLMK_BF16) return launch_out<__nv_bfloat16>(swap != 0, tile, cluster != 0, mp, mq, C, ldc, split_stride, M, N, K, splits, kblocks_per_split, stream);
   return llmk_fail(-1, "gemm_tc: unsupported output kind %d", out_dtype);
+}
+
+// C [M, N] (bfloat16) = act(A W^T + bias) with the pair kernel: bias float32 [N], act 0..3 (see epilogue_act), tile a multiple of
+// 32 up to 256.
+LLMK_API int llmk_gemm_tc_bias_act(const void* A, const void* W, void* C, const float* bias, int M, int N, int K, long long lda,
+                                   long long ldw, long long ldc, int tile, int act, cudaStream_t stream) {
+  if (M == 0 || N == 0) return 0;
+  LLMK_REQUIRE(bias != nullptr && act >= 0 && act <= 3, "gemm_tc_bias_act: no bias, or an activation that is not one of 0..3");
+  LLMK_REQUIRE(tile % 32 == 0 && tile >= 32 && tile <= 256, "gemm_tc_bias_act: a tile of 32..256 in steps of 32, not %d", tile);
+  LLMK_REQUIRE(llmk_gemm_tc_supported(A, W, M, N, K, lda, ldw), "gemm_tc_bias_act: K=%d and the row pitches must be multiples of 8 and the bases 16-byte aligned", K);
+  int rc = ensure_err_flag();
+  if (rc) return rc;
+  CUtensorMap mp, mq;
+  if ((rc = get_map(&mp, A, M, K, lda, BP))) return rc;
+  if ((rc = get_map(&mq, W, N, K, ldw, tile / 2))) return rc;
+  RopeStore plain{};
+  plain.act_plus1 = act + 1;
+  plain.bias = bias;
+  return launch_pair<__nv_bfloat16, EPI_PLAIN>(mp, mq, C, ldc, M, N, K, tile, plain, stream);
 }
 
 // Several products in one launch of the one-tile kernel (see Grouping).  A and W bfloat16.

@@ -46,17 +46,20 @@ struct State {
 // ---- single tokens -----------------------------------------------------------------------------------------
 constexpr int DEC_TX = COLS / 4, DEC_ROWS = 8, DEC_THREADS = DEC_TX * DEC_ROWS, DEC_BATCH = 16, DEC_MAX_DIM = 512;
 
-// proj row e: [q: heads * dim | k: heads * dim | v: heads * vdim | .. | at gate_col: i: heads | f: heads].
+// proj row e: [q: heads * dim | k: heads * dim | v: heads * vdim | .. | at gate_col: i: heads | f: heads].  What the CTA needs of it
+// is summed into shared memory first, every load of the partial results in flight at once (VEC: four columns a thread; dim and
+// proj_stride on the 4-grid), under the loads of the state's first rows.
+template <bool VEC>
 __global__ void __launch_bounds__(DEC_THREADS)
 mlstm_decode_kernel(float* __restrict__ out, long long out_stride, MaybePartial<float> proj, long long proj_stride, long long gate_col,
                     Gates gt, State st, int heads, int dim, int vdim) {
-  __shared__ float q_s[DEC_MAX_DIM], k_s[DEC_MAX_DIM];
+  __shared__ __align__(16) float q_s[DEC_MAX_DIM], k_s[DEC_MAX_DIM], v_s[COLS], z_s[2];
   __shared__ float4 part[DEC_ROWS][DEC_TX];
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
   const int tid = threadIdx.x, tx = tid % DEC_TX, ty = tid / DEC_TX;
-  const int entry = blockIdx.z, head = blockIdx.y, col = blockIdx.x * COLS + tx * 4;
+  const int entry = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * COLS, col = col0 + tx * 4;
   const size_t row = (size_t)entry * proj_stride;
   const bool live = col < vdim;                           // vdim is a multiple of 4
   float* slot = st.base + (size_t)st.slots[entry] * st.slot_stride;
@@ -72,26 +75,39 @@ mlstm_decode_kernel(float* __restrict__ out, long long out_stride, MaybePartial<
       if (live && r < dim) s[i] = S[(size_t)r * pitch];
     }
   };
-  load(0);                                                // under the sums and the gates below
+  load(0);
   const float m_old = *m_g;
-  const float zi = proj.at(row + gate_col + head) + gt.i_bias[head], zf = proj.at(row + gate_col + heads + head) + gt.f_bias[head];
-  const float gi = soft_cap(zi, gt.cap), gf = log_sigmoid(soft_cap(zf, gt.cap));
+  const size_t q0 = row + (size_t)head * dim, k0 = row + (size_t)(heads + head) * dim, v0 = row + (size_t)2 * heads * dim + (size_t)head * vdim + col0;
+  const int cols = min(COLS, vdim - col0);
+  constexpr int N = VEC ? 4 : 1;
+  // from the last thread down, so that the two gates' sums run beside the vectors'
+  if (tid >= DEC_THREADS - 2) z_s[tid - (DEC_THREADS - 2)] = proj.at(row + gate_col + (tid - (DEC_THREADS - 2)) * heads + head);
+  for (int i = tid; i < (2 * dim + cols) / N; i += DEC_THREADS) {
+    const int e = i * N;
+    float* dst = e < dim ? q_s + e : e < 2 * dim ? k_s + e - dim : v_s + e - 2 * dim;
+    const size_t src = e < dim ? q0 + e : e < 2 * dim ? k0 + e - dim : v0 + e - 2 * dim;
+    if constexpr (VEC) {
+      float v[4];
+      proj.at4(src, v);
+      *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+    } else {
+      *dst = proj.at(src);
+    }
+  }
+  __syncthreads();
+  const float gi = soft_cap(z_s[0] + gt.i_bias[head], gt.cap), gf = log_sigmoid(soft_cap(z_s[1] + gt.f_bias[head], gt.cap));
   const float m = fmaxf(gf + m_old, gi), keep = expf(gf + m_old - m), write = expf(gi - m);
   float nq = 0.f;
   for (int d = tid; d < dim; d += DEC_THREADS) {
-    const float qd = proj.at(row + (size_t)head * dim + d) * gt.q_scale;
-    const float kd = proj.at(row + (size_t)(heads + head) * dim + d) * write;
-    q_s[d] = qd;
-    k_s[d] = kd;
-    const float nd = fmaf(keep, n_g[d], kd);
+    const float nd = fmaf(keep, n_g[d], k_s[d] * write);
     n_g[d] = nd;
-    nq = fmaf(nd, qd, nq);
+    nq = fmaf(nd, q_s[d], nq);
   }
   float v[4] = {0.f, 0.f, 0.f, 0.f};
-  if (live)
-#pragma unroll
-    for (int c = 0; c < 4; ++c) v[c] = proj.at(row + (size_t)2 * heads * dim + (size_t)head * vdim + col + c);
-  nq = block_sum(nq, red);                                // its barriers also stand between q_s, k_s and their readers
+  if (live) {
+    const float4 v4 = *reinterpret_cast<const float4*>(v_s + 4 * tx);
+    v[0] = v4.x * write; v[1] = v4.y * write; v[2] = v4.z * write; v[3] = v4.w * write;
+  }
   float o[4] = {0.f, 0.f, 0.f, 0.f};
   for (int r0 = 0; r0 < dim; r0 += DEC_BATCH * DEC_ROWS) {
     if (r0) load(r0);
@@ -108,7 +124,7 @@ mlstm_decode_kernel(float* __restrict__ out, long long out_stride, MaybePartial<
     }
   }
   part[ty][tx] = make_float4(o[0], o[1], o[2], o[3]);
-  __syncthreads();
+  nq = block_sum(nq, red) * gt.q_scale;                   // its barriers also stand between part and its readers
   if (tid == 0) *m_g = m;                                 // every thread has read the old one
   if (ty == 0 && live) {
     float4 a = part[0][tx];
@@ -117,9 +133,9 @@ mlstm_decode_kernel(float* __restrict__ out, long long out_stride, MaybePartial<
       const float4 b = part[g][tx];
       a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
     }
-    const float den = fmaxf(fabsf(nq), expf(-m)) + DENOM_EPS;
+    const float f = gt.q_scale / (fmaxf(fabsf(nq), expf(-m)) + DENOM_EPS);
     float* dst = out + (size_t)entry * out_stride + (size_t)head * vdim + col;
-    dst[0] = a.x / den; dst[1] = a.y / den; dst[2] = a.z / den; dst[3] = a.w / den;
+    dst[0] = a.x * f; dst[1] = a.y * f; dst[2] = a.z * f; dst[3] = a.w * f;
   }
 }
 
@@ -645,8 +661,9 @@ LLMK_API int llmk_mlstm_scan(float* out, long long out_stride, const float* proj
                  DEC_MAX_DIM, vdim);
     LLMK_REQUIRE(slot_stride % 4 == 0 && (uintptr_t)state % 16 == 0, "mlstm_decode: the state must lie on the 16-byte grid");
     const MaybePartial<float> p{proj, partials, splits, split_stride};
-    launch_kernel(mlstm_decode_kernel, grid, dim3(DEC_THREADS), 0, stream, out, out_stride, p, proj_stride, gate_col, gt, st, heads, dim,
-                  vdim);
+    const bool vec = dim % 4 == 0 && proj_stride % 4 == 0 && p.vector_ok();
+    launch_kernel(vec ? mlstm_decode_kernel<true> : mlstm_decode_kernel<false>, grid, dim3(DEC_THREADS), 0, stream, out, out_stride, p,
+                  proj_stride, gate_col, gt, st, heads, dim, vdim);
     LLMK_LAUNCH_CHECK("mlstm_decode");
   }
   LLMK_REQUIRE(proj != nullptr, "mlstm_scan: partial results are for single tokens");

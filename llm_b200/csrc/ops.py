@@ -42,13 +42,23 @@ class BiasedRows:
         self.rows, self.bias = rows, bias
 
 
+class ScaledPair:
+    """sa * a + sb * b, still to be summed by the kernel that reads it; a and b tensors or PartialSums."""
+
+    def __init__(self, a, b, sa: float, sb: float):
+        self.a, self.b, self.sa, self.sb = a, b, sa, sb
+
+
 class WeightedRows:
     """The result of a routed feed-forward before its last sum: row t is sum_j weights[t, j] * y[pair_slot[t, j]] for y
     float32 [slots, cols] (a slot of -1 counts nothing).  The norm behind the residual sum takes it as it is (sum_rmsnorm);
-    the buffers are valid until the next routed feed-forward runs."""
+    the buffers are valid until the next routed feed-forward runs.  Further terms, which add_rmsnorms takes too: choices with
+    ids[t, j] >= first_identity count x[t]; shared[t] (a tensor or a PartialSum) times shared_gate[t], if given."""
 
-    def __init__(self, y: torch.Tensor, pair_slot: torch.Tensor, weights: torch.Tensor, top: int, rows: int):
+    def __init__(self, y: torch.Tensor, pair_slot: torch.Tensor, weights: torch.Tensor, top: int, rows: int, shared=None,
+                 shared_gate=None, ids=None, first_identity: int = 0, x=None):
         self.y, self.pair_slot, self.weights, self.top, self.rows = y, pair_slot, weights, top, rows
+        self.shared, self.shared_gate, self.ids, self.first_identity, self.x = shared, shared_gate, ids, first_identity, x
 
 
 def _split_args(x):
@@ -171,6 +181,7 @@ def sum_rmsnorm(resid: torch.Tensor, alpha: float, y, gain: torch.Tensor, out, r
     wy = slots = weights = None
     top = 0
     if isinstance(y, WeightedRows):
+        assert y.shared is None and y.ids is None
         wy, slots, weights, top = y.y, y.pair_slot, y.weights, y.top
         assert wy.dtype == weights.dtype == torch.float32 and slots.dtype == torch.int32 and wy.is_contiguous() and wy.shape[1] == hidden
         assert slots.is_contiguous() and weights.is_contiguous() and slots.numel() >= rows * top and weights.numel() >= rows * top
@@ -247,27 +258,51 @@ def add_layernorm(resid: torch.Tensor, delta, post, mult: float, pre, out, rows:
                                      c_int(rows), c_int(hidden), c_float(eps), c_int(_kind(ref.dtype)), _stream()))
 
 
-def add_rmsnorms(resid: torch.Tensor, delta, post, mult: float, pre, out, rows: int, eps: float, delta_bias=None) -> None:
-    """RMS norms on both sides of the residual sum: resid[:rows] += mult * rms(delta + delta_bias) * post where delta (a tensor
-    or a PartialSum) is given (post None: mult * delta); out[:rows] = rms(resid) * pre where out is given.  delta_bias: float32
-    [hidden] or None."""
+def add_rmsnorms(resid: torch.Tensor, delta, post, mult: float, pre, out, rows: int, eps: float, dtype: torch.dtype = None) -> None:
+    """RMS norms on both sides of the residual sum (sandwich.cu): resid[:rows] += mult * rms(delta) * post where delta is given
+    (post None: mult * delta); out[:rows] = rms(resid) * pre where out is given.  delta: a tensor, a PartialSum, BiasedRows, a
+    ScaledPair or WeightedRows.  dtype: the compute dtype (default: out's or delta's)."""
     assert resid.dtype == torch.float32 and resid.is_contiguous()
     hidden = resid.shape[-1]
-    ref = out if out is not None else delta
-    if ref is None:
-        return
-    for w in (post, pre, delta_bias):
+    for w in (post, pre):
         assert w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == hidden)
-    if isinstance(delta, PartialSum):
-        assert delta.cols == hidden and delta.rows == rows
-    elif delta is not None:
-        assert delta.is_contiguous() and delta.shape[-1] == hidden
+    a = b = bias = gate = wr = None
+    sa = sb = 1.0
+    if isinstance(delta, BiasedRows):
+        a, bias = delta.rows, delta.bias
+        assert bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == hidden
+    elif isinstance(delta, ScaledPair):
+        a, b, sa, sb = delta.a, delta.b, delta.sa, delta.sb
+        assert not (isinstance(a, PartialSum) and isinstance(b, PartialSum))      # they would share one buffer
+    elif isinstance(delta, WeightedRows):
+        wr, b, gate = delta, delta.shared, delta.shared_gate
+        assert wr.y.dtype == wr.weights.dtype == torch.float32 and wr.pair_slot.dtype == torch.int32 and wr.y.is_contiguous()
+        assert wr.y.shape[1] == hidden and wr.pair_slot.numel() >= rows * wr.top and wr.weights.numel() >= rows * wr.top
+        assert gate is None or (b is not None and gate.dtype == torch.float32 and gate.is_contiguous() and gate.numel() >= rows)
+        if wr.ids is not None:
+            _rows_contig(wr.x, "x")
+            assert wr.ids.dtype == torch.int32 and wr.ids.numel() >= rows * wr.top and wr.x.shape[1] == hidden
+    else:
+        a = delta
+    for t in (a, b):
+        if isinstance(t, PartialSum):
+            assert t.cols == hidden and t.rows == rows
+        elif t is not None:
+            assert t.is_contiguous() and t.shape[-1] == hidden
     if out is not None:
         assert pre is not None and out.is_contiguous() and out.shape[-1] == hidden
-        assert delta is None or delta.dtype == out.dtype
-    d, parts, splits, stride = _split_args(delta)
-    _check(load().llmk_add_rmsnorms(_ptr(resid), d, parts, splits, stride, _ptr(delta_bias), _ptr(post), c_float(mult), _ptr(pre),
-                                    _ptr(out), c_int(rows), c_int(hidden), c_float(eps), c_int(_kind(ref.dtype)), _stream()))
+    kinds = {t.dtype for t in (out, a, b, wr.x if wr is not None else None) if t is not None}
+    if dtype is not None:
+        kinds.add(dtype)
+    if delta is None and out is None:
+        return
+    assert len(kinds) <= 1
+    weighted = ((_ptr(wr.y), _ptr(wr.pair_slot), _ptr(wr.weights), c_int(wr.top), _ptr(wr.ids), c_int(wr.first_identity), _ptr(wr.x),
+                 c_longlong(wr.x.stride(0) if wr.x is not None else 0)) if wr is not None else
+                (c_void_p(0), c_void_p(0), c_void_p(0), c_int(0), c_void_p(0), c_int(0), c_void_p(0), c_longlong(0)))
+    _check(load().llmk_sandwich_norms(_ptr(resid), *_split_args(a), c_float(sa), _ptr(bias), *_split_args(b), c_float(sb), _ptr(gate),
+                                      *weighted, _ptr(post), c_float(mult), _ptr(pre), _ptr(out), c_int(rows), c_int(hidden), c_float(eps),
+                                      c_int(_kind(kinds.pop() if kinds else torch.float32)), _stream()))
 
 
 def softcap(x: torch.Tensor, rows: int, cap: float) -> None:
@@ -1887,8 +1922,8 @@ def gemm_act_available(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, rows
     return PAIR_GEMM and rows > 128 and out.dtype == torch.bfloat16 and gemm_fast_available(a, w, out, rows)
 
 
-def gemm_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, rows: int, act: str) -> None:
-    """out[:rows] = act(a[:rows] @ w.T) with the activation applied to the float32 accumulator in the epilogue of
+def gemm_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, rows: int, act: str, bias=None) -> None:
+    """out[:rows] = act(a[:rows] @ w.T (+ bias, float32 [out features])) with the activation applied to the float32 accumulator in the epilogue of
     the pair kernel, so the product itself never reaches memory."""
     _rows_contig(a, "a"); _rows_contig(w, "w"); _rows_contig(out, "out")
     n, k = w.shape
@@ -1897,6 +1932,12 @@ def gemm_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, rows: int, act
         raise KernelError(f"gemm_act does not take {rows} rows of {a.dtype} -> {out.dtype}")
     tile = 256 if n % 256 == 0 or n % 256 > 128 or n < 128 else 128
     tile = min(tile, _ceil_div(n, 32) * 32)
+    if bias is not None:
+        assert bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == n
+        _check_t(load_tensor().llmk_gemm_tc_bias_act(_ptr(a), _ptr(w), _ptr(out), _ptr(bias), c_int(rows), c_int(n), c_int(k),
+                                                     c_longlong(a.stride(0)), c_longlong(w.stride(0)), c_longlong(out.stride(0)),
+                                                     c_int(tile), c_int(ACTIVATIONS[act]), _stream()))
+        return
     _check_t(load_tensor().llmk_gemm_tc(_ptr(a), _ptr(w), _ptr(out), c_int(rows), c_int(n), c_int(k),
                                c_longlong(a.stride(0)), c_longlong(w.stride(0)), c_longlong(out.stride(0)),
                                c_int(_BF16), c_int(0), c_int(tile), c_int(1), c_int(_ceil_div(k, 64)),

@@ -244,6 +244,76 @@ norm_rope_kv_write_kernel(MaybePartial<T> src, long long src_stride, T* __restri
   }
 }
 
+// ---- the same without norms: rotation, store ------------------------------------------------------------------
+// Nothing ties a token's heads together, so a warp takes a head (query heads, then key heads, then value heads) and the heads of a
+// token may be spread over CTAs (gridDim.y) where there are few tokens.  The angles' sines and cosines are made once per CTA in
+// shared memory.  VEC: four channels a lane (rot_pairs, dim, vdim and every row on the 4-grid).
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+rope_kv_store_kernel(MaybePartial<T> src, long long src_stride, T* q_out, long long q_out_stride, const float* __restrict__ freqs,
+                     int rot_pairs, int halves, const int* __restrict__ positions, const int* __restrict__ slot_map,
+                     T* __restrict__ k_pages, T* __restrict__ v_pages, int n_heads, int n_kv, int dim, int vdim, int page_size,
+                     float amp, int v_from_k) {
+  extern __shared__ float2 turn_s[];          // [rot_pairs]: cosine, sine
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const float pos = (float)positions[t];
+  for (int i = threadIdx.x; i < rot_pairs; i += blockDim.x) {
+    float sn, cs;
+    sincosf(pos * freqs[i], &sn, &cs);
+    turn_s[i] = make_float2(cs * amp, sn * amp);
+  }
+  __syncthreads();
+  size_t page = 0, off = 0;
+  if (n_kv) {
+    const int slot = slot_map[t];
+    page = slot / page_size; off = slot % page_size;
+  }
+  const size_t row = (size_t)t * src_stride;
+  constexpr int N = VEC ? 4 : 1;
+  const int heads = n_heads + n_kv * (v_from_k ? 1 : 2);
+  for (int head = blockIdx.y * warps + (threadIdx.x >> 5); head < heads; head += gridDim.y * warps) {
+    const bool is_q = head < n_heads, is_v = head >= n_heads + n_kv;
+    const int g = is_q ? 0 : (head - n_heads) % n_kv, width = is_v ? vdim : dim;
+    const size_t c0 = row + (is_v ? (size_t)(n_heads + n_kv) * dim + (size_t)g * vdim : (size_t)head * dim);
+    const size_t place = (page * n_kv + g) * page_size + off;
+    T* dst = is_q ? q_out + (size_t)t * q_out_stride + (size_t)head * dim : is_v ? v_pages + place * vdim : k_pages + place * dim;
+    T* raw = !is_q && !is_v && v_from_k ? v_pages + place * dim : nullptr;      // the key before it turns, as the value
+    auto load = [&](int d, float (&v)[N]) { if constexpr (VEC) src.at4(c0 + d, v); else v[0] = src.at(c0 + d); };
+    auto store = [&](T* p, const float (&v)[N]) { if constexpr (VEC) Vec4<T>::store(p, v); else *p = from_f32<T>(v[0]); };
+    const int pairs = is_v ? 0 : rot_pairs;
+    if (halves) {
+      for (int i = lane * N; i < pairs; i += 32 * N) {
+        float u[N], w[N], a[N], b[N];
+        load(i, u); load(i + pairs, w);
+#pragma unroll
+        for (int x = 0; x < N; ++x) {
+          const float2 cs = turn_s[i + x];
+          a[x] = u[x] * cs.x - w[x] * cs.y;
+          b[x] = w[x] * cs.x + u[x] * cs.y;
+        }
+        if (raw) { store(raw + i, u); store(raw + i + pairs, w); }
+        store(dst + i, a); store(dst + i + pairs, b);
+      }
+    } else {
+      for (int i = lane; i < pairs; i += 32) {
+        const float u = src.at(c0 + 2 * i), w = src.at(c0 + 2 * i + 1);
+        const float2 cs = turn_s[i];
+        if (raw) { raw[2 * i] = from_f32<T>(u); raw[2 * i + 1] = from_f32<T>(w); }
+        dst[2 * i] = from_f32<T>(u * cs.x - w * cs.y);
+        dst[2 * i + 1] = from_f32<T>(w * cs.x + u * cs.y);
+      }
+    }
+    for (int d = 2 * pairs + lane * N; d < width; d += 32 * N) {
+      float v[N];
+      load(d, v);
+      if (raw) store(raw + d, v);
+      store(dst + d, v);
+    }
+  }
+}
+
 // ---- norm per head with one shared weight, store; k and v with head counts of their own ----------------------
 // A row holds n_q query heads and n_k key heads of dim numbers, then n_v value heads of vdim.  Every q and k head is
 // divided by its own root mean square (eps inside the root) and multiplied by gain [dim], one weight vector for all of them
@@ -322,10 +392,20 @@ LLMK_API int llmk_norm_rope_kv_write(const void* qkv, const float* partials, int
   LLMK_REQUIRE(rot_pairs == 0 || freqs != nullptr, "norm_rope_kv_write: frequencies are missing");
   LLMK_REQUIRE(!v_from_k || vdim == dim, "norm_rope_kv_write: keys that are values have one size, not %d and %d", dim, vdim);
   const size_t smem = (size_t)(n_heads + n_kv) * dim * sizeof(float);
-  LLMK_REQUIRE(smem <= 200 * 1024, "norm_rope_kv_write: a projection of %d numbers does not fit shared memory", (n_heads + n_kv) * dim);
+  LLMK_REQUIRE(smem <= 200 * 1024 || (!q_gain && !k_gain), "norm_rope_kv_write: a projection of %d numbers does not fit shared memory", (n_heads + n_kv) * dim);
   return dispatch_dtype(dtype, [&](auto* tag) {
     using T = LLMK_ELEM(tag);
     MaybePartial<T> src{(const T*)qkv, partials, splits, split_stride};
+    if (!q_gain && !k_gain) {
+      const bool vec = rot_pairs % 4 == 0 && dim % 4 == 0 && vdim % 4 == 0 && src_stride % 4 == 0 && q_out_stride % 4 == 0 &&
+                       src.vector_ok() && (uintptr_t)q_out % 16 == 0 && (uintptr_t)k_pages % 16 == 0 && (uintptr_t)v_pages % 16 == 0;
+      const int heads = n_heads + n_kv * (v_from_k ? 1 : 2);
+      const dim3 grid(n_tokens, n_tokens <= 128 ? (heads + 7) / 8 : 1);
+      launch_kernel(vec ? rope_kv_store_kernel<T, true> : rope_kv_store_kernel<T, false>, grid, dim3(256), (size_t)rot_pairs * sizeof(float2),
+                    stream, src, src_stride, (T*)q_out, q_out_stride, freqs, rot_pairs, halves, positions, slot_map, (T*)k_pages,
+                    (T*)v_pages, n_heads, n_kv, dim, vdim, page_size, amp, v_from_k);
+      LLMK_LAUNCH_CHECK("rope_kv_store");
+    }
     if (smem > 48 * 1024)
       cudaFuncSetAttribute(norm_rope_kv_write_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_kernel(norm_rope_kv_write_kernel<T>, dim3(n_tokens), dim3(256), smem, stream, src, src_stride, (T*)q_out,

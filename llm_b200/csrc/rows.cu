@@ -544,41 +544,42 @@ __global__ void act_rows8_kernel(T* __restrict__ out, MaybePartial<T> in, int ki
 }
 
 // out = act(in + bias[column]) over rows of `cols` elements: the activation behind a biased projection, the bias added to the
-// float32 sum.  VEC: eight columns a thread.
+// float32 sum.  blockIdx.y is a row; VEC: eight columns a thread.
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
-bias_act_rows_kernel(T* __restrict__ out, MaybePartial<T> in, const float* __restrict__ bias, int kind, int cols, size_t total) {
+bias_act_rows_kernel(T* __restrict__ out, MaybePartial<T> in, const float* __restrict__ bias, int kind, int cols, int rows) {
   pdl_launch_dependents();
   pdl_wait();
-  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
-    if (VEC) {
-      float v[8], b[8];
-      in.at8(i * 8, v);
-      Vec8<float>::load(bias + (i * 8) % cols, b);
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * (VEC ? 8 : 1);
+  if (c >= cols) return;
+  float b[VEC ? 8 : 1];
+  if constexpr (VEC) Vec8<float>::load(bias + c, b); else b[0] = bias[c];
+  for (int t = blockIdx.y; t < rows; t += gridDim.y) {
+    const size_t i = (size_t)t * cols + c;
+    if constexpr (VEC) {
+      float v[8];
+      in.at8(i, v);
 #pragma unroll
       for (int k = 0; k < 8; ++k) v[k] = apply_act(v[k] + b[k], kind);
-      Vec8<T>::store(out + i * 8, v);
+      Vec8<T>::store(out + i, v);
     } else {
-      out[i] = from_f32<T>(apply_act(in.at(i) + bias[i % cols], kind));
+      out[i] = from_f32<T>(apply_act(in.at(i) + b[0], kind));
     }
   }
 }
 
 LLMK_API int llmk_bias_act_rows(void* out, const void* in, const float* partials, int splits, long long split_stride,
                                 const float* bias, int rows, int cols, int kind, int dtype, cudaStream_t stream) {
-  const size_t total = (size_t)rows * cols;
-  if (total == 0) return 0;
+  if (rows <= 0 || cols <= 0) return 0;
   LLMK_REQUIRE((in != nullptr) != (partials != nullptr), "bias_act_rows: give in or partials");
   LLMK_REQUIRE(kind >= 0 && kind <= 4 && bias != nullptr, "bias_act_rows: unknown activation %d or no bias", kind);
   return dispatch_dtype(dtype, [&](auto* tag) {
     using T = LLMK_ELEM(tag);
     MaybePartial<T> x{(const T*)in, partials, splits, split_stride};
     const bool vec = cols % 8 == 0 && x.vector_ok() && (uintptr_t)out % 16 == 0 && (uintptr_t)bias % 16 == 0;
-    const size_t n = vec ? total / 8 : total;
-    size_t blocks = (n + 255) / 256;
-    if (blocks > (size_t)llmk_sm_count() * 32) blocks = (size_t)llmk_sm_count() * 32;
-    launch_kernel(vec ? bias_act_rows_kernel<T, true> : bias_act_rows_kernel<T, false>, dim3((unsigned)blocks), dim3(256), 0, stream,
-                  (T*)out, x, bias, kind, cols, n);
+    const dim3 grid((cols + (vec ? 2048 : 256) - 1) / (vec ? 2048 : 256), rows < 4096 ? rows : 4096);
+    launch_kernel(vec ? bias_act_rows_kernel<T, true> : bias_act_rows_kernel<T, false>, grid, dim3(256), 0, stream, (T*)out, x, bias,
+                  kind, cols, rows);
     LLMK_LAUNCH_CHECK("bias_act_rows");
   });
 }
@@ -611,12 +612,11 @@ LLMK_API int llmk_act_rows(void* out, const void* in, const float* partials, int
 //     out    = ln(resid; pre)                (out null: nothing more)
 // with ln(x; w) = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w: a weight, no bias, the
 // variance taken from the deviations (two passes over the row in shared memory).  Both halves are
-// optional, all arithmetic is float32, and a row is read from memory once.  RMS: the mean is left out, ln(x; w) becomes
-// x / sqrt(mean(x^2) + eps) * w.  dbias (or null) is added to delta's rows first: the bias of the product that made them.
-template <typename T, bool RMS>
+// optional, all arithmetic is float32, and a row is read from memory once.
+template <typename T>
 __global__ void __launch_bounds__(256)
-add_layernorm_kernel(float* __restrict__ resid, MaybePartial<T> delta, const float* __restrict__ dbias, const float* __restrict__ post,
-                     float mult, const float* __restrict__ pre, T* __restrict__ out, int hidden, float eps) {
+add_layernorm_kernel(float* __restrict__ resid, MaybePartial<T> delta, const float* __restrict__ post, float mult,
+                     const float* __restrict__ pre, T* __restrict__ out, int hidden, float eps) {
   extern __shared__ float row_s[];
   __shared__ float scratch[32];
   pdl_launch_dependents();
@@ -626,13 +626,13 @@ add_layernorm_kernel(float* __restrict__ resid, MaybePartial<T> delta, const flo
   if (delta.present()) {
     float s = 0.f;
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-      const float v = delta.at(base + c) + (dbias ? dbias[c] : 0.f);
+      const float v = delta.at(base + c);
       row_s[c] = v;
       s += v;
     }
     float mean = 0.f, rstd = 1.f;
     if (post) {
-      if (!RMS) mean = block_sum(s, scratch) * inv_n;
+      mean = block_sum(s, scratch) * inv_n;
       float q = 0.f;
       for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
         const float d = row_s[c] - mean;
@@ -650,12 +650,9 @@ add_layernorm_kernel(float* __restrict__ resid, MaybePartial<T> delta, const flo
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) row_s[c] = resid[base + c];
   }
   if (!out) return;
-  float mean = 0.f;
-  if (!RMS) {
-    float s = 0.f;
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) s += row_s[c];
-    mean = block_sum(s, scratch) * inv_n;
-  }
+  float s = 0.f;
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x) s += row_s[c];
+  const float mean = block_sum(s, scratch) * inv_n;
   float q = 0.f;
   for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
     const float d = row_s[c] - mean;
@@ -668,10 +665,10 @@ add_layernorm_kernel(float* __restrict__ resid, MaybePartial<T> delta, const flo
 
 // The same for rows of up to NV * 2048 elements on the 8-grid: the row stays in registers (NV vectors of eight per
 // thread), every access is 16 bytes wide, and the statistics are the same two passes (mean, then squared deviations).
-template <typename T, int NV, bool RMS>
+template <typename T, int NV>
 __global__ void __launch_bounds__(256)
-add_layernorm_vec_kernel(float* __restrict__ resid, MaybePartial<T> delta, const float* __restrict__ dbias, const float* __restrict__ post,
-                         float mult, const float* __restrict__ pre, T* __restrict__ out, int hidden, float eps) {
+add_layernorm_vec_kernel(float* __restrict__ resid, MaybePartial<T> delta, const float* __restrict__ post, float mult,
+                         const float* __restrict__ pre, T* __restrict__ out, int hidden, float eps) {
   __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
@@ -686,19 +683,13 @@ add_layernorm_vec_kernel(float* __restrict__ resid, MaybePartial<T> delta, const
       const int c = (v * 256 + threadIdx.x) * 8;
       if (c < hidden) {
         delta.at8(base + c, y[v]);
-        if (dbias) {
-          float b[8];
-          Vec8<float>::load(dbias + c, b);
-#pragma unroll
-          for (int i = 0; i < 8; ++i) y[v][i] += b[i];
-        }
 #pragma unroll
         for (int i = 0; i < 8; ++i) s += y[v][i];
       }
     }
     float mean = 0.f, rstd = 1.f;
     if (post) {
-      if (!RMS) mean = block_sum(s, scratch) * inv_n;
+      mean = block_sum(s, scratch) * inv_n;
       float q = 0.f;
 #pragma unroll
       for (int v = 0; v < NV; ++v) {
@@ -734,18 +725,15 @@ add_layernorm_vec_kernel(float* __restrict__ resid, MaybePartial<T> delta, const
     }
   }
   if (!out) return;
-  float mean = 0.f;
-  if (!RMS) {
-    float s = 0.f;
+  float s = 0.f;
 #pragma unroll
-    for (int v = 0; v < NV; ++v) {
-      if ((v * 256 + threadIdx.x) * 8 < hidden) {
+  for (int v = 0; v < NV; ++v) {
+    if ((v * 256 + threadIdx.x) * 8 < hidden) {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) s += r[v][i];
-      }
+      for (int i = 0; i < 8; ++i) s += r[v][i];
     }
-    mean = block_sum(s, scratch) * inv_n;
   }
+  const float mean = block_sum(s, scratch) * inv_n;
   float q = 0.f;
 #pragma unroll
   for (int v = 0; v < NV; ++v) {
@@ -768,49 +756,34 @@ add_layernorm_vec_kernel(float* __restrict__ resid, MaybePartial<T> delta, const
   }
 }
 
-template <bool RMS>
-static int add_norms(const char* name, float* resid, const void* delta, const float* partials, int splits, long long split_stride,
-                     const float* dbias, const float* post, float mult, const float* pre, void* out, int rows, int hidden, float eps,
-                     int dtype, cudaStream_t stream) {
-  if (rows == 0) return 0;
-  LLMK_REQUIRE(!(delta && partials), "%s: give delta or partials, not both", name);
-  LLMK_REQUIRE(out == nullptr || pre != nullptr, "%s: an output needs its weight", name);
-  const size_t smem = (size_t)hidden * sizeof(float);
-  LLMK_REQUIRE(smem <= 200 * 1024, "%s: rows of %d elements exceed the shared memory", name, hidden);
-  return dispatch_dtype(dtype, [&](auto* tag) {
-    using T = LLMK_ELEM(tag);
-    MaybePartial<T> d{(const T*)delta, partials, splits, split_stride};
-    const bool vec = hidden % 8 == 0 && hidden <= 8192 && d.vector_ok() && (uintptr_t)resid % 16 == 0 && (uintptr_t)post % 16 == 0 &&
-                     (uintptr_t)pre % 16 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)dbias % 16 == 0;
-    if (vec) {
-      auto kernel = hidden <= 2048 ? add_layernorm_vec_kernel<T, 1, RMS> : hidden <= 4096 ? add_layernorm_vec_kernel<T, 2, RMS>
-                                                                                        : add_layernorm_vec_kernel<T, 4, RMS>;
-      launch_kernel(kernel, dim3(rows), dim3(256), 0, stream, resid, d, dbias, post, mult, pre, (T*)out, hidden, eps);
-    } else {
-      if (smem > 48 * 1024)
-        cudaFuncSetAttribute(add_layernorm_kernel<T, RMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      launch_kernel(add_layernorm_kernel<T, RMS>, dim3(rows), dim3(256), smem, stream, resid, d, dbias, post, mult, pre, (T*)out,
-                    hidden, eps);
-    }
-    LLMK_LAUNCH_CHECK(name);
-  });
-}
-
 // delta: [rows, hidden] of the element kind, or float32 partial results, or neither; post, pre: float32
 // [hidden] or null; out: [rows, hidden] of the element kind or null (then pre is not read).
 LLMK_API int llmk_add_layernorm(float* resid, const void* delta, const float* partials, int splits, long long split_stride,
                                 const float* post, float mult, const float* pre, void* out, int rows, int hidden, float eps,
                                 int dtype, cudaStream_t stream) {
-  return add_norms<false>("add_layernorm", resid, delta, partials, splits, split_stride, nullptr, post, mult, pre, out, rows, hidden,
-                          eps, dtype, stream);
-}
-
-// The same with RMS norms, and a bias (float32 [hidden] or null) added to delta's rows before the first.
-LLMK_API int llmk_add_rmsnorms(float* resid, const void* delta, const float* partials, int splits, long long split_stride,
-                               const float* dbias, const float* post, float mult, const float* pre, void* out, int rows, int hidden,
-                               float eps, int dtype, cudaStream_t stream) {
-  return add_norms<true>("add_rmsnorms", resid, delta, partials, splits, split_stride, dbias, post, mult, pre, out, rows, hidden, eps,
-                         dtype, stream);
+  if (rows == 0) return 0;
+  LLMK_REQUIRE(!(delta && partials), "add_layernorm: give delta or partials, not both");
+  LLMK_REQUIRE(out == nullptr || pre != nullptr, "add_layernorm: an output needs its weight");
+  const size_t smem = (size_t)hidden * sizeof(float);
+  LLMK_REQUIRE(smem <= 200 * 1024, "add_layernorm: rows of %d elements exceed the shared memory", hidden);
+  return dispatch_dtype(dtype, [&](auto* tag) {
+    using T = LLMK_ELEM(tag);
+    MaybePartial<T> d{(const T*)delta, partials, splits, split_stride};
+    const bool vec = hidden % 8 == 0 && hidden <= 8192 && d.vector_ok() && (uintptr_t)resid % 16 == 0 && (uintptr_t)post % 16 == 0 &&
+                     (uintptr_t)pre % 16 == 0 && (uintptr_t)out % 16 == 0;
+    if (vec && hidden <= 2048)
+      launch_kernel(add_layernorm_vec_kernel<T, 1>, dim3(rows), dim3(256), 0, stream, resid, d, post, mult, pre, (T*)out, hidden, eps);
+    else if (vec && hidden <= 4096)
+      launch_kernel(add_layernorm_vec_kernel<T, 2>, dim3(rows), dim3(256), 0, stream, resid, d, post, mult, pre, (T*)out, hidden, eps);
+    else if (vec)
+      launch_kernel(add_layernorm_vec_kernel<T, 4>, dim3(rows), dim3(256), 0, stream, resid, d, post, mult, pre, (T*)out, hidden, eps);
+    else {
+      if (smem > 48 * 1024)
+        cudaFuncSetAttribute(add_layernorm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      launch_kernel(add_layernorm_kernel<T>, dim3(rows), dim3(256), smem, stream, resid, d, post, mult, pre, (T*)out, hidden, eps);
+    }
+    LLMK_LAUNCH_CHECK("add_layernorm");
+  });
 }
 
 // ---- soft cap ---------------------------------------------------------------------
@@ -934,10 +907,11 @@ head_rmsnorm_sigmoid_kernel(T* __restrict__ out, const float* __restrict__ x, co
   if (VEC) {
     for (int c = 4 * lane; c < n; c += 128) {
       const float4 v = *reinterpret_cast<const float4*>(row + c), w4 = *reinterpret_cast<const float4*>(wh + c);
-      const float y[4] = {v.x * w4.x, v.y * w4.y, v.z * w4.z, v.w * w4.w};
+      float g[4], y[4] = {v.x * w4.x, v.y * w4.y, v.z * w4.z, v.w * w4.w};
+      gate.at4(g0 + c, g);
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
-        out[(size_t)item * n + c + i] = from_f32<T>(y[i] * r / (1.f + expf(-gate.at(g0 + c + i))));
+      for (int i = 0; i < 4; ++i) y[i] *= r / (1.f + expf(-g[i]));
+      Vec4<T>::store(out + (size_t)item * n + c, y);
     }
   } else {
     for (int c = lane; c < n; c += 32)
@@ -953,7 +927,8 @@ LLMK_API int llmk_head_rmsnorm_sigmoid(void* out, const float* x, const float* w
   if (items == 0) return 0;
   LLMK_REQUIRE((gate != nullptr) != (partials != nullptr), "head_rmsnorm_sigmoid: give gate or partials");
   LLMK_REQUIRE(gate_dtype == dtype || gate_dtype == LLMK_F32, "head_rmsnorm_sigmoid: the gate is float32 or of the output's kind");
-  const bool vec = n % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0;
+  const bool vec = n % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)gate % 16 == 0 &&
+                   (uintptr_t)partials % 16 == 0 && split_stride % 4 == 0 && gate_stride % 4 == 0 && gate_col % 4 == 0;
   const dim3 grid((unsigned)((items + 3) / 4));
   return dispatch_dtype(dtype, [&](auto* tag) {
     using T = LLMK_ELEM(tag);

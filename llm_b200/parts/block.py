@@ -82,15 +82,16 @@ class SandwichBlock:
             if self.parts[r] is not None and not hasattr(self.parts[r], "attach"):
                 raise ValueError(f"sandwich block: the norm '{part_specs[r].kind}' cannot stand behind a sublayer (no attach)")
         self.mixer, self.ffn = self.parts["mixer"], self.parts["ffn"]
-        # a feed-forward whose last bias the norm behind it can add leaves it to that norm
-        self.biased = ({"allow_biased": True} if getattr(self.ffn, "leaves_bias", False)
-                       and getattr(self.parts["post2"], "takes_bias", False) else {})
+        # a sublayer that can leave its last sums to the norm behind it does so
+        unsummed = lambda part, post: ({"allow_unsummed": True} if getattr(part, "leaves_unsummed", False)
+                                       and getattr(self.parts[post], "takes_unsummed", False) else {})
+        self.mixer_options, self.ffn_options = unsummed(self.mixer, "post1"), unsummed(self.ffn, "post2")
 
     def forward(self, stream: ResidualStream, ctx, view) -> None:
         p = self.parts
-        p["post1"].attach(stream, self.mixer.forward(p["norm1"].forward(stream, ctx), ctx, view), self.mult)
+        p["post1"].attach(stream, self.mixer.forward(p["norm1"].forward(stream, ctx), ctx, view, **self.mixer_options), self.mult)
         if self.ffn is not None:
-            p["post2"].attach(stream, self.ffn.forward(p["norm2"].forward(stream, ctx), ctx, **self.biased), self.mult)
+            p["post2"].attach(stream, self.ffn.forward(p["norm2"].forward(stream, ctx), ctx, **self.ffn_options), self.mult)
 
 
 register_part("block", "sandwich", SandwichBlock)
@@ -119,7 +120,7 @@ class PostNormBlock:
         if self.ffn is not None and hasattr(self.ffn, "state_need"):
             raise ValueError("postnorm block: the feed-forward keeps no state of its own")
         # a feed-forward that can leave its last weighted sum to the norm does so
-        self.unsummed = {"allow_unsummed": True} if getattr(self.ffn, "leaves_unsummed", False) else {}
+        self.unsummed = {"allow_unsummed": True} if getattr(self.ffn, "leaves_weighted_rows", False) else {}
 
     def forward(self, stream: ResidualStream, ctx, view) -> None:
         p = self.parts

@@ -76,8 +76,8 @@ register_part("ffn", "swiglu", SwiGLU)
 class ActMLP(Part):
     """down(act(up(x))): a feed-forward with one up-projection and an element-wise activation
     ("relu2": the square of relu, "gelu": erf, "gelu_tanh", "silu").  Tensors `<prefix>.up` and
-    `<prefix>.down` unless other names are given; with bias also `<up>.b` and `<down>.b`, of which the first is added in the
-    activation's kernel and the second, where the caller allows it, by the kernel that reads the result (ops.BiasedRows)."""
+    `<prefix>.down` unless other names are given; with bias also `<up>.b` and `<down>.b`, of which the first is added where the
+    activation is taken and the second, where the caller allows it, by the kernel that reads the result (ops.BiasedRows)."""
 
     role = "ffn"
 
@@ -91,7 +91,7 @@ class ActMLP(Part):
         self.w_up = self.w_down = self.b_up = self.b_down = None
 
     @property
-    def leaves_bias(self) -> bool:
+    def leaves_unsummed(self) -> bool:
         return self.bias
 
     def parameters(self):
@@ -109,14 +109,15 @@ class ActMLP(Part):
             self.b_up = tensors[self.name(self.up_name + ".b")].contiguous()
             self.b_down = tensors[self.name(self.down_name + ".b")].contiguous()
 
-    def forward(self, x: torch.Tensor, ctx, tag: str = "ffn", allow_biased: bool = False):
+    def forward(self, x: torch.Tensor, ctx, tag: str = "ffn", allow_unsummed: bool = False):
         T, ws = ctx.n_tokens, ctx.workspace
         act = ws.get(tag + "_act", T, self.intermediate_size, self.dtype)
         if self.bias:
-            up = linear(x, self.w_up, ws.get(tag + "_up", T, self.intermediate_size, self.dtype), T, allow_partial=FUSE_PARTIALS)
-            ops.bias_act_rows(act, up, self.b_up, T, self.activation)
+            if not linear_act(x, self.w_up, act, T, self.activation, bias=self.b_up):
+                up = linear(x, self.w_up, ws.get(tag + "_up", T, self.intermediate_size, self.dtype), T, allow_partial=FUSE_PARTIALS)
+                ops.bias_act_rows(act, up, self.b_up, T, self.activation)
             out = ws.get(tag + "_out", T, self.hidden_size, self.dtype)
-            if allow_biased:
+            if allow_unsummed:
                 return ops.BiasedRows(linear(act, self.w_down, out, T, allow_partial=FUSE_PARTIALS), self.b_down)
             return linear(act, self.w_down, out, T, bias=self.b_down)
         if not linear_act(x, self.w_up, act, T, self.activation):      # many rows: the activation in the product's epilogue

@@ -52,8 +52,11 @@ class MatrixLSTM(Part):
 
     def bind(self, tensors):
         n = lambda k: tensors[self.name(self.names[k])]
-        self.w_in = torch.cat([n("q"), n("k"), n("v"), n("gate"), n("i"), n("f")], dim=0).contiguous()
-        self.w_qkvg, self.w_if = self.w_in[:self.gate_col], self.w_in[self.gate_col:]
+        rows = [n("q"), n("k"), n("v"), n("gate"), n("i"), n("f")]
+        used = self.gate_col + 2 * self.num_heads
+        rows.append(rows[0].new_zeros(-used % 4, self.hidden_size))      # rows of the product on the 16-byte grid
+        self.w_in = torch.cat(rows, dim=0).contiguous()
+        self.w_qkvg, self.w_if = self.w_in[:self.gate_col], self.w_in[self.gate_col:used]
         self.b_i, self.b_f, self.gain, self.w_o = n("i_bias").contiguous(), n("f_bias").contiguous(), n("norm").contiguous(), n("out").contiguous()
 
     def cache_need(self):

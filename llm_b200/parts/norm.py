@@ -58,7 +58,7 @@ class RMSNorm(Part):
         stream.pending = None
         return out
 
-    takes_bias = True      # attach() takes ops.BiasedRows
+    takes_unsummed = True      # attach() takes a sublayer's result before its last sums (what ops.add_rmsnorms takes)
 
     def attach(self, stream: ResidualStream, y, mult: float = 1.0) -> None:
         """A sublayer's output left pending, to be normed by this part and scaled by `mult` before it joins the residual: x +=
@@ -69,10 +69,7 @@ class RMSNorm(Part):
         part, mult = stream.pending_post
         if not isinstance(part, RMSNorm) or part.eps != self.eps:
             raise ValueError("a pending term that another kind of norm is to treat cannot be folded by this one")
-        y, bias = stream.pending, None
-        if isinstance(y, ops.BiasedRows):
-            y, bias = y.rows, y.bias
-        ops.add_rmsnorms(stream.resid, y, part.gain, mult, pre, out, stream.rows, self.eps, delta_bias=bias)
+        ops.add_rmsnorms(stream.resid, stream.pending, part.gain, mult, pre, out, stream.rows, self.eps, self.dtype)
         stream.pending = stream.pending_post = None
 
     def fold(self, stream: ResidualStream, ctx) -> None:

@@ -508,7 +508,12 @@ class ParallelMixers(Part):
         n = self.left_cols + self.right_cols
         return StateNeed((n,), torch.float32) if n else None
 
-    def forward(self, x: torch.Tensor, ctx, view) -> torch.Tensor:
+    @property
+    def leaves_unsummed(self) -> bool:
+        """Whether the two sides may be left to be summed by the kernel that reads them (ops.ScaledPair)."""
+        return self.combine == "scaled_sum"
+
+    def forward(self, x: torch.Tensor, ctx, view, allow_unsummed: bool = False):
         T, ws = ctx.n_tokens, ctx.workspace
         ls = view.state[:, :self.left_cols] if self.left_cols else None
         rs = view.state[:, self.left_cols:] if self.right_cols else None
@@ -516,6 +521,8 @@ class ParallelMixers(Part):
         # unsummed partial results live until the next product: the left side's are summed before the right side runs
         a = ops.settle(a, ws.get("parallel_left", T, self.hidden_size, self.dtype), T)
         b = self.right.forward(x, ctx, _sub_view(view, rs))
+        if allow_unsummed and self.leaves_unsummed:
+            return ops.ScaledPair(a, b, self.left_scale, self.right_scale)
         out = ws.get("parallel_out", T, self.hidden_size, self.dtype)
         if self.combine == "scaled_sum":
             ops.scaled_sum(out, a, b, self.left_scale, self.right_scale, T)

@@ -130,13 +130,15 @@ class RoutedFFN(Part):
         else:
             ops.silu_mul(act, gate_up, rows)
 
+    leaves_unsummed = True      # the last sum (a token's experts, the shared one) can be left to the kernel that reads it
+
     @property
-    def leaves_unsummed(self) -> bool:
-        """Whether the weighted sum of a token's experts can be left to the kernel that reads it (no shared expert beside it)."""
+    def leaves_weighted_rows(self) -> bool:
+        """Whether that sum is one over the experts' rows alone."""
         return self.shared is None and not self.identity
 
     def forward(self, x: torch.Tensor, ctx, allow_unsummed: bool = False):
-        """With allow_unsummed (and no shared expert) the result is an ops.WeightedRows, else a tensor."""
+        """With allow_unsummed the result is an ops.WeightedRows, else a tensor."""
         T, ws, top, E = ctx.n_tokens, ctx.workspace, self.top, self.experts
         # bfloat16 runs the experts on the tensor cores (tiles of 128 slots, or of 16 or 32 where an expert gets few rows; rows
         # gathered into slot order first); float32, and shapes the tensor-core kernel refuses, on the CUDA cores (tiles of 64)
@@ -183,11 +185,11 @@ class RoutedFFN(Part):
             ops.moe_gemm_tc(act, tile_expert, meta, self.w_down, y, max_tiles, tile=tile)
         else:
             ops.moe_gemm(act, 0, slot_src, tile_expert, meta, self.w_down, y, max_tiles)
-        if allow_unsummed and self.leaves_unsummed:
-            return ops.WeightedRows(y, pair_slot, wts, top, T)
         shared = self.shared.forward(x, ctx, tag="ffn_shared") if self.shared is not None else None
-        out = ws.get("ffn_out", T, self.hidden_size, self.dtype)
         more = {"ids": ids, "first_identity": E, "x": x} if self.identity else {}
+        if allow_unsummed:
+            return ops.WeightedRows(y, pair_slot, wts, top, T, shared=shared, shared_gate=gate, **more)
+        out = ws.get("ffn_out", T, self.hidden_size, self.dtype)
         ops.moe_combine(out, y, pair_slot, wts, shared, T, top, shared_gate=gate, **more)
         return out
 

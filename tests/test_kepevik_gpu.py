@@ -58,18 +58,62 @@ def test_rms_norms_on_both_sides_of_the_residual_sum(dtype, hidden, rows):
     x, y, bias = torch.randn(rows, hidden, generator=g), bf(torch.randn(rows, hidden, generator=g)), torch.randn(hidden, generator=g)
     post, pre, eps, mult = torch.randn(hidden, generator=g), torch.randn(hidden, generator=g), 1e-3, 0.8
     d = lambda t: t.double()
+    with_bias = lambda b: dev(y, dtype) if b is None else ops.BiasedRows(dev(y, dtype), dev(b))
     for b in (None, bias):
         want = d(x) + mult * P.rms_unit(d(y) + (0 if b is None else d(b)), eps) * d(post)
         resid, out = dev(x), torch.empty(rows, hidden, device="cuda", dtype=DT[dtype])
-        ops.add_rmsnorms(resid, dev(y, dtype), dev(post), mult, dev(pre), out, rows, eps, delta_bias=None if b is None else dev(b))
+        ops.add_rmsnorms(resid, with_bias(b), dev(post), mult, dev(pre), out, rows, eps)
         assert max_err(resid, want) < 1e-6 and max_err(out, P.rms_unit(want, eps) * d(pre)) < KTOL[dtype]
         resid = dev(x)
-        ops.add_rmsnorms(resid, dev(y, dtype), dev(post), mult, None, None, rows, eps, delta_bias=None if b is None else dev(b))
+        ops.add_rmsnorms(resid, with_bias(b), dev(post), mult, None, None, rows, eps)
         assert max_err(resid, want) < 1e-6
     parts = torch.randn(3, rows, hidden, generator=g)
     resid = dev(x)
     ops.add_rmsnorms(resid, ops.PartialSum(dev(parts), 3, rows, hidden, DT[dtype]), dev(post), mult, dev(pre), out, rows, eps)
     assert max_err(resid, d(x) + mult * P.rms_unit(d(parts).sum(0), eps) * d(post)) < 1e-6
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("hidden,rows", [(8, 3), (100, 5), (2048, 4), (4096, 2), (8200, 2)])
+def test_norms_take_a_sublayers_last_sums(dtype, hidden, rows):
+    """Two mixers' rows with their scales; a routed feed-forward's rows with identity experts and a gated shared expert, the norm's
+    output written over the input those experts pass."""
+    from llm_b200.csrc import ops
+    g = torch.Generator().manual_seed(hidden + 1)
+    x, a, b = torch.randn(rows, hidden, generator=g), bf(torch.randn(rows, hidden, generator=g)), torch.randn(2, rows, hidden, generator=g)
+    post, pre, eps = torch.randn(hidden, generator=g), torch.randn(hidden, generator=g), 1e-4
+    part = ops.PartialSum(dev(b), 2, rows, hidden, DT[dtype])
+    pair = 0.7 * a.double() - 1.3 * b.double().sum(0)
+    want = x.double() + P.rms_unit(pair, eps) * post.double()
+    resid, out = dev(x), torch.empty(rows, hidden, device="cuda", dtype=DT[dtype])
+    ops.add_rmsnorms(resid, ops.ScaledPair(dev(a, dtype), part, 0.7, -1.3), dev(post), 1.0, dev(pre), out, rows, eps)
+    assert max_err(resid, want) < 2e-6 and max_err(out, P.rms_unit(want, eps) * pre.double()) < KTOL[dtype]
+    top, E = 3, 4
+    y, w, h = torch.randn(6, hidden, generator=g), torch.rand(rows, top, generator=g), bf(torch.randn(rows, hidden, generator=g))
+    ids = torch.randint(0, E + 2, (rows, top), generator=g)
+    ids[0, 0], ids[-1, -1] = E, E + 1
+    slots = torch.where(ids < E, ids, torch.full_like(ids, -1))
+    gate = torch.rand(rows, generator=g)
+    terms = torch.where((ids < E).unsqueeze(-1), y.double()[slots.clamp(min=0)], h.double().unsqueeze(1))
+    routed = (w.double().unsqueeze(-1) * terms).sum(1)
+    for shared, scale in ((None, 0.0), (part, 1.0)):
+        want = x.double() + 0.5 * P.rms_unit(routed + scale * gate.double().unsqueeze(1) * b.double().sum(0), eps) * post.double()
+        resid, hd = dev(x), dev(h, dtype)
+        rows_of = ops.WeightedRows(dev(y), i32(slots.flatten().tolist()), dev(w), top, rows, shared=shared, shared_gate=dev(gate) if shared else None,
+                                   ids=i32(ids.flatten().tolist()), first_identity=E, x=hd)
+        ops.add_rmsnorms(resid, rows_of, dev(post), 0.5, dev(pre), hd, rows, eps)
+        assert max_err(resid, want) < 2e-6 and max_err(hd, P.rms_unit(want, eps) * pre.double()) < KTOL[dtype]
+
+
+@pytest.mark.parametrize("rows,ff,width", [(129, 72, 64), (300, 328, 128), (1000, 1000, 512)])
+def test_bias_and_activation_in_the_products_epilogue(rows, ff, width):
+    """Many rows in bfloat16: gelu(x W^T + b) is made in the epilogue of the product; widths off the tile's among them."""
+    from llm_b200.parts.linear import linear_act
+    g = torch.Generator().manual_seed(rows)
+    x, w, b = bf(torch.randn(rows, width, generator=g)), bf(torch.randn(ff, width, generator=g) / math.sqrt(width)), torch.randn(ff, generator=g)
+    out = torch.empty(rows, ff, device="cuda", dtype=torch.bfloat16)
+    assert linear_act(dev(x, "bfloat16"), dev(w, "bfloat16"), out, rows, "gelu", bias=dev(b))
+    assert max_err(out, P.gelu(x.double() @ w.double().T + b.double())) < KTOL["bfloat16"]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -168,6 +212,11 @@ def test_routed_feed_forward_alone(dtype, W, F, E, I, top, shared, T):
     assert I == 0 or bool((ids >= E).any()), "premise: some tokens choose an identity expert"
     ctx = SimpleNamespace(n_tokens=T, workspace=Workspace(max(T, 64), torch.device("cuda")), decode_only=False)
     out = part.forward(dev(x, dtype), ctx)
+    late = part.forward(dev(x, dtype), ctx, allow_unsummed=True)
+    resid = torch.zeros(T, W, device="cuda")
+    from llm_b200.csrc import ops
+    ops.add_rmsnorms(resid, late, None, 1.0, None, None, T, 1e-6)
+    assert max_err(resid, out) < (1e-6 if dtype == "float32" else 8e-3)
     clear = margin > (1e-5 if dtype == "float32" else 1e-2)
     assert int(clear.sum()) > T // 2 and max_err(out[clear.cuda()], ref[clear]) < (2e-6 if dtype == "float32" else 1.5e-2)
 
