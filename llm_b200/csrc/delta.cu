@@ -289,11 +289,13 @@ int launch_delta_of(const DeltaArgs& a, int n_entries, cudaStream_t stream) {
 // W, Y, B and the scaled q and k do not depend on the state: delta_prepare makes them for every chunk of the step side by
 // side (a CTA per chunk and head: unit norms, the two Gram matrices, forward substitution with a column per thread) and
 // leaves them chunk by chunk, padded with zeros to whole chunks, Y and the scaled q with the tokens innermost.
-// delta_chunk_walk then runs an entry's chunks one after another: per chunk three small matrix products on the CUDA cores
-// with the operands in shared memory (asynchronous copies, the next chunk's under this chunk's arithmetic) and register
-// tiles of 16 to 32 sums a thread, the state's tile in registers from chunk to chunk and mirrored in shared memory for the
-// products that read all of it.  What is left of the chain from token to token is one step per chunk.  All of it float32;
-// the sums of a token are grouped by where its chunk begins, which moves results by rounding only.
+// delta_chunk_walk then runs an entry's chunks one after another and does only what the chain needs: U = W - Y S_0 (left in
+// W's place) and the next S_0 (left for every chunk), two small matrix products on the CUDA cores with the operands in
+// shared memory (asynchronous copies, the next chunk's under this chunk's arithmetic), the first with its sum over the state's
+// rows split over the warps, the state's tile in registers from chunk to chunk and mirrored in shared memory.
+// delta_chunk_out makes the outputs of all chunks side by side again.  What is left of the chain from token to token is one
+// step per chunk.  All of it float32; the sums of a token are grouped by where its chunk begins, which moves results by
+// rounding only.
 //
 // With a decay per key channel (CH) L_t is a vector over the channels and the decays stand inside the Gram matrices,
 //     A_ts = beta_t sum_d exp(L_td - L_sd) k_td k_sd,    B_ts alike with q_t,
@@ -315,6 +317,7 @@ struct PrepArgs {
   // per chunk c and head h, at (c * heads + h) * size: YQ [dim][2 CC] (Y's tokens, then the scaled q's), K [CC][dim],
   // W [CC][vdim], B [CC][CC], G [1] (the chunk's whole decay; CH: [dim])
   float *YQ, *K, *W, *B, *G;
+  bool vec;                 // q, k and (CH) a and dt_bias may be read four channels at a time
 };
 
 // The chunk with the running number idx: its first token and its length, or false when the step has fewer chunks.
@@ -327,8 +330,20 @@ __device__ __forceinline__ bool chunk_of(const int* cu_tokens, int n_entries, in
   return false;
 }
 
+constexpr int PT = 256;                      // threads of a preparing CTA
+constexpr int FAR_S = CB * (CC / CB) * (CC / CB - 1) / 2;      // rows of keys scaled to the token before a later block, over all blocks
+constexpr float LOG2_E = 1.44269504088896340736f;
+
+// Floats of shared memory: unit k and q [CC][pitch], A with its rows innermost [CC][CC + 4], beta [CC], the decays' running sums
+// ([CC], CH: [CC][pitch]) and (CH) the scaled rows: k before each block [FAR_S][pitch], k and q of the blocks [2][CC - CB][pitch].
+__host__ __device__ inline int prepare_pitch(int dim) { return (dim + 3) / 4 * 4 + 4; }
+inline size_t prepare_floats(int dim, bool ch) {
+  const int p = prepare_pitch(dim);
+  return (size_t)2 * CC * p + CC * (CC + 4) + CC + (ch ? (size_t)(CC + FAR_S + 2 * (CC - CB)) * p : (size_t)CC);
+}
+
 template <typename T, bool CH>
-__global__ void __launch_bounds__(256, CH ? 2 : 1)
+__global__ void __launch_bounds__(PT, 2)
 delta_prepare_kernel(PrepArgs a) {
   extern __shared__ __align__(16) float smem[];
   pdl_launch_dependents();
@@ -336,150 +351,200 @@ delta_prepare_kernel(PrepArgs a) {
   int c0, n;
   if (!chunk_of(a.cu_tokens, a.n_entries, blockIdx.x, c0, n)) return;
   const int head = blockIdx.y, qk_head = head / (a.heads / a.qk_heads);
-  const int dim = a.dim, vdim = a.vdim, pitch = dim + 1;
+  const int dim = a.dim, vdim = a.vdim, pitch = prepare_pitch(dim), dim4 = pitch - 4;
   const size_t unit = (size_t)blockIdx.x * a.heads + head;
-  float* kn = smem;                        // [CC][dim + 1]
-  float* qn = kn + CC * pitch;             // [CC][dim + 1]
-  float* A_s = qn + CC * pitch;            // [CC][CC + 1]
-  float* beta_s = A_s + CC * (CC + 1);     // [CC]
-  float* L_s = beta_s + CC;                // [CC]: log g, then its running sum; CH: [CC][dim + 1]
-  float* kr_s = L_s + CC * pitch;          // CH: [CC - CB][dim + 1] keys scaled to the token before a block
-  float* xr_s = kr_s + (CC - CB) * pitch;  // CH: [2][CB][dim + 1] the block's k and q scaled from that token
+  constexpr int AP = CC + 4;
+  float* kn = smem;                        // [CC][pitch], zeros behind dim
+  float* qn = kn + CC * pitch;
+  float* At = qn + CC * pitch;             // [CC][AP]: At[s][t] = A_ts, zero unless s < t
+  float* beta_s = At + CC * AP;
+  float* L_s = beta_s + CC;                // the running sums of log2 g
+  float* kr_s = L_s + CC * pitch;          // CH
+  float* xr_s = kr_s + FAR_S * pitch;      // CH
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const T *q = (const T*)a.q, *k = (const T*)a.k, *v = (const T*)a.v, *pb = (const T*)a.b;
   using A = typename std::conditional<CH, float, T>::type;
   const A* pa = (const A*)a.a;
-  const float neg_a = -expf(a.a_log[head]), dt_b = CH ? 0.f : a.dt_bias[head];
-  // unit q and k, beta and log g: a warp per token
-  for (int t = warp; t < CC; t += 8) {
-    const size_t at = (size_t)(c0 + t) * a.qk_stride + (size_t)qk_head * dim;
-    float sq = 0.f, sk = 0.f;
-    if (t < n)
-      for (int d = lane; d < dim; d += 32) {
-        const float x = to_f32(q[at + d]), y = to_f32(k[at + d]);
-        sq = fmaf(x, x, sq); sk = fmaf(y, y, sk);
+  const float neg_a = -expf(a.a_log[head]) * LOG2_E, dt_b = CH ? 0.f : a.dt_bias[head];
+
+  // q, k and the logarithms of the decays as they come; beta.  Every loop over channels takes four of them a thread; loads go
+  // to clamped places, so that none waits for a test.
+  const int quads = dim4 / 4;
+  auto put4 = [](float* p, float x, float y, float z, float w) { *reinterpret_cast<float4*>(p) = make_float4(x, y, z, w); };
+  auto at4 = [](const float* p) { return *reinterpret_cast<const float4*>(p); };
+#pragma unroll 4
+  for (int i = tid; i < CC * quads; i += PT) {
+    const int t = i / quads, d = 4 * (i % quads);
+    const size_t row = (size_t)(c0 + min(t, n - 1));
+    const T *qp = q + row * a.qk_stride + (size_t)qk_head * dim, *kp = k + row * a.qk_stride + (size_t)qk_head * dim;
+    float qv[4], kv[4], zv[4] = {0.f, 0.f, 0.f, 0.f}, bv[4] = {0.f, 0.f, 0.f, 0.f};
+    if (a.vec) {
+      Vec4<T>::load(qp + d, qv); Vec4<T>::load(kp + d, kv);
+      if constexpr (CH) { Vec4<float>::load(pa + row * a.a_stride + (size_t)head * dim + d, zv); Vec4<float>::load(a.dt_bias + (size_t)head * dim + d, bv); }
+    } else {
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int e = min(d + x, dim - 1);
+        qv[x] = to_f32(qp[e]); kv[x] = to_f32(kp[e]);
+        if (CH) { zv[x] = to_f32(pa[row * a.a_stride + (size_t)head * dim + e]); bv[x] = a.dt_bias[(size_t)head * dim + e]; }
       }
-    const float rq = a.q_scale / sqrtf(warp_sum(sq) + a.norm_eps), rk = 1.f / sqrtf(warp_sum(sk) + a.norm_eps);
-    for (int d = lane; d < dim; d += 32) {
-      qn[t * pitch + d] = t < n ? to_f32(q[at + d]) * rq : 0.f;
-      kn[t * pitch + d] = t < n ? to_f32(k[at + d]) * rk : 0.f;
-      if (CH)
-        L_s[t * pitch + d] = t < n ? neg_a * softplus_d(to_f32(pa[(size_t)(c0 + t) * a.a_stride + (size_t)head * dim + d]) +
-                                                        a.dt_bias[(size_t)head * dim + d]) : 0.f;
     }
-    if (lane == 0) {
-      beta_s[t] = t < n ? 1.f / (1.f + expf(-to_f32(pb[(size_t)(c0 + t) * a.b_stride + head]))) : 0.f;
-      if (!CH) L_s[t] = t < n ? neg_a * softplus_d(to_f32(pa[(size_t)(c0 + t) * a.a_stride + head]) + dt_b) : 0.f;      // log g: the decay without its exponential
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      const bool on = t < n && d + x < dim;
+      qv[x] = on ? qv[x] : 0.f; kv[x] = on ? kv[x] : 0.f;
+      if (CH) zv[x] = on ? neg_a * softplus_d(zv[x] + bv[x]) : 0.f;
     }
+    put4(qn + t * pitch + d, qv[0], qv[1], qv[2], qv[3]);
+    put4(kn + t * pitch + d, kv[0], kv[1], kv[2], kv[3]);
+    if (CH) put4(L_s + t * pitch + d, zv[0], zv[1], zv[2], zv[3]);
   }
+  if (tid < CC) {
+    const int t = tid;
+    beta_s[t] = t < n ? 1.f / (1.f + expf(-to_f32(pb[(size_t)(c0 + t) * a.b_stride + head]))) : 0.f;
+    if (!CH) L_s[t] = t < n ? neg_a * softplus_d(to_f32(pa[(size_t)(c0 + t) * a.a_stride + head]) + dt_b) : 0.f;
+  }
+  for (int i = tid; i < CC * AP; i += PT) At[i] = 0.f;
+  for (int i = tid; i < CC * CC; i += PT)
+    if (i % CC > i / CC) a.B[unit * CC * CC + i] = 0.f;
   __syncthreads();
+  // unit q and k: a warp per token; the running sums
+  for (int t = warp; t < CC; t += PT / 32) {
+    float sq = 0.f, sk = 0.f;
+    for (int d = lane; d < dim; d += 32) {
+      sq = fmaf(qn[t * pitch + d], qn[t * pitch + d], sq);
+      sk = fmaf(kn[t * pitch + d], kn[t * pitch + d], sk);
+    }
+    const float rq = a.q_scale / sqrtf(warp_sum(sq) + a.norm_eps), rk = 1.f / sqrtf(warp_sum(sk) + a.norm_eps);
+    for (int d = lane; d < dim; d += 32) { qn[t * pitch + d] *= rq; kn[t * pitch + d] *= rk; }
+  }
   if (CH) {
-    for (int d = tid; d < dim; d += 256) {
+    for (int d = tid; d < dim; d += PT) {
       float run = 0.f;
+#pragma unroll
       for (int t = 0; t < CC; ++t) { run += L_s[t * pitch + d]; L_s[t * pitch + d] = run; }
     }
   } else if (tid == 0) {
     float run = 0.f;
+#pragma unroll
     for (int t = 0; t < CC; ++t) { run += L_s[t]; L_s[t] = run; }
   }
   __syncthreads();
+  // the two Gram matrices with their decays
+  auto dot4 = [](const float4& x, const float4& y, float s) { return fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, s)))); };
   if (CH) {
-    for (int idx = tid; idx < CC * CC; idx += 256) {          // beyond the diagonal
-      const int t = idx / CC, s2 = idx % CC;
-      if (s2 > t) { A_s[t * (CC + 1) + s2] = 0.f; a.B[unit * CC * CC + idx] = 0.f; }
+    // rows scaled to and from the token before each block but the first
+    auto scaled = [&](const float4& x, const float4& hi, const float4& lo) {
+      return make_float4(x.x * exp2f(hi.x - lo.x), x.y * exp2f(hi.y - lo.y), x.z * exp2f(hi.z - lo.z), x.w * exp2f(hi.w - lo.w));
+    };
+#pragma unroll 2
+    for (int i = tid; i < FAR_S * quads; i += PT) {
+      int s2 = i / quads, blk = 1;
+      const int d = 4 * (i % quads), row = s2;
+      while (s2 >= blk * CB) { s2 -= blk * CB; ++blk; }
+      *reinterpret_cast<float4*>(kr_s + row * pitch + d) = scaled(at4(kn + s2 * pitch + d), at4(L_s + (blk * CB - 1) * pitch + d), at4(L_s + s2 * pitch + d));
+    }
+#pragma unroll 2
+    for (int i = tid; i < 2 * (CC - CB) * quads; i += PT) {
+      const int row = i / quads, d = 4 * (i % quads), t = row % (CC - CB) + CB;
+      *reinterpret_cast<float4*>(xr_s + row * pitch + d) =
+          scaled(at4((row < CC - CB ? kn : qn) + t * pitch + d), at4(L_s + t * pitch + d), at4(L_s + (t / CB * CB - 1) * pitch + d));
     }
     // pairs within a block: four threads a pair, an exponential for every channel
     constexpr int PAIRS = CB * (CB + 1) / 2;
-    for (int w = tid / 4; w < CC / CB * PAIRS; w += 64) {
+    static_assert(CC / CB * PAIRS % 8 == 0, "a warp's eight pairs are all there or none");
+    for (int w = tid / 4; w < CC / CB * PAIRS; w += PT / 4) {
       const int blk = w / PAIRS;
       int i = 0, left = w % PAIRS;
       while (left > i) { left -= i + 1; ++i; }                // the pair (i, left), left <= i, of the block's lower triangle
       const int t = blk * CB + i, s2 = blk * CB + left;
       float kk = 0.f, qk = 0.f;
-      for (int d = tid % 4; d < dim; d += 4) {
-        const float x = expf(L_s[t * pitch + d] - L_s[s2 * pitch + d]) * kn[s2 * pitch + d];
-        kk = fmaf(kn[t * pitch + d], x, kk);
-        qk = fmaf(qn[t * pitch + d], x, qk);
+      for (int d = 4 * (tid % 4); d < dim4; d += 16) {
+        const float4 lt = at4(L_s + t * pitch + d), ls = at4(L_s + s2 * pitch + d);
+        float4 x = at4(kn + s2 * pitch + d);
+        x.x *= exp2f(lt.x - ls.x); x.y *= exp2f(lt.y - ls.y); x.z *= exp2f(lt.z - ls.z); x.w *= exp2f(lt.w - ls.w);
+        kk = dot4(at4(kn + t * pitch + d), x, kk);
+        qk = dot4(at4(qn + t * pitch + d), x, qk);
       }
-      static_assert(CC / CB * PAIRS % 8 == 0, "a warp's eight pairs are all there or none");
       kk += __shfl_xor_sync(0xffffffffu, kk, 1); kk += __shfl_xor_sync(0xffffffffu, kk, 2);
       qk += __shfl_xor_sync(0xffffffffu, qk, 1); qk += __shfl_xor_sync(0xffffffffu, qk, 2);
       if (tid % 4 == 0) {
-        A_s[t * (CC + 1) + s2] = s2 < t ? kk * beta_s[t] : 0.f;
-        a.B[unit * CC * CC + t * CC + s2] = t < n ? qk : 0.f;
+        if (s2 < t) At[s2 * AP + t] = kk * beta_s[t];
+        a.B[unit * CC * CC + t * CC + s2] = qk;
       }
     }
-    // pairs of two blocks, one later block at a time
-    for (int t0 = CB; t0 < CC && t0 < n; t0 += CB) {
-      const float* ref = L_s + (t0 - 1) * pitch;
-      for (int idx = tid; idx < t0 * dim; idx += 256) {
-        const int s2 = idx / dim, d = idx % dim;
-        kr_s[s2 * pitch + d] = expf(ref[d] - L_s[s2 * pitch + d]) * kn[s2 * pitch + d];
+    __syncthreads();
+    // pairs of two blocks: a thread a token and two earlier ones
+    for (int w = tid; w < CB * FAR_S / 2; w += PT) {
+      const int i = w % CB;
+      int s2 = w / CB * 2, blk = 1;
+      const int far = s2;
+      while (s2 >= blk * CB) { s2 -= blk * CB; ++blk; }
+      const int t = blk * CB + i;
+      const float *xk = xr_s + (t - CB) * pitch, *xq = xk + (CC - CB) * pitch, *y0 = kr_s + far * pitch, *y1 = y0 + pitch;
+      float kk0 = 0.f, kk1 = 0.f, qk0 = 0.f, qk1 = 0.f;
+#pragma unroll 2
+      for (int d = 0; d < dim4; d += 4) {
+        const float4 k4 = at4(xk + d), q4 = at4(xq + d), u = at4(y0 + d), w4 = at4(y1 + d);
+        kk0 = dot4(k4, u, kk0); kk1 = dot4(k4, w4, kk1);
+        qk0 = dot4(q4, u, qk0); qk1 = dot4(q4, w4, qk1);
       }
-      for (int idx = tid; idx < CB * dim; idx += 256) {
-        const int i = idx / dim, d = idx % dim;
-        const float e = expf(L_s[(t0 + i) * pitch + d] - ref[d]);
-        xr_s[i * pitch + d] = e * kn[(t0 + i) * pitch + d];
-        xr_s[(CB + i) * pitch + d] = e * qn[(t0 + i) * pitch + d];
-      }
-      __syncthreads();
-      for (int idx = tid; idx < CB * t0; idx += 256) {
-        const int i = idx % CB, s2 = idx / CB, t = t0 + i;
-        float kk = 0.f, qk = 0.f;
-        for (int d = 0; d < dim; ++d) {
-          const float x = kr_s[s2 * pitch + d];
-          kk = fmaf(xr_s[i * pitch + d], x, kk);
-          qk = fmaf(xr_s[(CB + i) * pitch + d], x, qk);
-        }
-        A_s[t * (CC + 1) + s2] = kk * beta_s[t];
-        a.B[unit * CC * CC + t * CC + s2] = t < n ? qk : 0.f;
-      }
-      __syncthreads();
-    }
-    // blocks behind the chunk's last token
-    for (int idx = tid; idx < CC * CC; idx += 256) {
-      const int t = idx / CC, s2 = idx % CC;
-      if (t / CB * CB >= n && t >= CB && s2 < t / CB * CB) { A_s[t * (CC + 1) + s2] = 0.f; a.B[unit * CC * CC + idx] = 0.f; }
+      At[s2 * AP + t] = kk0 * beta_s[t]; At[(s2 + 1) * AP + t] = kk1 * beta_s[t];
+      *reinterpret_cast<float2*>(a.B + unit * CC * CC + t * CC + s2) = make_float2(qk0, qk1);
     }
   } else {
-    // the two Gram matrices with their decays
-    for (int idx = tid; idx < CC * CC; idx += 256) {
-      const int t = idx / CC, s2 = idx % CC;
-      float kk = 0.f, qk = 0.f;
-      if (s2 <= t && t < n) {
-        for (int d = 0; d < dim; ++d) {
-          const float ks = kn[s2 * pitch + d];
-          kk = fmaf(kn[t * pitch + d], ks, kk);
-          qk = fmaf(qn[t * pitch + d], ks, qk);
+    // a thread two tokens and two others
+    static_assert(CC / 2 * (CC / 2) == PT, "a tile of 2 x 2 pairs a thread");
+    const int t = 2 * (tid / (CC / 2)), s2 = 2 * (tid % (CC / 2));
+    if (s2 <= t) {
+      float kk[2][2] = {{0.f, 0.f}, {0.f, 0.f}}, qk[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
+#pragma unroll 2
+      for (int d = 0; d < dim4; d += 4) {
+        const float4 x[2] = {at4(kn + s2 * pitch + d), at4(kn + (s2 + 1) * pitch + d)};
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const float4 k4 = at4(kn + (t + i) * pitch + d), q4 = at4(qn + (t + i) * pitch + d);
+#pragma unroll
+          for (int j = 0; j < 2; ++j) { kk[i][j] = dot4(k4, x[j], kk[i][j]); qk[i][j] = dot4(q4, x[j], qk[i][j]); }
         }
-        const float e = expf(L_s[t] - L_s[s2]);
-        kk *= e * beta_s[t];
-        qk *= e;
       }
-      A_s[t * (CC + 1) + s2] = s2 < t ? kk : 0.f;
-      a.B[unit * CC * CC + idx] = (s2 <= t && t < n) ? qk : 0.f;
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const float e = exp2f(L_s[t + i] - L_s[s2 + j]);
+          if (s2 + j < t + i) At[(s2 + j) * AP + t + i] = kk[i][j] * e * beta_s[t + i];
+          if (s2 + j <= t + i) a.B[unit * CC * CC + (t + i) * CC + s2 + j] = qk[i][j] * e;
+        }
     }
   }
   __syncthreads();
-  // forward substitution: a thread per column of [beta V | beta exp(L) K], the column in registers
-  for (int col = tid; col < vdim + dim; col += 256) {
+  // forward substitution: a thread per column of [beta V | beta exp(L) K], the column in registers, earlier tokens taken off later
+  // ones token by token
+  for (int col = tid; col < vdim + dim; col += PT) {
     float x[CC];
     const bool is_v = col < vdim;
     const int d = col - vdim;
+    if (is_v) {
+      const T* vp = v + (size_t)c0 * a.v_stride + (size_t)head * vdim + col;
 #pragma unroll
-    for (int t = 0; t < CC; ++t) {
-      float r = 0.f;
-      if (t < n)
-        r = is_v ? beta_s[t] * to_f32(v[(size_t)(c0 + t) * a.v_stride + (size_t)head * vdim + col])
-                 : beta_s[t] * expf(CH ? L_s[t * pitch + d] : L_s[t]) * kn[t * pitch + d];
-      x[t] = r;
+      for (int t = 0; t < CC; ++t) x[t] = to_f32(vp[(size_t)min(t, n - 1) * a.v_stride]);
+#pragma unroll
+      for (int t = 0; t < CC; ++t) x[t] *= beta_s[t];        // beta is zero behind the chunk's last token
+    } else {
+#pragma unroll
+      for (int t = 0; t < CC; ++t) x[t] = beta_s[t] * exp2f(CH ? L_s[t * pitch + d] : L_s[t]) * kn[t * pitch + d];
     }
 #pragma unroll
-    for (int t = 1; t < CC; ++t) {
-      float r = x[t];
+    for (int s2 = 0; s2 < CC - 1; ++s2) {
 #pragma unroll
-      for (int s2 = 0; s2 < t; ++s2) r = fmaf(-A_s[t * (CC + 1) + s2], x[s2], r);
-      x[t] = r;
+      for (int t = (s2 + 1) / 4 * 4; t < CC; t += 4) {
+        const float4 f = at4(At + s2 * AP + t);               // zero up to token s2
+        if (t > s2) x[t] = fmaf(-f.x, x[s2], x[t]);
+        if (t + 1 > s2) x[t + 1] = fmaf(-f.y, x[s2], x[t + 1]);
+        if (t + 2 > s2) x[t + 2] = fmaf(-f.z, x[s2], x[t + 2]);
+        if (t + 3 > s2) x[t + 3] = fmaf(-f.w, x[s2], x[t + 3]);
+      }
     }
     if (is_v) {
 #pragma unroll
@@ -490,25 +555,37 @@ delta_prepare_kernel(PrepArgs a) {
       for (int t = 0; t < CC; t += 4) *reinterpret_cast<float4*>(dst + t) = make_float4(x[t], x[t + 1], x[t + 2], x[t + 3]);
     }
   }
-  // q and k with the decays that the walk needs: to the token from the chunk's start, from the token to the chunk's end
-  for (int idx = tid; idx < CC * dim; idx += 256) {
-    const int t = idx % CC, d = idx / CC;
-    a.YQ[(unit * dim + d) * (2 * CC) + CC + t] = t < n ? expf(CH ? L_s[t * pitch + d] : L_s[t]) * qn[t * pitch + d] : 0.f;
+  // q and k with the decays that follow need: to the token from the chunk's start, from the token to the chunk's end
+  for (int i = tid; i < dim * (CC / 4); i += PT) {
+    const int d = i % dim, t = i / dim * 4;
+    float y[4];
+#pragma unroll
+    for (int x = 0; x < 4; ++x) y[x] = exp2f(CH ? L_s[(t + x) * pitch + d] : L_s[t + x]) * qn[(t + x) * pitch + d];
+    *reinterpret_cast<float4*>(a.YQ + (unit * dim + d) * (2 * CC) + CC + t) = make_float4(y[0], y[1], y[2], y[3]);
   }
-  for (int idx = tid; idx < CC * dim; idx += 256) {
-    const int t = idx / dim, d = idx % dim;
-    const float rest = CH ? L_s[(n - 1) * pitch + d] - L_s[t * pitch + d] : L_s[n - 1] - L_s[t];
-    a.K[(unit * CC + t) * dim + d] = t < n ? expf(rest) * kn[t * pitch + d] : 0.f;
+#pragma unroll 2
+  for (int i = tid; i < CC * quads; i += PT) {
+    const int t = i / quads, d = 4 * (i % quads);
+    const float4 k4 = at4(kn + t * pitch + d);                // zero behind the last token
+    float y[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+    for (int x = 0; x < 4; ++x) y[x] *= exp2f(CH ? L_s[(n - 1) * pitch + d + x] - L_s[t * pitch + d + x] : L_s[n - 1] - L_s[t]);
+    float* dst = a.K + (unit * CC + t) * dim + d;
+    if (dim % 4 == 0) put4(dst, y[0], y[1], y[2], y[3]);
+    else
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+        if (d + x < dim) dst[x] = y[x];
   }
   if (CH)
-    for (int d = tid; d < dim; d += 256) a.G[unit * dim + d] = expf(L_s[(n - 1) * pitch + d]);
+    for (int d = tid; d < dim; d += PT) a.G[unit * dim + d] = exp2f(L_s[(n - 1) * pitch + d]);
   else if (tid == 0)
-    a.G[unit] = expf(L_s[n - 1]);
+    a.G[unit] = exp2f(L_s[n - 1]);
 }
 
 struct WalkArgs {
-  float* out; long long out_stride;
-  const float *YQ, *K, *W, *B, *G;
+  const float *YQ, *K, *G;
+  float *W, *S;             // W [CC][vdim] becomes U; S [dim][vdim]: the state that enters the chunk
   float* state; long long slot_stride;
   const int *state_slots, *cu_tokens;
   int heads, dim, vdim;
@@ -521,255 +598,282 @@ __device__ __forceinline__ void cp_async16(void* smem_dst, const void* src) {
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-constexpr int WT = 128, WV = 16;             // threads of a walking CTA, value columns it owns
-constexpr int TXN = WV / 4, TYN = WT / TXN;  // the threads as TYN x TXN: a thread's 4 columns start at 4 tx
-static_assert(2 * CC % TYN == 0 && CC % TYN == 0, "rows of the products divide among the threads");
+// DPAD: a head's rows rounded up to 32, 64, 128 or 256; WV: value columns a CTA owns (16, or 8 where there would be few CTAs).
+constexpr int WT = 256;                      // threads of a walking CTA
 
-// RT: rows of the state a thread keeps (a head's rows / 32, rounded up to 1, 2, 4 or 8).  STAGES chunks of operands lie in
-// shared memory (2: the next chunk's copies run under this chunk's arithmetic; 1 where two do not fit).
-template <int RT, int STAGES, bool CH>
+template <int DPAD, int WV>
+struct WalkShape {
+  static constexpr int C = 2;                                         // columns of a thread in both products
+  static constexpr int R1 = 4, SLICE = CC / R1 * (WV / C);            // Y S_0: rows of a thread, threads of a slice of the sum
+  static constexpr int KS = WT / SLICE, DEPTH = DPAD / KS;            // slices, and the state's rows in each
+  static constexpr int TX = WV / C, TY = WT / TX, R2 = DPAD / TY;     // K^T U: the threads as TY x TX, rows of a thread
+  static constexpr int STAGE = DPAD * CC + CC * DPAD + CC * WV;       // floats of one stage: Y, K, W
+  static constexpr size_t SMEM = (size_t)(2 * STAGE + DPAD * WV + KS * CC * WV + CC * WV) * sizeof(float);
+  static_assert(R2 >= 1 && DEPTH >= 1 && KS * DEPTH == DPAD && R2 * TY == DPAD, "the products divide among the threads");
+};
+
+template <int DPAD, int WV, bool CH>
 __global__ void __launch_bounds__(WT)
 delta_chunk_walk_kernel(WalkArgs a) {
+  using Sh = WalkShape<DPAD, WV>;
+  constexpr int R1 = Sh::R1, R2 = Sh::R2;
   extern __shared__ __align__(16) float smem[];
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int DPAD = TYN * RT, BP = CC + 4, RA = 2 * CC / TYN, RB = CC / TYN;      // rows a thread takes of the two products
-  constexpr int STAGE = DPAD * 2 * CC + CC * DPAD + CC * WV + CC * BP;      // floats of one stage: YQ, K, W, B
-  float* S_s = smem + STAGES * STAGE;      // [DPAD][WV]: the state as the products read it
-  float* u_s = S_s + DPAD * WV;            // [CC][WV]
-  float* o_s = u_s + CC * WV;              // [CC][WV]
-  const int tid = threadIdx.x, ty = tid / TXN, tx = tid % TXN;
+  float* S_s = smem + 2 * Sh::STAGE;        // [DPAD][WV]: the state as the first product reads it
+  float* part_s = S_s + DPAD * WV;          // [KS][CC][WV]
+  float* u_s = part_s + Sh::KS * CC * WV;   // [CC][WV]
+  const int tid = threadIdx.x, ty = tid / Sh::TX, tx = tid % Sh::TX;
+  const int ks = tid / Sh::SLICE, ry = (tid % Sh::SLICE) / (WV / 2), cx = tid % (WV / 2);
   const int entry = blockIdx.z, head = blockIdx.y;
-  const int dim = a.dim, vdim = a.vdim, colb = blockIdx.x * WV;
+  const int dim = a.dim, vdim = a.vdim, colb = blockIdx.x * WV, col = colb + 2 * tx;
   const int t0 = a.cu_tokens[entry], t1 = a.cu_tokens[entry + 1];
   if (t0 >= t1) return;
   int chunk = 0;                            // the running number of the entry's first chunk
   for (int e = 0; e < entry; ++e) chunk += (a.cu_tokens[e + 1] - a.cu_tokens[e] + CC - 1) / CC;
-  const bool vec = dim % 4 == 0 && vdim % 4 == 0;
+  const bool vec = dim % 4 == 0 && vdim % 4 == 0, even = vdim % 2 == 0;
   float* S_g = a.state + (size_t)a.state_slots[entry] * a.slot_stride + ((size_t)head * dim) * vdim;
-  float S[RT][4];                           // rows RT ty .., columns 4 tx ..
+  float S[R2][2];                           // rows R2 ty .., columns 2 tx ..
+  auto put = [&](float* dst) {              // the thread's tile of the state, to a [dim][vdim] array
+    const bool pairs = even && (uintptr_t)dst % 8 == 0;
 #pragma unroll
-  for (int i = 0; i < RT; ++i) {
-    const int d = ty * RT + i;
+    for (int i = 0; i < R2; ++i) {
+      const int d = ty * R2 + i;
+      if (d >= dim) continue;
+      float* at = dst + (size_t)d * vdim + col;
+      if (pairs && col < vdim) *reinterpret_cast<float2*>(at) = make_float2(S[i][0], S[i][1]);
+      else
 #pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      const int col = colb + 4 * tx + c;
-      S[i][c] = (d < dim && col < vdim) ? S_g[(size_t)d * vdim + col] : 0.f;
+        for (int c = 0; c < 2; ++c)
+          if (col + c < vdim) at[c] = S[i][c];
     }
-    *reinterpret_cast<float4*>(S_s + d * WV + 4 * tx) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+  };
+#pragma unroll
+  for (int i = 0; i < R2; ++i) {
+    const int d = ty * R2 + i;
+#pragma unroll
+    for (int c = 0; c < 2; ++c) S[i][c] = (d < dim && col + c < vdim) ? S_g[(size_t)d * vdim + col + c] : 0.f;
+    *reinterpret_cast<float2*>(S_s + d * WV + 2 * tx) = make_float2(S[i][0], S[i][1]);
   }
   // request the operands of chunk number c into a stage (they are padded with zeros to whole chunks where they were made)
   auto issue = [&](int c, float* st) {
     const size_t unit = (size_t)c * a.heads + head;
-    float *yq_s = st, *k_s = st + DPAD * 2 * CC, *w_s = k_s + CC * DPAD, *b_s = w_s + CC * WV;
+    float *y_s = st, *k_s = st + DPAD * CC, *w_s = k_s + CC * DPAD;
+    const float *y = a.YQ + unit * dim * 2 * CC, *k = a.K + unit * CC * dim, *w = a.W + unit * CC * vdim;
+    for (int i = tid; i < dim * CC / 4; i += WT) cp_async16(y_s + 4 * i, y + (size_t)(i / (CC / 4)) * 2 * CC + 4 * (i % (CC / 4)));
     if (vec) {
-      const float* src = a.YQ + unit * dim * 2 * CC;
-      for (int i = tid; i < dim * 2 * CC / 4; i += WT) cp_async16(yq_s + 4 * i, src + 4 * i);
-      src = a.K + unit * CC * dim;
-      for (int i = tid; i < CC * dim / 4; i += WT) { const int t = (4 * i) / dim, d = (4 * i) % dim; cp_async16(k_s + t * DPAD + d, src + 4 * i); }
-      src = a.W + unit * CC * vdim;
+      if (dim == DPAD)
+        for (int i = tid; i < CC * DPAD / 4; i += WT) cp_async16(k_s + 4 * i, k + 4 * i);
+      else
+        for (int i = tid; i < CC * dim / 4; i += WT) cp_async16(k_s + (4 * i) / dim * DPAD + (4 * i) % dim, k + 4 * i);
       for (int i = tid; i < CC * WV / 4; i += WT) {
-        const int t = (4 * i) / WV, c4 = (4 * i) % WV;
-        if (colb + c4 < vdim) cp_async16(w_s + 4 * i, src + (size_t)t * vdim + colb + c4);
+        const int c4 = (4 * i) % WV;
+        if (colb + c4 < vdim) cp_async16(w_s + 4 * i, w + (size_t)((4 * i) / WV) * vdim + colb + c4);
       }
     } else {
-      const float* src = a.YQ + unit * dim * 2 * CC;
-      for (int i = tid; i < dim * 2 * CC; i += WT) yq_s[i] = src[i];
-      src = a.K + unit * CC * dim;
-      for (int i = tid; i < CC * dim; i += WT) k_s[(i / dim) * DPAD + i % dim] = src[i];
-      src = a.W + unit * CC * vdim;
-      for (int i = tid; i < CC * WV; i += WT) if (colb + i % WV < vdim) w_s[i] = src[(size_t)(i / WV) * vdim + colb + i % WV];
+      for (int i = tid; i < CC * dim; i += WT) k_s[(i / dim) * DPAD + i % dim] = k[i];
+      for (int i = tid; i < CC * WV; i += WT)
+        if (colb + i % WV < vdim) w_s[i] = w[(size_t)(i / WV) * vdim + colb + i % WV];
     }
-    const float* src = a.B + unit * CC * CC;
-    for (int i = tid; i < CC * CC / 4; i += WT) cp_async16(b_s + ((4 * i) / CC) * BP + (4 * i) % CC, src + 4 * i);
     cp_async_commit();
   };
-  // rows of K beyond the head's and columns of W beyond the values' are never copied: they stay zero
-  for (int i = tid; i < STAGES * STAGE; i += WT) smem[i] = 0.f;
+  // rows of Y and K beyond the head's and columns of W beyond the values' are never copied: they stay zero
+  for (int i = tid; i < 2 * Sh::STAGE; i += WT) smem[i] = 0.f;
   __syncthreads();
   issue(chunk, smem);
   int at_stage = 0;
-  for (int c0 = t0; c0 < t1; c0 += CC, ++chunk) {
-    const int n = min(CC, t1 - c0);
-    float g_end[CH ? RT : 1];
+  for (int c0 = t0; c0 < t1; c0 += CC, ++chunk, at_stage ^= 1) {
+    const size_t unit = (size_t)chunk * a.heads + head;
+    const float *y_s = smem + at_stage * Sh::STAGE, *k_s = y_s + DPAD * CC, *w_s = k_s + CC * DPAD;
+    float g_end[CH ? R2 : 1];
     if (CH) {
 #pragma unroll
-      for (int i = 0; i < RT; ++i)
-        g_end[CH ? i : 0] = ty * RT + i < dim ? a.G[((size_t)chunk * a.heads + head) * dim + ty * RT + i] : 0.f;
+      for (int i = 0; i < R2; ++i) g_end[CH ? i : 0] = ty * R2 + i < dim ? a.G[unit * dim + ty * R2 + i] : 0.f;
     } else {
-      g_end[0] = a.G[(size_t)chunk * a.heads + head];
+      g_end[0] = a.G[unit];
     }
-    const float* st = smem + at_stage * STAGE;
-    const float *yq_s = st, *k_s = st + DPAD * 2 * CC, *w_s = k_s + CC * DPAD, *b_s = w_s + CC * WV;
-    const bool more = c0 + CC < t1;
-    if (STAGES == 2 && more) {
-      issue(chunk + 1, smem + (at_stage ^ 1) * STAGE);      // that stage's last readers passed the barrier below
+    put(a.S + unit * dim * vdim);            // under the waits below
+    if (c0 + CC < t1) {
+      issue(chunk + 1, smem + (at_stage ^ 1) * Sh::STAGE);      // that stage's last readers passed the barrier below
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
     }
     __syncthreads();                         // the stage has landed; S_s holds the state that enters the chunk
-    // [Y; exp(L) Q] S_0: 2 CC rows x WV columns, a thread RA rows (RA ty ..) x 4 columns
-    {
-      float acc[RA][4];
+    {                                        // this slice's share of Y S_0: rows R1 ry .., columns 2 cx ..
+      float acc[R1][2];
 #pragma unroll
-      for (int i = 0; i < RA; ++i)
+      for (int i = 0; i < R1; ++i) acc[i][0] = acc[i][1] = 0.f;
+#pragma unroll 8
+      for (int x = 0; x < Sh::DEPTH; ++x) {
+        const int d = ks * Sh::DEPTH + x;
+        const float4 y4 = *reinterpret_cast<const float4*>(y_s + d * CC + R1 * ry);
+        const float2 s2 = *reinterpret_cast<const float2*>(S_s + d * WV + 2 * cx);
+        const float yv[R1] = {y4.x, y4.y, y4.z, y4.w};
 #pragma unroll
-        for (int c = 0; c < 4; ++c) acc[i][c] = 0.f;
-      // four rows of the state and of the operands a step, the next step's loads issued before this step's multiply-adds
-      // (one warp per scheduler hides nothing by itself); rows beyond the head's are zero on both sides
-      float4 sa[4], sb[4];
-      float2 ra[4], rb[4];
-      auto load = [&](int d0, float4 (&sv)[4], float2 (&rv)[4]) {
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          sv[j] = *reinterpret_cast<const float4*>(S_s + (d0 + j) * WV + 4 * tx);
-          rv[j] = *reinterpret_cast<const float2*>(yq_s + (d0 + j) * 2 * CC + RA * ty);
-        }
-      };
-      auto mac = [&](const float4 (&sv)[4], const float2 (&rv)[4]) {
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const float s4[4] = {sv[j].x, sv[j].y, sv[j].z, sv[j].w};
-#pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            acc[0][c] = fmaf(rv[j].x, s4[c], acc[0][c]);
-            acc[1][c] = fmaf(rv[j].y, s4[c], acc[1][c]);
-          }
-        }
-      };
-      static_assert(RA == 2 && DPAD % 8 == 0, "a thread takes two rows of [Y; Q]");
-      load(0, sa, ra);
-#pragma unroll 1
-      for (int d0 = 0; d0 < DPAD; d0 += 8) {
-        load(d0 + 4, sb, rb);
-        mac(sa, ra);
-        if (d0 + 8 < DPAD) load(d0 + 8, sa, ra);
-        mac(sb, rb);
-      }
-#pragma unroll
-      for (int i = 0; i < RA; ++i) {
-        const int row = RA * ty + i;          // < CC: a row of Y (u = w - y S_0); else a row of the scaled q
-        if (row < CC) {
-          const float4 w4 = *reinterpret_cast<const float4*>(w_s + row * WV + 4 * tx);
-          *reinterpret_cast<float4*>(u_s + row * WV + 4 * tx) = make_float4(w4.x - acc[i][0], w4.y - acc[i][1], w4.z - acc[i][2], w4.w - acc[i][3]);
-        } else {
-          *reinterpret_cast<float4*>(o_s + (row - CC) * WV + 4 * tx) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+        for (int i = 0; i < R1; ++i) {
+          acc[i][0] = fmaf(yv[i], s2.x, acc[i][0]);
+          acc[i][1] = fmaf(yv[i], s2.y, acc[i][1]);
         }
       }
+#pragma unroll
+      for (int i = 0; i < R1; ++i)
+        *reinterpret_cast<float2*>(part_s + (ks * CC + R1 * ry + i) * WV + 2 * cx) = make_float2(acc[i][0], acc[i][1]);
     }
     __syncthreads();
-    // the outputs: o_t = (state's share) + sum_{s <= t} B_ts u_s; a thread RB tokens (RB ty ..) x 4 columns
-    {
-      float4 o[RB];
 #pragma unroll
-      for (int i = 0; i < RB; ++i) o[i] = *reinterpret_cast<const float4*>(o_s + (RB * ty + i) * WV + 4 * tx);
+    for (int i = tid; i < CC * WV; i += WT) {
+      float u = w_s[i];
+#pragma unroll
+      for (int k = 0; k < Sh::KS; ++k) u -= part_s[k * CC * WV + i];
+      u_s[i] = u;
+      if (colb + i % WV < vdim) a.W[(unit * CC + i / WV) * vdim + colb + i % WV] = u;
+    }
+    __syncthreads();
+    // the state at the chunk's end: decays times S_0, plus (scaled K)^T U
+#pragma unroll
+    for (int i = 0; i < R2; ++i) { S[i][0] *= g_end[CH ? i : 0]; S[i][1] *= g_end[CH ? i : 0]; }
 #pragma unroll 8
-      for (int s2 = 0; s2 < CC; ++s2) {      // B is zero beyond the diagonal
-        const float4 u4 = *reinterpret_cast<const float4*>(u_s + s2 * WV + 4 * tx);
+    for (int s2 = 0; s2 < CC; ++s2) {
+      const float2 u2 = *reinterpret_cast<const float2*>(u_s + s2 * WV + 2 * tx);
+      const float* kr = k_s + s2 * DPAD + ty * R2;
+      float kv[R2];
+      if constexpr (R2 % 4 == 0) {
 #pragma unroll
-        for (int i = 0; i < RB; ++i) {
-          const float bts = b_s[(RB * ty + i) * BP + s2];
-          o[i].x = fmaf(bts, u4.x, o[i].x); o[i].y = fmaf(bts, u4.y, o[i].y);
-          o[i].z = fmaf(bts, u4.z, o[i].z); o[i].w = fmaf(bts, u4.w, o[i].w);
+        for (int i = 0; i < R2; i += 4) {
+          const float4 k4 = *reinterpret_cast<const float4*>(kr + i);
+          kv[i] = k4.x; kv[i + 1] = k4.y; kv[i + 2] = k4.z; kv[i + 3] = k4.w;
         }
+      } else if constexpr (R2 == 2) {
+        const float2 k2 = *reinterpret_cast<const float2*>(kr);
+        kv[0] = k2.x; kv[1] = k2.y;
+      } else {
+        kv[0] = kr[0];
       }
 #pragma unroll
-      for (int i = 0; i < RB; ++i) {
-        const int t = RB * ty + i, col = colb + 4 * tx;
-        if (t >= n) continue;
-        float* dst = a.out + (size_t)(c0 + t) * a.out_stride + (size_t)head * vdim + col;
-        const float ov[4] = {o[i].x, o[i].y, o[i].z, o[i].w};
-#pragma unroll
-        for (int c = 0; c < 4; ++c)
-          if (col + c < vdim) dst[c] = ov[c];
-      }
-    }
-    // the state at the chunk's end: exp(L_C) S_0 + (scaled K)^T U; a thread RT rows x 4 columns, kept in registers
-#pragma unroll
-    for (int i = 0; i < RT; ++i)
-#pragma unroll
-      for (int c = 0; c < 4; ++c) S[i][c] *= g_end[CH ? i : 0];
-    {
-      float4 ua, ub;
-      float ka[RT], kb[RT];
-      auto load = [&](int s2, float4& u4, float (&kv)[RT]) {
-        u4 = *reinterpret_cast<const float4*>(u_s + s2 * WV + 4 * tx);
-        const float* kr = k_s + s2 * DPAD + ty * RT;
-        if (RT % 4 == 0) {
-#pragma unroll
-          for (int i = 0; i < RT; i += 4) {
-            const float4 k4 = *reinterpret_cast<const float4*>(kr + i);
-            kv[i] = k4.x; kv[(i + 1) % RT] = k4.y; kv[(i + 2) % RT] = k4.z; kv[(i + 3) % RT] = k4.w;      // (the wrap only quiets the bounds check where RT < 4)
-          }
-        } else {
-#pragma unroll
-          for (int i = 0; i < RT; ++i) kv[i] = kr[i];
-        }
-      };
-      auto mac = [&](const float4& u4, const float (&kv)[RT]) {
-        const float uv[4] = {u4.x, u4.y, u4.z, u4.w};
-#pragma unroll
-        for (int i = 0; i < RT; ++i)
-#pragma unroll
-          for (int c = 0; c < 4; ++c) S[i][c] = fmaf(kv[i], uv[c], S[i][c]);
-      };
-      load(0, ua, ka);
-#pragma unroll 2
-      for (int s2 = 0; s2 < CC; s2 += 2) {
-        load(s2 + 1, ub, kb);
-        mac(ua, ka);
-        if (s2 + 2 < CC) load(s2 + 2, ua, ka);
-        mac(ub, kb);
+      for (int i = 0; i < R2; ++i) {
+        S[i][0] = fmaf(kv[i], u2.x, S[i][0]);
+        S[i][1] = fmaf(kv[i], u2.y, S[i][1]);
       }
     }
-    __syncthreads();                         // every thread is done with this stage, u_s, o_s and the old S_s
+    // every reader of the old S_s passed the second barrier above
 #pragma unroll
-    for (int i = 0; i < RT; ++i)
-      *reinterpret_cast<float4*>(S_s + (ty * RT + i) * WV + 4 * tx) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
-    if (STAGES == 2) at_stage ^= 1;
-    else if (more) issue(chunk + 1, smem);
+    for (int i = 0; i < R2; ++i) *reinterpret_cast<float2*>(S_s + (ty * R2 + i) * WV + 2 * tx) = make_float2(S[i][0], S[i][1]);
+    __syncthreads();                         // this stage may be overwritten
   }
-#pragma unroll
-  for (int i = 0; i < RT; ++i) {
-    const int d = ty * RT + i;
-    if (d >= dim) continue;
-#pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      const int col = colb + 4 * tx + c;
-      if (col < vdim) S_g[(size_t)d * vdim + col] = S[i][c];
-    }
-  }
+  put(S_g);
 }
 
-template <int RT, bool CH>
+template <int DPAD, int WV, bool CH>
 int launch_walk(const WalkArgs& a, int n_entries, cudaStream_t stream) {
-  constexpr int STAGES = RT <= 4 ? 2 : 1;      // two stages of a head of 256 rows exceed an SM's shared memory
-  constexpr int DPAD = TYN * RT;
-  const size_t stage = (size_t)DPAD * 2 * CC + CC * DPAD + CC * WV + CC * (CC + 4);
-  const size_t smem = (STAGES * stage + DPAD * WV + 2 * CC * WV) * sizeof(float);
-  if (smem > 48 * 1024)
-    cudaFuncSetAttribute(delta_chunk_walk_kernel<RT, STAGES, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  launch_kernel(delta_chunk_walk_kernel<RT, STAGES, CH>, dim3((a.vdim + WV - 1) / WV, a.heads, n_entries), dim3(WT), smem, stream, a);
+  constexpr size_t smem = WalkShape<DPAD, WV>::SMEM;
+  if (smem > 48 * 1024) cudaFuncSetAttribute(delta_chunk_walk_kernel<DPAD, WV, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  launch_kernel(delta_chunk_walk_kernel<DPAD, WV, CH>, dim3((a.vdim + WV - 1) / WV, a.heads, n_entries), dim3(WT), smem, stream, a);
   LLMK_LAUNCH_CHECK("delta_chunk_walk");
 }
 
+template <int DPAD, bool CH>
+int launch_walk_of(const WalkArgs& a, int n_entries, cudaStream_t stream) {
+  if (DPAD >= 64 && (long long)(a.vdim + 15) / 16 * a.heads * n_entries < llmk_sm_count())
+    return launch_walk<DPAD, DPAD >= 64 ? 8 : 16, CH>(a, n_entries, stream);
+  return launch_walk<DPAD, 16, CH>(a, n_entries, stream);
+}
+
+// The outputs of a chunk: o_t = (scaled q_t)^T S_0 + sum_{s <= t} B_ts u_s; a CTA makes OV columns of one head's chunk, a thread 4
+// tokens x 4 columns.  Grid (chunks, heads, column tiles).
+constexpr int OV = 64, OT = CC / 4 * (OV / 4), BP = CC + 4;
+
+struct OutArgs {
+  float* out; long long out_stride;
+  const float *YQ, *B, *U, *S;
+  const int* cu_tokens; int n_entries;
+  int heads, dim, vdim;
+};
+
+__global__ void __launch_bounds__(OT)
+delta_chunk_out_kernel(OutArgs a) {
+  extern __shared__ __align__(16) float smem[];
+  pdl_launch_dependents();
+  pdl_wait();
+  int c0, n;
+  if (!chunk_of(a.cu_tokens, a.n_entries, blockIdx.x, c0, n)) return;
+  const int head = blockIdx.y, colb = blockIdx.z * OV, dim = a.dim, vdim = a.vdim, tid = threadIdx.x;
+  const size_t unit = (size_t)blockIdx.x * a.heads + head;
+  float* q_s = smem;                        // [dim][CC]
+  float* S_s = q_s + dim * CC;              // [dim][OV]
+  float* u_s = S_s + dim * OV;              // [CC][OV]
+  float* b_s = u_s + CC * OV;               // [CC][BP]: B with its rows (tokens) innermost
+  for (int i = tid; i < dim * CC / 4; i += OT)
+    cp_async16(q_s + 4 * i, a.YQ + (unit * dim + i / (CC / 4)) * 2 * CC + CC + 4 * (i % (CC / 4)));
+  auto bring = [&](float* dst, const float* src, int rows) {      // rows x OV columns from colb on, zeros beyond the values
+    for (int i = tid; i < rows * OV / 4; i += OT) {
+      const int r = i / (OV / 4), c = 4 * (i % (OV / 4));
+      const float* at = src + (size_t)r * vdim + colb + c;
+      if (vdim % 4 == 0 && colb + c < vdim) cp_async16(dst + 4 * i, at);
+      else
+        for (int k = 0; k < 4; ++k) dst[4 * i + k] = colb + c + k < vdim ? at[k] : 0.f;
+    }
+  };
+  bring(S_s, a.S + unit * dim * vdim, dim);
+  bring(u_s, a.U + unit * CC * vdim, CC);
+  for (int i = tid; i < CC * CC; i += OT) b_s[(i % CC) * BP + i / CC] = a.B[unit * CC * CC + i];
+  cp_async_commit();
+  cp_async_wait<0>();
+  __syncthreads();
+  const int ty = tid / (OV / 4), tx = tid % (OV / 4);
+  float o[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) o[i][c] = 0.f;
+  auto mac = [&](const float* rows, int pitch, const float* cols, int depth) {
+#pragma unroll 8
+    for (int d = 0; d < depth; ++d) {
+      const float4 r4 = *reinterpret_cast<const float4*>(rows + d * pitch + 4 * ty), c4 = *reinterpret_cast<const float4*>(cols + d * OV + 4 * tx);
+      const float r[4] = {r4.x, r4.y, r4.z, r4.w}, c[4] = {c4.x, c4.y, c4.z, c4.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[i][j] = fmaf(r[i], c[j], o[i][j]);
+    }
+  };
+  mac(q_s, CC, S_s, dim);
+  mac(b_s, BP, u_s, min(CC, 4 * ty + 4));      // B is zero beyond the diagonal
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int t = 4 * ty + i, col = colb + 4 * tx;
+    if (t >= n) continue;
+    float* dst = a.out + (size_t)(c0 + t) * a.out_stride + (size_t)head * vdim + col;
+    if (vdim % 4 == 0 && (uintptr_t)dst % 16 == 0) {
+      if (col < vdim) *reinterpret_cast<float4*>(dst) = make_float4(o[i][0], o[i][1], o[i][2], o[i][3]);
+      continue;
+    }
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+      if (col + c < vdim) dst[c] = o[i][c];
+  }
+}
+
 template <bool CH>
-int launch_chunks(const PrepArgs& p, WalkArgs w, int n_tokens, int dtype, cudaStream_t stream) {
+int launch_chunks(const PrepArgs& p, const WalkArgs& w, const OutArgs& o, int n_tokens, int dtype, cudaStream_t stream) {
   const int chunks = n_tokens / CC + p.n_entries;
-  const size_t own = CH ? (size_t)(CC + CC - CB + 2 * CB) * (p.dim + 1) : (size_t)CC;
-  const size_t smem = ((size_t)2 * CC * (p.dim + 1) + CC * (CC + 1) + CC + own) * sizeof(float);
+  const size_t smem = prepare_floats(p.dim, CH) * sizeof(float);
   int rc = dispatch_dtype(dtype, [&](auto* tag) {
     using T = LLMK_ELEM(tag);
     if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prepare_kernel<T, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_kernel(delta_prepare_kernel<T, CH>, dim3(chunks, p.heads), dim3(256), smem, stream, p);
+    launch_kernel(delta_prepare_kernel<T, CH>, dim3(chunks, p.heads), dim3(PT), smem, stream, p);
     LLMK_LAUNCH_CHECK("delta_prepare");
   });
   if (rc) return rc;
-  if (p.dim <= 32) return launch_walk<1, CH>(w, p.n_entries, stream);
-  if (p.dim <= 64) return launch_walk<2, CH>(w, p.n_entries, stream);
-  if (p.dim <= 128) return launch_walk<4, CH>(w, p.n_entries, stream);
-  return launch_walk<8, CH>(w, p.n_entries, stream);
+  if (p.dim <= 32) rc = launch_walk_of<32, CH>(w, p.n_entries, stream);
+  else if (p.dim <= 64) rc = launch_walk_of<64, CH>(w, p.n_entries, stream);
+  else if (p.dim <= 128) rc = launch_walk_of<128, CH>(w, p.n_entries, stream);
+  else rc = launch_walk_of<256, CH>(w, p.n_entries, stream);
+  if (rc) return rc;
+  const size_t osmem = ((size_t)p.dim * (CC + OV) + CC * OV + CC * BP) * sizeof(float);
+  if (osmem > 48 * 1024) cudaFuncSetAttribute(delta_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)osmem);
+  launch_kernel(delta_chunk_out_kernel, dim3(chunks, p.heads, (p.vdim + OV - 1) / OV), dim3(OT), osmem, stream, o);
+  LLMK_LAUNCH_CHECK("delta_chunk_out");
 }
 
 }  // namespace
@@ -797,20 +901,23 @@ LLMK_API int llmk_delta_scan(float* out, long long out_stride, const void* q, co
 
 // The same rule for a step with prompt portions, chunk by chunk (see delta_prepare_kernel).  n_tokens: the step's tokens.
 // Float32 scratch for n_tokens / 32 + n_entries chunks of every head: YQ (dim * 64 floats a chunk and head), K (32 * dim),
-// W (32 * vdim), B (32 * 32), G (1; per_channel: dim).
+// W (32 * vdim), B (32 * 32), G (1; per_channel: dim), S (dim * vdim).
 LLMK_API int llmk_delta_chunk_scan(float* out, long long out_stride, const void* q, const void* k, long long qk_stride,
                                    const void* v, long long v_stride, const void* b, long long b_stride, const void* a,
                                    long long a_stride, const float* a_log, const float* dt_bias, float* state, long long slot_stride,
                                    const int* state_slots, const int* cu_tokens, int n_entries, int n_tokens, int heads,
                                    int qk_heads, int dim, int vdim, float q_scale, float norm_eps, int per_channel, float* YQ, float* K,
-                                   float* W, float* B, float* G, int dtype, cudaStream_t stream) {
+                                   float* W, float* B, float* G, float* S, int dtype, cudaStream_t stream) {
   if (n_entries == 0 || n_tokens == 0) return 0;
   LLMK_REQUIRE(dim > 0 && dim <= 256, "delta_chunk_scan: key size %d (1 to 256)", dim);
   LLMK_REQUIRE(qk_heads > 0 && heads % qk_heads == 0 && vdim > 0, "delta_chunk_scan: %d heads do not divide into %d key heads", heads, qk_heads);
   LLMK_REQUIRE(n_entries <= 65535 && heads <= 65535, "delta_chunk_scan: too many entries or heads for one launch");
-  LLMK_REQUIRE(YQ && K && W && B && G, "delta_chunk_scan: the scratch is missing");
+  LLMK_REQUIRE(YQ && K && W && B && G && S, "delta_chunk_scan: the scratch is missing");
   const PrepArgs p = {q, k, qk_stride, v, v_stride, b, a, b_stride, a_stride, a_log, dt_bias, cu_tokens, n_entries, heads, qk_heads, dim,
-                      vdim, q_scale, norm_eps, YQ, K, W, B, G};
-  const WalkArgs w = {out, out_stride, YQ, K, W, B, G, state, slot_stride, state_slots, cu_tokens, heads, dim, vdim};
-  return per_channel ? launch_chunks<true>(p, w, n_tokens, dtype, stream) : launch_chunks<false>(p, w, n_tokens, dtype, stream);
+                      vdim, q_scale, norm_eps, YQ, K, W, B, G,
+                      dim % 4 == 0 && qk_stride % 4 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)k % 16 == 0 &&
+                          (!per_channel || (a_stride % 4 == 0 && (uintptr_t)a % 16 == 0 && (uintptr_t)dt_bias % 16 == 0))};
+  const WalkArgs w = {YQ, K, G, W, S, state, slot_stride, state_slots, cu_tokens, heads, dim, vdim};
+  const OutArgs o = {out, out_stride, YQ, B, W, S, cu_tokens, n_entries, heads, dim, vdim};
+  return per_channel ? launch_chunks<true>(p, w, o, n_tokens, dtype, stream) : launch_chunks<false>(p, w, o, n_tokens, dtype, stream);
 }

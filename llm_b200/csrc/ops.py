@@ -828,16 +828,16 @@ DELTA_CHUNK = 32       # tokens that the chunk-wise delta rule solves together (
 
 
 def delta_chunk_scratch(n_chunks: int, heads: int, dim: int, vdim: int, per_channel: bool = False):
-    """Float32 element counts of the chunk-wise delta rule's five scratch buffers for n_chunks chunks."""
+    """Float32 element counts of the chunk-wise delta rule's six scratch buffers for n_chunks chunks."""
     c = DELTA_CHUNK
-    return [n_chunks * heads * n for n in (dim * 2 * c, c * dim, c * vdim, c * c, dim if per_channel else 1)]
+    return [n_chunks * heads * n for n in (dim * 2 * c, c * dim, c * vdim, c * c, dim if per_channel else 1, dim * vdim)]
 
 
 def delta_chunk_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b: torch.Tensor, a: torch.Tensor,
                      a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, ctx, heads: int, qk_heads: int, dim: int,
                      vdim: int, q_scale: float, norm_eps: float, scratch, per_channel: bool = False) -> None:
     """delta_scan for a step with prompt portions: the rule chunk by chunk (32 tokens solved together, chunks chained through
-    the state; see delta.cu).  scratch: five flat float32 tensors of at least delta_chunk_scratch(ctx.n_tokens // 32 +
+    the state; see delta.cu).  scratch: six flat float32 tensors of at least delta_chunk_scratch(ctx.n_tokens // 32 +
     ctx.n_entries, ...) elements."""
     _delta_operands(out, q, k, v, b, a, a_log, dt_bias, state, heads, qk_heads, dim, vdim, per_channel)
     T = ctx.n_tokens
@@ -849,7 +849,7 @@ def delta_chunk_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: tor
                                         _ptr(ctx.cu_tokens), c_int(ctx.n_entries), c_int(T), c_int(heads), c_int(qk_heads),
                                         c_int(dim), c_int(vdim), c_float(q_scale), c_float(norm_eps), c_int(int(per_channel)),
                                         *[_ptr(t) for t in scratch], c_int(_kind(q.dtype)), _stream()))
-    count_launches(1)
+    count_launches(2)
 
 
 # ---- matrix memory with exponential gates (mlstm.cu) ----------------------------------------

@@ -365,7 +365,7 @@ class GatedDeltaRule(Part):
             # a step with prompt portions: chunks of 32 tokens solved together, chained through the state
             cap = ws.max_rows // ops.DELTA_CHUNK + ctx.cu_tokens.numel()          # chunks of any step: the buffers' sizes
             sizes = ops.delta_chunk_scratch(cap, H, self.head_dim, self.value_dim, self.channel_decay)
-            scratch = [ws.flat("delta_chunk_" + tag, numel, torch.float32) for tag, numel in zip(("yq", "k", "w", "b", "g"), sizes)]
+            scratch = [ws.flat("delta_chunk_" + tag, numel, torch.float32) for tag, numel in zip(("yq", "k", "w", "b", "g", "s"), sizes)]
             ops.delta_chunk_scan(*operands, scratch, per_channel=self.channel_decay)
         else:
             ops.delta_scan(*operands, per_channel=self.channel_decay)
