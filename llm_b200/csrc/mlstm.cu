@@ -270,15 +270,17 @@ __device__ __forceinline__ void chunk_gates(const float* z, long long z_stride, 
                                             float* b_s, float* g_s, float* h_s) {
   const int lane = threadIdx.x & 31;
   float gi[2], gf[2];
+  const float ib = gt.i_bias[head], fb = gt.f_bias[head];
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
-    const int t = 2 * lane + x;
-    gi[x] = -INFINITY; gf[x] = 0.f;
-    if (t < n) {
-      const float* p = z + (size_t)(c0 + t) * z_stride;
-      gi[x] = soft_cap(p[head] + gt.i_bias[head], gt.cap);
-      gf[x] = log_sigmoid(soft_cap(p[heads + head] + gt.f_bias[head], gt.cap));
-    }
+    const float* p = z + (size_t)(c0 + min(2 * lane + x, n - 1)) * z_stride;
+    gi[x] = p[head]; gf[x] = p[heads + head];
+  }
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const bool on = 2 * lane + x < n;
+    gi[x] = on ? soft_cap(gi[x] + ib, gt.cap) : -INFINITY;
+    gf[x] = on ? log_sigmoid(soft_cap(gf[x] + fb, gt.cap)) : 0.f;
   }
   float sum = gf[0] + gf[1];
 #pragma unroll
@@ -466,6 +468,7 @@ mlstm_chunk_out_kernel(float* __restrict__ out, long long out_stride, const bf16
                        const int* __restrict__ cu_tokens, int n_entries, int heads, int dim, int vdim, Scratch sc) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ float b_s[CC], g_s[CC], h_s[CC], m_s[CC], nq_s[CC];
+  __shared__ __align__(8) float n_s[256];                 // n_0
   pdl_launch_dependents();
   pdl_wait();
   Chunk ch;
@@ -494,6 +497,7 @@ mlstm_chunk_out_kernel(float* __restrict__ out, long long out_stride, const bf16
   bring_rows<CC, THREADS>(q_s, kp, q + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
   bring_rows<CC, THREADS>(k_s, kp, k + (size_t)c0 * stride + (size_t)head * dim, stride, n, dim, dim);
   bring_rows<CC, THREADS>(v_s, VP, v + (size_t)c0 * stride + (size_t)head * vdim + col0, stride, n, min(VT, vdim - col0), VT);
+  if (threadIdx.x < dim) n_s[threadIdx.x] = sc.e[unit * dim + threadIdx.x];
   const float m0 = sc.fm[unit * 4 + 2];
   if (threadIdx.x < 32) {
     chunk_gates(z, z_stride, gt, head, heads, c0, n, b_s, g_s, h_s);
@@ -525,10 +529,10 @@ mlstm_chunk_out_kernel(float* __restrict__ out, long long out_stride, const bf16
   __syncthreads();
   {                                                       // n_0 . q of every token: four threads a token
     const int t = threadIdx.x >> 2, l = threadIdx.x & 3;
-    const float* n0 = sc.e + unit * dim;
     float a = 0.f;
+#pragma unroll 4
     for (int d = 2 * l; d < dim; d += 8) {
-      const float2 nv = *reinterpret_cast<const float2*>(n0 + d);
+      const float2 nv = *reinterpret_cast<const float2*>(n_s + d);
       const float2 qv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(q_s + t * kp + d));
       a = fmaf(nv.x, qv.x, a); a = fmaf(nv.y, qv.y, a);
     }
