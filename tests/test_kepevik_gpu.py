@@ -245,7 +245,7 @@ def test_values_stored_are_the_keys_before_rotation(dtype, H, G, D, dims, page):
         assert torch.equal(v_pages[s // page, :, s % page].cpu().float(), qk[t, H * D:].view(G, D))
 
 
-MLSTM_SIZES = [(1, 4, 4), (2, 16, 24), (3, 10, 6), (2, 48, 64), (4, 32, 72), (1, 100, 130), (2, 128, 128), (1, 256, 8), (5, 7, 67)]
+MLSTM_SIZES = [(1, 4, 4), (2, 16, 24), (3, 10, 6), (3, 48, 56), (4, 32, 72), (1, 100, 130), (2, 128, 128), (1, 256, 8), (5, 7, 67)]
 
 
 def _mlstm_inputs(T, H, D, V, seed, spread=2.0, mean_f=1.5):
